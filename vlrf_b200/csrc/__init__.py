@@ -110,10 +110,10 @@ _SIGNATURES = {
                                   _c_int, _c_void_p, _c_void_p, _c_float, _c_int, _c_float, _c_void_p, _c_void_p],
     "vlrf_attn_window_ex": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_float, _c_float, _c_int, _c_void_p,
-                            _c_void_p, _c_int, _c_void_p, _c_void_p],
+                            _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "vlrf_attn_window_mma_ex": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                                 _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_float,
-                                _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p],
+                                _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "vlrf_embed_bigram": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
                           _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p],
     "vlrf_scale_values": [_c_void_p, ctypes.c_longlong, _c_float, _c_void_p],
@@ -129,6 +129,21 @@ _SIGNATURES = {
                       _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "vlrf_ssd_gate_norm": [_c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                            _c_float, _c_float, _c_void_p],
+        "vlrf_matrix_state_scan": [_c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int,
+        _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_float, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
+        _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+        "vlrf_matrix_state_force_columns": [_c_int],
+        "vlrf_conv_unit": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p,
+        _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+        "vlrf_lowrank_rows": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_float, _c_int,
+        _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_float,
+        _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+        "vlrf_head_rows": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p,
+        _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p],
+        "vlrf_norm_pair_add": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float,
+        _c_float, _c_int, _c_void_p],
+        "vlrf_embed_sinusoid": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
+        _c_int, _c_int, _c_float, _c_void_p, _c_void_p],
     "vlrf_gemm_heads": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                         _c_int, _c_int, _c_void_p],
     "vlrf_gemm_grouped": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
@@ -155,7 +170,7 @@ _SIGNATURES = {
     "vlrf_moe_route_scored": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p,
                               _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p],
     "vlrf_moe_plan": [_c_void_p, _c_void_p, _c_int, _c_void_p],
-    "vlrf_moe_gather": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
+    "vlrf_moe_gather": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                         _c_void_p],
     "vlrf_moe_combine": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
                          _c_void_p, _c_void_p, _c_int, _c_void_p],

@@ -23,6 +23,7 @@
 //   Further parameters (attn_window_ex): softcap c > 0 squashes every score to c · tanh(score / c) after the scale;
 //   keep_first n > 0 lets every query also see the keys at positions below n, whatever the window (they keep their
 //   positions); gate (float32 [T][ld_gate], a logit per query head) multiplies head h's result by sigmoid(gate[t][h]);
+//   slopes (a float32 per query head) take slope_h · (query position − key position) off every score, behind the cap;
 //   sink (one float32 a query head) adds the term exp(sink_h) to the softmax's denominator and nothing to its numerator.
 #include "common.cuh"
 
@@ -224,7 +225,7 @@ attn_window_kernel(const ET* __restrict__ q_in, int ldq, const ET* __restrict__ 
                    const int* __restrict__ block_table, int max_blocks, const int* __restrict__ tok_slot,
                    const int* __restrict__ tok_pos, ET* __restrict__ out, int ld_out, int H, int Hkv, int dk, int dv, int BT,
                    float scale, int window, float out_scale, float softcap, int keep_first, const float* __restrict__ sink,
-                   const float* __restrict__ gate, int ld_gate, int* __restrict__ dev_err) {
+                   const float* __restrict__ gate, int ld_gate, const float* __restrict__ slopes, int* __restrict__ dev_err) {
     pdl_wait();
     pdl_launch_dependents();
     extern __shared__ float q_sm[];  // [AW_WARPS][dk]
@@ -244,6 +245,7 @@ attn_window_kernel(const ET* __restrict__ q_in, int ldq, const ET* __restrict__ 
 #pragma unroll
     for (int i = 0; i < AW_MAX / 32; ++i) acc[i] = 0.f;
     float m = -INFINITY, l = 0.f;
+    const float slope = slopes != nullptr ? slopes[h] : 0.f;     // what a step of distance takes off a score
     const int first = (window > 0) ? max(0, pos - window + 1) : 0;
     const int* table = block_table + (size_t)slot * max_blocks;
     bool lost = false;
@@ -265,6 +267,7 @@ attn_window_kernel(const ET* __restrict__ q_in, int ldq, const ET* __restrict__ 
             float dot = 0.f;
             for (int c = 0; c < dk; ++c) dot = fmaf(q[c], ElemIO<ET>::load(krow + c), dot);
             s = softcap > 0.f ? softcap * tanhf(dot / softcap) : dot;
+            s -= slope * (float)(pos - key);
         }
         const float m_new = fmaxf(m, warp_max(s));      // at least one key of the chunk is valid
         const float p = valid ? expf(s - m_new) : 0.f;
@@ -348,7 +351,7 @@ extern "C" int vlrf_qkv_rope_append(const float* proj, int ld, int q_off, int k_
 extern "C" int vlrf_attn_window_ex(const void* q, int dtype, int ldq, const void* Kc, const void* Vc, const int* block_table,
                                    int max_blocks, const int* tok_slot, const int* tok_pos, void* out, int ld_out, int T, int H,
                                    int Hkv, int dk, int dv, int BT, float scale, int window, float out_scale, float softcap,
-                                   int keep_first, const float* sink, const float* gate, int ld_gate, int* dev_err,
+                                   int keep_first, const float* sink, const float* gate, int ld_gate, const float* slopes, int* dev_err,
                                    cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && H > 0 && Hkv > 0 && max_blocks > 0, "attn_window: bad sizes");
     VLRF_REQUIRE(H % Hkv == 0, "attn_window: %d heads cannot share %d key/value heads", H, Hkv);
@@ -363,12 +366,12 @@ extern "C" int vlrf_attn_window_ex(const void* q, int dtype, int ldq, const void
     if (dtype == VLRF_F32)
         launch_chained(attn_window_kernel<float>, grid, dim3(AW_WARPS * 32), smem, stream, (const float*)q, ldq, (const float*)Kc,
                        (const float*)Vc, block_table, max_blocks, tok_slot, tok_pos, (float*)out, ld_out, H, Hkv, dk, dv, BT, scale,
-                       window, out_scale, softcap, keep_first, sink, gate, ld_gate, dev_err);
+                       window, out_scale, softcap, keep_first, sink, gate, ld_gate, slopes, dev_err);
     else if (dtype == VLRF_BF16)
         launch_chained(attn_window_kernel<__nv_bfloat16>, grid, dim3(AW_WARPS * 32), smem, stream, (const __nv_bfloat16*)q, ldq,
                        (const __nv_bfloat16*)Kc, (const __nv_bfloat16*)Vc, block_table, max_blocks, tok_slot, tok_pos,
                        (__nv_bfloat16*)out, ld_out, H, Hkv, dk, dv, BT, scale, window, out_scale, softcap, keep_first, sink, gate, ld_gate,
-                       dev_err);
+                       slopes, dev_err);
     else
         return vlrf_fail(VLRF_ERR_INVALID_ARG, "attn_window: unknown dtype %d", dtype);
     return vlrf_check_launch("attn_window");
@@ -379,5 +382,5 @@ extern "C" int vlrf_attn_window(const void* q, int dtype, int ldq, const void* K
                                 int Hkv, int dk, int dv, int BT, float scale, int window, float out_scale, int* dev_err,
                                 cudaStream_t stream) {
     return vlrf_attn_window_ex(q, dtype, ldq, Kc, Vc, block_table, max_blocks, tok_slot, tok_pos, out, ld_out, T, H, Hkv, dk, dv, BT,
-                               scale, window, out_scale, 0.f, 0, nullptr, nullptr, 0, dev_err, stream);
+                               scale, window, out_scale, 0.f, 0, nullptr, nullptr, 0, nullptr, dev_err, stream);
 }

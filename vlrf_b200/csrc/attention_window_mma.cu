@@ -18,7 +18,8 @@
 // every query also see the keys at positions below n (the tiles that hold them come first in a CTA's list of tiles,
 // ahead of the window's); sink (a float32 per query head) adds exp(sink_h) to the softmax's denominator where the parts
 // of a row are complete (in the kernel, or in the merge of a cut context); gate (float32 [rows][ld_gate], a logit per
-// query head) multiplies head h's finished result by sigmoid(gate[row][h]), at the same places.
+// query head) multiplies head h's finished result by sigmoid(gate[row][h]), at the same places; slopes (a float32 per
+// query head) take slope_h · (query position − key position) off every score, behind the cap.
 #include "common.cuh"
 
 namespace {
@@ -61,7 +62,8 @@ attn_window_mma_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv_
                        const int* __restrict__ seq_slot, const int* __restrict__ seq_start, const int* __restrict__ seq_pos0,
                        __nv_bfloat16* __restrict__ out, int ld_out, float* __restrict__ partials, int H, int Hkv, int dk, int dv,
                        float scale, int window, float out_scale, int n_split, float softcap, int keep_first,
-                       const float* __restrict__ sink, const float* __restrict__ gate, int ld_gate, int* __restrict__ dev_err) {
+                       const float* __restrict__ sink, const float* __restrict__ gate, int ld_gate, const float* __restrict__ slopes,
+                       int* __restrict__ dev_err) {
     constexpr int KS = DKP + 8, VS = DVP + 8;       // row strides in elements: 16 bytes of padding keep ldmatrix off bank conflicts
     constexpr int WKEYS = DEC ? WM_BK / WM_WARPS : WM_BK;      // keys of a tile that one warp takes
     constexpr int NT_S = WKEYS / 8, NT_O = DVP / 8, KS_QK = DKP / 16, KS_PV = WKEYS / 16;
@@ -140,6 +142,11 @@ attn_window_mma_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv_
     const float cap2 = softcap * 1.4426950408889634f, cap_in = softcap > 0.f ? 2.f / softcap : 0.f;   // (v · cap_in = 2 x log2e / c)
     const int lr[2] = {wrow + g, wrow + g + 8};                                  // this thread's two rows of the tile
     const int q_row[2] = {q_first + lr[0] / R, q_first + lr[1] / R};             // … and their positions
+    float slope2[2] = {0.f, 0.f};                   // what a step of distance takes off a score, in units of log2 e
+    if (slopes != nullptr) {
+        slope2[0] = slopes[hk * R + lr[0] % R] * 1.4426950408889634f;
+        slope2[1] = slopes[hk * R + lr[1] % R] * 1.4426950408889634f;
+    }
 
     for (int i = 0; i < n_kt; ++i) {
         cp_wait<NST - 2>();                         // everything but the newest NST − 2 groups has landed: tile i (and the queries)
@@ -179,8 +186,9 @@ attn_window_mma_kernel(const __nv_bfloat16* __restrict__ q, int ldq, const __nv_
                     float v = s[j][e] * sl2;
                     if (softcap > 0.f)      // c · tanh(x / c) = c · (1 − 2 / (2^(2x log2e / c) + 1)), in units of log2 e
                         v = cap2 * (1.f - __fdividef(2.f, exp2f(v * cap_in) + 1.f));
+                    const int key = k_base + wkey + j * 8 + 2 * t + (e & 1);
+                    v = fmaf(slope2[r], (float)(key - q_row[r]), v);
                     if (need_mask) {
-                        const int key = k_base + wkey + j * 8 + 2 * t + (e & 1);
                         if (key > q_row[r] || (window > 0 && key <= q_row[r] - window && key >= keep_first)) v = -INFINITY;
                     }
                     s[j][e] = v;
@@ -337,7 +345,8 @@ template <int DKP, int DVP, bool DEC>
 int launch_window_mma(const void* q, int ldq, const void* Kc, const void* Vc, const int* block_table, int max_blocks,
                       const int* seq_slot, const int* seq_start, const int* seq_pos0, void* out, int ld_out, float* partials,
                       int n_seqs, int max_new, int H, int Hkv, int dk, int dv, float scale, int window, float out_scale, int n_split,
-                      float softcap, int keep_first, const float* sink, const float* gate, int ld_gate, int* dev_err, cudaStream_t stream) {
+                      float softcap, int keep_first, const float* sink, const float* gate, int ld_gate, const float* slopes, int* dev_err,
+                      cudaStream_t stream) {
     // stages of a decode step: as many as leave room for two or three CTAs an SM
     constexpr int NST = DEC ? (DKP + DVP <= 160 ? 4 : DKP + DVP <= 224 ? 3 : 2) : 2;
     const size_t smem = (size_t)((DEC ? 16 : 64) * (DKP + 8) + NST * 64 * (DKP + 8) + NST * 64 * (DVP + 8)) * 2;
@@ -353,7 +362,7 @@ int launch_window_mma(const void* q, int ldq, const void* Kc, const void* Vc, co
     cudaError_t e = launch_chained(kern, grid, dim3(WM_WARPS * 32), smem, stream, (const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)Kc,
                                    (const __nv_bfloat16*)Vc, block_table, max_blocks, seq_slot, seq_start, seq_pos0,
                                    (__nv_bfloat16*)out, ld_out, partials, H, Hkv, dk, dv, scale, window, out_scale, n_split, softcap,
-                                   keep_first, sink, gate, ld_gate, dev_err);
+                                   keep_first, sink, gate, ld_gate, slopes, dev_err);
     if (e != cudaSuccess) return vlrf_fail(VLRF_ERR_CUDA, "attn_window_mma: %s", cudaGetErrorString(e));
     return vlrf_check_launch("attn_window_mma");
 }
@@ -370,7 +379,7 @@ extern "C" int vlrf_attn_window_mma_ex(const void* q, int ldq, const void* Kc, c
                                        const int* seq_slot, const int* seq_start, const int* seq_pos0, void* out, int ld_out,
                                        float* partials, int n_seqs, int max_new, int H, int Hkv, int dk, int dv, int BT, float scale,
                                        int window, float out_scale, int n_split, float softcap, int keep_first, const float* sink,
-                                       const float* gate, int ld_gate, int* dev_err, cudaStream_t stream) {
+                                       const float* gate, int ld_gate, const float* slopes, int* dev_err, cudaStream_t stream) {
     VLRF_REQUIRE(vlrf_attn_window_mma_takes(H, Hkv, dk, dv, BT, ldq, ld_out), "attn_window_mma: heads %d/%d, sizes %d and %d, block %d are not taken",
                  H, Hkv, dk, dv, BT);
     VLRF_REQUIRE(n_seqs >= 0 && max_new >= 0 && max_blocks > 0 && window >= 0 && dev_err != nullptr, "attn_window_mma: bad arguments");
@@ -384,9 +393,9 @@ extern "C" int vlrf_attn_window_mma_ex(const void* q, int ldq, const void* Kc, c
     int st = VLRF_ERR_UNSUPPORTED;
     const bool dec = max_new == 1 && H / Hkv <= 16;            // every tile holds one token's heads: the warps deal the keys
 #define GO(A, B) if (kp == A && vp == B) st = dec ? launch_window_mma<A, B, true>(q, ldq, Kc, Vc, block_table, max_blocks, seq_slot, seq_start, seq_pos0, \
-        out, ld_out, partials, n_seqs, max_new, H, Hkv, dk, dv, scale, window, out_scale, n_split, softcap, keep_first, sink, gate, ld_gate, dev_err, stream) \
+        out, ld_out, partials, n_seqs, max_new, H, Hkv, dk, dv, scale, window, out_scale, n_split, softcap, keep_first, sink, gate, ld_gate, slopes, dev_err, stream) \
         : launch_window_mma<A, B, false>(q, ldq, Kc, Vc, block_table, max_blocks, seq_slot, seq_start, seq_pos0, \
-        out, ld_out, partials, n_seqs, max_new, H, Hkv, dk, dv, scale, window, out_scale, n_split, softcap, keep_first, sink, gate, ld_gate, dev_err, stream);
+        out, ld_out, partials, n_seqs, max_new, H, Hkv, dk, dv, scale, window, out_scale, n_split, softcap, keep_first, sink, gate, ld_gate, slopes, dev_err, stream);
     GO(32, 32) GO(32, 64) GO(32, 96) GO(32, 128) GO(64, 32) GO(64, 64) GO(64, 96) GO(64, 128)
     GO(96, 32) GO(96, 64) GO(96, 96) GO(96, 128) GO(128, 32) GO(128, 64) GO(128, 96) GO(128, 128)
 #undef GO
@@ -405,5 +414,5 @@ extern "C" int vlrf_attn_window_mma(const void* q, int ldq, const void* Kc, cons
                                     int window, float out_scale, int n_split, int* dev_err, cudaStream_t stream) {
     return vlrf_attn_window_mma_ex(q, ldq, Kc, Vc, block_table, max_blocks, seq_slot, seq_start, seq_pos0, out, ld_out, partials,
                                    n_seqs, max_new, H, Hkv, dk, dv, BT, scale, window, out_scale, n_split, 0.f, 0, nullptr, nullptr, 0,
-                                   dev_err, stream);
+                                   nullptr, dev_err, stream);
 }

@@ -13,8 +13,9 @@
 //                output by itself, instead of the softmax over all of them; everything else is the same.
 //   moe_plan     offsets[e] = rows of the experts before e (E + 1 entries); the counters are left zero.
 //   moe_gather   pair (token, j) gets row offsets[expert] + rank of the expert-sorted buffer: the token's input row
-//                is copied there and the row's number kept.
-//   moe_combine  y[t] = Σ_j weight[t][j] · expert_out[row[t][j]] (+ gate[t] · shared_out[t]) (+ residual[t]), float32,
+//                is copied there, multiplied by the pair's weight where the weights act on the experts' inputs, and the
+//                row's number kept.
+//   moe_combine  y[t] = Σ_j weight[t][j] · expert_out[row[t][j]] (no weights: 1) (+ gate[t] · shared_out[t]) (+ residual[t]), float32,
 //                j in order.
 //
 // Between gather and combine run the grouped products (gemm_heads.cu: gemm_grouped) and the gate (norm_rms.cu).
@@ -203,7 +204,7 @@ __global__ void moe_plan_kernel(int* __restrict__ counts, int* __restrict__ offs
 template <typename ET>
 __global__ void __launch_bounds__(128)
 moe_gather_kernel(const ET* __restrict__ h, int width, const int* __restrict__ ids, const int* __restrict__ rank,
-                  const int* __restrict__ offsets, ET* __restrict__ sorted, int* __restrict__ row_of, int top) {
+                  const int* __restrict__ offsets, const float* __restrict__ wts, ET* __restrict__ sorted, int* __restrict__ row_of, int top) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
     const int pair = blockIdx.x;
@@ -213,6 +214,11 @@ moe_gather_kernel(const ET* __restrict__ h, int width, const int* __restrict__ i
     if (threadIdx.x == 0) row_of[pair] = row;
     const ET* src = h + (size_t)(pair / top) * width;
     ET* dst = sorted + (size_t)row * width;
+    if (wts != nullptr) {
+        const float f = wts[pair];
+        for (int i = threadIdx.x; i < width; i += 128) ElemIO<ET>::store(dst + i, f * ElemIO<ET>::load(src + i));
+        return;
+    }
     for (int i = threadIdx.x; i < width; i += 128) dst[i] = src[i];
 }
 
@@ -228,7 +234,7 @@ moe_combine_kernel(const float* __restrict__ expert_out, int width, const int* _
         float s = 0.f;
         for (int j = 0; j < top; ++j) {
             const int row = row_of[(size_t)t * top + j];
-            if (row >= 0) s = fmaf(wts[(size_t)t * top + j], expert_out[(size_t)row * width + i], s);
+            if (row >= 0) s = fmaf(wts != nullptr ? wts[(size_t)t * top + j] : 1.f, expert_out[(size_t)row * width + i], s);
             else if (ids != nullptr && ids[(size_t)t * top + j] == -2)                      // an expert that returns its input
                 s = fmaf(wts[(size_t)t * top + j], ElemIO<HT>::load(h + (size_t)t * width + i), s);
         }
@@ -275,13 +281,13 @@ extern "C" int vlrf_moe_plan(int* counts, int* offsets, int E, cudaStream_t stre
 }
 
 extern "C" int vlrf_moe_gather(const void* h, int dtype, int width, const int* ids, const int* rank, const int* offsets,
-                               void* sorted, int* row_of, int T, int top, cudaStream_t stream) {
+                               const float* wts, void* sorted, int* row_of, int T, int top, cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && width > 0 && top > 0, "moe_gather: bad sizes");
     if (T == 0) return VLRF_OK;
     if (dtype == VLRF_F32)
-        launch_chained(moe_gather_kernel<float>, dim3(T * top), dim3(128), (size_t)(0), stream, (const float*)h, width, ids, rank, offsets, (float*)sorted, row_of, top);
+        launch_chained(moe_gather_kernel<float>, dim3(T * top), dim3(128), (size_t)(0), stream, (const float*)h, width, ids, rank, offsets, wts, (float*)sorted, row_of, top);
     else if (dtype == VLRF_BF16)
-        launch_chained(moe_gather_kernel<__nv_bfloat16>, dim3(T * top), dim3(128), (size_t)(0), stream, (const __nv_bfloat16*)h, width, ids, rank, offsets, (__nv_bfloat16*)sorted, row_of, top);
+        launch_chained(moe_gather_kernel<__nv_bfloat16>, dim3(T * top), dim3(128), (size_t)(0), stream, (const __nv_bfloat16*)h, width, ids, rank, offsets, wts, (__nv_bfloat16*)sorted, row_of, top);
     else return vlrf_fail(VLRF_ERR_INVALID_ARG, "moe_gather: unknown dtype %d", dtype);
     return vlrf_check_launch("moe_gather");
 }
@@ -290,6 +296,7 @@ extern "C" int vlrf_moe_combine(const float* expert_out, int width, const int* r
                                 const float* shared_out, const float* gate, const float* residual, float* y, int T,
                                 const int* ids, const void* h, int h_dtype, cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && width > 0 && top > 0, "moe_combine: bad sizes");
+    VLRF_REQUIRE(wts != nullptr || ids == nullptr, "moe_combine: experts that return their input need weights");
     VLRF_REQUIRE((ids == nullptr) == (h == nullptr), "moe_combine: experts that return their input need ids and the input rows");
     if (T == 0) return VLRF_OK;
     if (h != nullptr && h_dtype == VLRF_BF16)

@@ -868,16 +868,19 @@ def moe_plan(counts, offsets, n_experts: int) -> None:
     call("vlrf_moe_plan", _ptr(counts), _ptr(offsets), n_experts, _stream())
 
 
-def moe_gather(h, ids, rank, offsets, sorted_rows, row_of, n_tokens: int, top: int) -> None:
+def moe_gather(h, ids, rank, offsets, sorted_rows, row_of, n_tokens: int, top: int, wts=None) -> None:
+    """The tokens' input rows sorted by expert; with `wts` (float32 [T, top]) every copied row times its pair's weight."""
+    if wts is not None:
+        _dev(wts, "wts", torch.float32)
     _dev(h, "h"); _dev(sorted_rows, "sorted_rows", h.dtype); _dev(row_of, "row_of", torch.int32)
     if sorted_rows.shape[1] != h.shape[1] or sorted_rows.shape[0] < n_tokens * top or h.shape[0] < n_tokens:
         raise KernelError("moe_gather: sizes do not match")
-    call("vlrf_moe_gather", _ptr(h), dtype_code(h.dtype), h.shape[1], _ptr(ids), _ptr(rank), _ptr(offsets), _ptr(sorted_rows),
+    call("vlrf_moe_gather", _ptr(h), dtype_code(h.dtype), h.shape[1], _ptr(ids), _ptr(rank), _ptr(offsets), _ptr(wts), _ptr(sorted_rows),
          _ptr(row_of), n_tokens, top, _stream())
 
 
 def moe_combine(expert_out, row_of, wts, top: int, shared_out, gate, y, n_tokens: int, residual=None, ids=None, h=None) -> None:
-    """y[t] = Σ_j wts[t, j] · expert_out[row_of[t, j]] (+ gate[t] · shared_out[t]) (+ residual[t]), float32.  With `ids` and
+    """y[t] = Σ_j wts[t, j] · expert_out[row_of[t, j]] (wts None: 1) (+ gate[t] · shared_out[t]) (+ residual[t]), float32.  With `ids` and
     the experts' input rows `h`: a pair whose id is −2 (an expert that returns its input) adds wts[t, j] · h[t]."""
     _dev(expert_out, "expert_out", torch.float32); _dev(y, "y", torch.float32)
     if (ids is None) != (h is None):
@@ -1033,6 +1036,13 @@ def qkv_rope_append(proj, q_off: int, k_off: int, v_off: int, freq, rot: int, q_
          1 if interleaved else 0, float(magnitude), _ptr(dev_err), _stream())
 
 
+def _check_slopes(slopes, n_heads: int) -> None:
+    if slopes is not None:
+        _dev(slopes, "slopes", torch.float32)
+        if slopes.numel() != n_heads:
+            raise KernelError("attention_window: one slope per query head")
+
+
 def _check_head_gate(gate, n_rows: int, n_heads: int) -> None:
     if gate is not None:
         _rows(gate, "gate", torch.float32)
@@ -1042,12 +1052,13 @@ def _check_head_gate(gate, n_rows: int, n_heads: int) -> None:
 
 def attention_window(q, k_cache, v_cache, block_table, tok_slot, tok_pos, out, n_tokens: int, n_heads: int, n_kv_heads: int,
                      dk: int, dv: int, scale: float, window: int, out_scale: float, dev_err, *, softcap: float = 0.0,
-                     keep_first: int = 0, sink=None, gate=None) -> None:
+                     keep_first: int = 0, sink=None, gate=None, slopes=None) -> None:
     """Each token's queries attend the visible keys of its slot; out may be a range of columns of wider rows.  softcap > 0
     squashes the scaled scores; keys at positions below keep_first stay visible whatever the window; sink: float32
     [heads], exp(sink) joins the softmax's denominator; gate: float32 [T, ≥ heads] (a range of columns of wider rows will
-    do), head h's result times sigmoid(gate[t, h])."""
+    do), head h's result times sigmoid(gate[t, h]); slopes: float32 [heads], slope · distance is taken off every score."""
     _check_head_gate(gate, n_tokens, n_heads)
+    _check_slopes(slopes, n_heads)
     if sink is not None:
         _dev(sink, "sink", torch.float32)
         if sink.numel() != n_heads:
@@ -1062,7 +1073,7 @@ def attention_window(q, k_cache, v_cache, block_table, tok_slot, tok_pos, out, n
     call("vlrf_attn_window_ex", _ptr(q), dtype_code(q.dtype), q.shape[1], _ptr(k_cache), _ptr(v_cache), _ptr(block_table),
          block_table.shape[1], _ptr(tok_slot), _ptr(tok_pos), _ptr(out), out.stride(0), n_tokens, n_heads, n_kv_heads, dk, dv, bt,
          float(scale), int(window), float(out_scale), float(softcap), int(keep_first), _ptr(sink), _ptr(gate),
-         gate.stride(0) if gate is not None else 0, _ptr(dev_err), _stream())
+         gate.stride(0) if gate is not None else 0, _ptr(slopes), _ptr(dev_err), _stream())
 
 
 # ---- a state-space recurrence with a matrix state per head -----------------------------------------------------------------
@@ -1140,7 +1151,8 @@ def window_decode_splits(n_rows: int, n_kv_heads: int, max_context: int, window:
 
 
 def attention_window_step(q, k_cache, v_cache, block_table, out, ctx, n_heads: int, n_kv_heads: int, dk: int, dv: int, scale: float,
-                          window: int, out_scale: float, *, softcap: float = 0.0, keep_first: int = 0, sink=None, gate=None) -> None:
+                          window: int, out_scale: float, *, softcap: float = 0.0, keep_first: int = 0, sink=None, gate=None,
+                          slopes=None) -> None:
     """The attention of a step (prompt tokens, single tokens or a mix) with the kernel that suits it: bfloat16 sizes that
     the tensor-core kernel takes go there (a decode step's contexts cut into parts), everything else to the kernel
     that takes a warp per token and head."""
@@ -1158,16 +1170,124 @@ def attention_window_step(q, k_cache, v_cache, block_table, out, ctx, n_heads: i
             if sink.numel() != n_heads:
                 raise KernelError("attention_window: one sink per query head")
         _check_head_gate(gate, ctx.n_tokens, n_heads)
+        _check_slopes(slopes, n_heads)
         call("vlrf_attn_window_mma_ex", _ptr(q), q.shape[1], _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
              _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(out), out.stride(0), _ptr(partials), ctx.n_seqs,
              ctx.max_new, n_heads, n_kv_heads, dk, dv, bt, float(scale), int(window), float(out_scale), n_split, float(softcap),
-             int(keep_first), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(ctx.dev_err), _stream())
+             int(keep_first), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(slopes), _ptr(ctx.dev_err), _stream())
         return
     attention_window(q, k_cache, v_cache, block_table, ctx.tok_slot, ctx.tok_pos, out, ctx.n_tokens, n_heads, n_kv_heads, dk, dv,
-                     scale, window, out_scale, ctx.dev_err, softcap=softcap, keep_first=keep_first, sink=sink, gate=gate)
+                     scale, window, out_scale, ctx.dev_err, softcap=softcap, keep_first=keep_first, sink=sink, gate=gate, slopes=slopes)
 
 
 def ssd_scan_step(xbc, proj, dt_off: int, dt_bias, a_log, d_skip, state, ctx, y, n_heads: int, n_groups: int, n_state: int, p: int) -> None:
     """The recurrence of a step with the kernel that suits it."""
     ssd_scan(xbc, proj, dt_off, dt_bias, a_log, d_skip, state, ctx.seq_slot, ctx.seq_start, ctx.seq_pos0, y, ctx.n_seqs, n_heads,
              n_groups, n_state, p, ctx.max_new)
+
+
+# ---- recurrences with a matrix state per head ------------------------------------------------------------------------------
+
+#: kinds of `matrix_state_scan` (see the kernel library's header), the most state rows and columns, channels of a
+#: convolved head and taps
+MATRIX_STATE_KINDS = {"decayed": 0, "delta": 1, "stabilized": 2}
+MATRIX_STATE_MAX_ROWS, MATRIX_STATE_MAX_COLUMNS, CONV_UNIT_MAX_HEAD, CONV_UNIT_MAX_TAPS = 512, 4096, 512, 16
+LOWRANK_FUNCTIONS = {"plain": 0, "sigmoid_power": 1, "softplus_decay": 2}
+
+
+def embed_sinusoid(table, freq, scale: float, ctx, out) -> None:
+    """out[t] = table[token] · scale + the position in sinusoids: float32 [T, d]; freq float64 [⌈d/2⌉]."""
+    _dev(table, "table"); _dev(freq, "freq", torch.float64); _dev(out, "out", torch.float32)
+    V, d = table.shape
+    if out.shape[0] < ctx.n_tokens or out.shape[1] != d or freq.numel() != (d + 1) // 2:
+        raise KernelError("embed_sinusoid: sizes do not match")
+    call("vlrf_embed_sinusoid", _ptr(table), dtype_code(table.dtype), _ptr(ctx.tokens), _ptr(ctx.tok_slot), _ptr(ctx.tok_pos), _ptr(freq),
+         _ptr(out), ctx.n_tokens, d, V, float(scale), _ptr(ctx.dev_err), _stream())
+
+
+def matrix_state_scan(kind: str, q, k, v, state, ctx, y, n_heads: int, n_groups: int, rows: int, cols: int, *, q_scale: float,
+                      decay=None, s0=None, s1=None, cap: float = 0.0, den=None) -> None:
+    """The recurrence of a step over every sequence's new tokens, from and into the state rows (see the kernel library's
+    header): float32 q, k [T, groups·rows], v [T, heads·cols] (column ranges of wider rows will do), decay [T, heads·rows],
+    s0, s1 [T, heads or groups], state [slots, 2, state_row]; y [T, heads·cols], den [T, heads·2]."""
+    T = ctx.n_tokens
+    for name, t, n in (("q", q, n_groups * rows), ("k", k, n_groups * rows), ("v", v, n_heads * cols), ("decay", decay, n_heads * rows),
+                       ("s0", s0, n_heads), ("s1", s1, n_groups if kind == "delta" else n_heads), ("y", y, n_heads * cols),
+                       ("den", den, 2 * n_heads)):
+        if t is not None:
+            _rows(t, name, torch.float32)
+            if t.shape[0] < T or t.shape[1] < n:
+                raise KernelError(f"matrix_state_scan: {name} does not match")
+    _dev(state, "state", torch.float32)
+    if state.dim() != 3 or state.shape[1] != 2 or (den is not None and den.stride(0) != 2 * n_heads):
+        raise KernelError("matrix_state_scan: the state is [slots, 2, row] and the denominators are [T, heads·2]")
+    ld = lambda t: t.stride(0) if t is not None else 0   # noqa: E731
+    call("vlrf_matrix_state_scan", MATRIX_STATE_KINDS[kind], _ptr(q), ld(q), _ptr(k), ld(k), _ptr(v), ld(v), _ptr(decay), ld(decay),
+         _ptr(s0), ld(s0), _ptr(s1), ld(s1), float(q_scale), float(cap), _ptr(state), state.shape[2], _ptr(ctx.seq_slot),
+         _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(y), ld(y), _ptr(den), ctx.n_seqs, ctx.max_new, n_heads, n_groups, rows, cols,
+         _stream())
+
+
+def conv_unit(proj, x_off: int, weight, state, conv_off: int, ctx, out, kq, n_heads: int, n_groups: int, rows: int, cols: int) -> None:
+    """Causal convolution, x·sigmoid(x) and unit norms of queries and keys (see the kernel library's header): weight float32
+    [channels, taps]; out float32 [T, channels]; kq float32 [T, groups] receives k · q."""
+    _rows(proj, "proj", torch.float32); _dev(weight, "weight", torch.float32); _dev(state, "state", torch.float32)
+    _dev(out, "out", torch.float32); _dev(kq, "kq", torch.float32)
+    channels, taps = weight.shape
+    T = ctx.n_tokens
+    if channels != 2 * n_groups * rows + n_heads * cols or out.shape[1] != channels or kq.shape[1] != n_groups or state.dim() != 3 \
+            or state.shape[1] != 2 or min(out.shape[0], kq.shape[0], proj.shape[0]) < T:
+        raise KernelError("conv_unit: sizes do not match")
+    call("vlrf_conv_unit", _ptr(proj), proj.stride(0), x_off, _ptr(weight), taps, _ptr(state), state.shape[2], conv_off, _ptr(ctx.seq_slot),
+         _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(out), _ptr(kq), ctx.n_seqs, ctx.max_new, n_heads, n_groups, rows, cols, _stream())
+
+
+def lowrank_rows(parts, n_rows: int) -> None:
+    """One or two short products behind short products in one launch.  A part: (a float32 rows [T, rank], w [cols, rank],
+    out float32 [T, cols], function, options) with function "plain", "sigmoid_power" (options tau, bias) or
+    "softplus_decay" (options a_log, per, bias)."""
+    args, dtype = [], parts[0][1].dtype
+    for a, w, out, fn, opt in parts:
+        _rows(a, "a", torch.float32); _dev(w, "w", dtype); _rows(out, "out", torch.float32)
+        cols, rank = w.shape
+        bias, a_log, per = opt.get("bias"), opt.get("a_log"), int(opt.get("per", 1))
+        for name, t, n in (("bias", bias, cols), ("a_log", a_log, -(-cols // per))):
+            if t is not None:
+                _dev(t, name, torch.float32)
+                if t.numel() != n:
+                    raise KernelError(f"lowrank_rows: {name} does not match")
+        if a.shape[1] != rank or out.shape[1] < cols or min(a.shape[0], out.shape[0]) < n_rows:
+            raise KernelError("lowrank_rows: sizes do not match")
+        args += [_ptr(a), a.stride(0), rank, _ptr(w), _ptr(bias), _ptr(a_log), LOWRANK_FUNCTIONS[fn], float(opt.get("tau", 1.0)), per,
+                 _ptr(out), out.stride(0), cols]
+    if len(parts) == 1:
+        args += [0, 0, 0, 0, 0, 0, 0, 1.0, 1, 0, 0, 0]
+    call("vlrf_lowrank_rows", *args, dtype_code(dtype), n_rows, _stream())
+
+
+def head_rows(y, weight, gate, act: str, out, n_rows: int, n_heads: int, cols: int, eps: float, factor: float = 1.0, den=None) -> None:
+    """out[t, h·cols + i] = factor · o / rms(o) · weight · act(gate) per head, o = y (divided by max(|den₀|, den₁) + 1e-6 where
+    den float32 [T, heads·2] is given); weight of cols or heads·cols numbers; act "silu" or "sigmoid"."""
+    _rows(y, "y", torch.float32); _rows(gate, "gate", torch.float32); _rows(out, "out"); _dev(weight, "weight", torch.float32)
+    n = n_heads * cols
+    if min(y.shape[1], gate.shape[1], out.shape[1]) < n or min(y.shape[0], gate.shape[0], out.shape[0]) < n_rows \
+            or weight.numel() not in (cols, n):
+        raise KernelError("head_rows: sizes do not match")
+    if den is not None:
+        _dev(den, "den", torch.float32)
+        if den.numel() < 2 * n_heads * n_rows or den.shape[1] != 2 * n_heads:
+            raise KernelError("head_rows: the denominators do not match")
+    call("vlrf_head_rows", _ptr(y), y.stride(0), _ptr(den), _ptr(weight), 1 if weight.numel() == n and n_heads > 1 else 0, _ptr(gate),
+         gate.stride(0), GATE[act], _ptr(out), dtype_code(out.dtype), out.stride(0), n_rows, n_heads, cols, float(eps), float(factor),
+         _stream())
+
+
+def norm_pair_add(a, b, wa, wb, x, n_rows: int, eps: float, factor: float, accumulate: bool = True) -> None:
+    """x[r] (+)= factor · (RMSnorm(a[r]) · wa + RMSnorm(b[r]) · wb), float32."""
+    for name, t in (("a", a), ("b", b), ("x", x), ("wa", wa), ("wb", wb)):
+        _dev(t, name, torch.float32)
+    d = x.shape[1]
+    if a.shape[1] != d or b.shape[1] != d or wa.numel() != d or wb.numel() != d or min(a.shape[0], b.shape[0], x.shape[0]) < n_rows:
+        raise KernelError("norm_pair_add: sizes do not match")
+    call("vlrf_norm_pair_add", _ptr(a), _ptr(b), _ptr(wa), _ptr(wb), _ptr(x), n_rows, d, float(eps), float(factor), 1 if accumulate else 0,
+         _stream())

@@ -17,6 +17,8 @@
 //   twice, a step reading the copy of the parity of the position it begins at and writing the copy of the parity of the
 //   position it ends at, so a step of one token leaves what it read and may run twice.  The CTA of a sequence's first
 //   token of the step also keeps the sequence's last token of the step, after its own read of the kept one.
+// embed_sinusoid: x[t] = table[token[t]] · scale + the position in sinusoids (entry 2i the sine, entry 2i + 1 the cosine of
+//   position · freq[i]), one stream.
 // softcap: v ← cap · tanh(v / cap) over float32 rows (logits).  scale_values: v ← v · factor.
 #include "common.cuh"
 
@@ -41,6 +43,33 @@ embed_streams_kernel(const WT* __restrict__ table, const int* __restrict__ token
     for (int i = threadIdx.x; i < d; i += ST_THREADS) {
         const float v = ElemIO<WT>::load(row + i) * scale;
         for (int s = 0; s < S; ++s) out[(size_t)s * d + i] = v;
+    }
+}
+
+// The angle is formed in 64-bit and brought into −π … π before the 32-bit sine and cosine, so that a far position loses nothing.
+template <typename WT>
+__global__ void __launch_bounds__(ST_THREADS)
+embed_sinusoid_kernel(const WT* __restrict__ table, const int* __restrict__ tokens, const int* __restrict__ tok_slot,
+                      const int* __restrict__ tok_pos, const double* __restrict__ freq, float* __restrict__ x, int d, int V, float scale,
+                      int* __restrict__ dev_err) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    if (tok_slot[t] < 0) return;              // padding row (the whole CTA leaves)
+    int id = tokens[t];
+    if (id < 0 || id >= V) {
+        if (threadIdx.x == 0) atomicOr(dev_err, VLRF_DEVERR_TOKEN_RANGE);
+        id = min(max(id, 0), V - 1);
+    }
+    const WT* row = table + (size_t)id * d;
+    float* out = x + (size_t)t * d;
+    const double pos = (double)tok_pos[t], turn = 6.283185307179586476925;
+    for (int i = threadIdx.x; 2 * i < d; i += ST_THREADS) {
+        const double a = pos * freq[i];
+        float sn, cn;
+        sincosf((float)(a - rint(a / turn) * turn), &sn, &cn);
+        out[2 * i] = fmaf(ElemIO<WT>::load(row + 2 * i), scale, sn);
+        if (2 * i + 1 < d) out[2 * i + 1] = fmaf(ElemIO<WT>::load(row + 2 * i + 1), scale, cn);
     }
 }
 
@@ -284,6 +313,22 @@ extern "C" int vlrf_streams_write_read(float* x, const float* mix, const float* 
 #undef GO_S
 #undef GO
     return vlrf_check_launch("streams_write_read");
+}
+
+extern "C" int vlrf_embed_sinusoid(const void* table, int w_dtype, const int* tokens, const int* tok_slot, const int* tok_pos,
+                                   const double* freq, float* x, int T, int d, int V, float scale, int* dev_err, cudaStream_t stream) {
+    VLRF_REQUIRE(T >= 0 && d > 0 && V > 0, "embed_sinusoid: bad sizes T=%d d=%d V=%d", T, d, V);
+    VLRF_REQUIRE(freq != nullptr && dev_err != nullptr, "embed_sinusoid: needs the frequencies and the error word");
+    if (T == 0) return VLRF_OK;
+    if (w_dtype == VLRF_F32)
+        launch_chained(embed_sinusoid_kernel<float>, dim3(T), dim3(ST_THREADS), (size_t)0, stream, (const float*)table, tokens, tok_slot,
+                       tok_pos, freq, x, d, V, scale, dev_err);
+    else if (w_dtype == VLRF_BF16)
+        launch_chained(embed_sinusoid_kernel<__nv_bfloat16>, dim3(T), dim3(ST_THREADS), (size_t)0, stream, (const __nv_bfloat16*)table,
+                       tokens, tok_slot, tok_pos, freq, x, d, V, scale, dev_err);
+    else
+        return vlrf_fail(VLRF_ERR_INVALID_ARG, "embed_sinusoid: unknown dtype %d", w_dtype);
+    return vlrf_check_launch("embed_sinusoid");
 }
 
 extern "C" int vlrf_embed_bigram(const void* table, const void* pairs, int w_dtype, const int* tokens, const int* tok_slot,

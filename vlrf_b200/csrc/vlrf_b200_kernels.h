@@ -229,6 +229,10 @@ int vlrf_streams_write_read(float* x, const float* mix, const float* b, const fl
 int vlrf_softcap(float* v, long long n, float cap, cudaStream_t stream);
 // v ← v · factor over n float32 numbers.
 int vlrf_scale_values(float* v, long long n, float factor, cudaStream_t stream);
+// x[t] = table[tokens[t]] · scale + the token's position in sinusoids: entry 2i the sine and 2i + 1 the cosine of position ·
+// freq[i], freq float64 [⌈d/2⌉]; float32 [T][d].  Padding rows (slot −1) are left alone.
+int vlrf_embed_sinusoid(const void* table, int w_dtype, const int* tokens, const int* tok_slot, const int* tok_pos, const double* freq,
+                        float* x, int T, int d, int V, float scale, int* dev_err, cudaStream_t stream);
 // x[t] = table[tokens[t]] · scale + pairs[row]: float32 [T][d] from tables [V][d] and [buckets + 1][d] of w_dtype; row =
 // (token before · mul_prev + token · mul_cur) mod buckets, or `buckets` at position 0.  The token before is the row above
 // where tok_slot and tok_pos say so, else kept[slot][position & 1]; kept int32 [slots][2] receives every sequence's last
@@ -265,11 +269,12 @@ int vlrf_attn_window(const void* q, int dtype, int ldq, const void* Kc, const vo
 // The same with a cap on the scores (softcap > 0: score ← softcap · tanh(score / softcap), after the scale), keys at
 // positions below keep_first visible whatever the window, and sink (null, or a float32 per query head): exp(sink[h])
 // is one more term of the softmax's denominator, with nothing in the numerator.  gate (null, or float32 [T][ld_gate], a logit
-// per query head): head h's result is multiplied by sigmoid(gate[t][h]).
+// per query head): head h's result is multiplied by sigmoid(gate[t][h]).  slopes (null, or a float32 per query head): slope ·
+// (query position − key position) is taken off every score, behind the cap.
 int vlrf_attn_window_ex(const void* q, int dtype, int ldq, const void* Kc, const void* Vc, const int* block_table, int max_blocks,
                         const int* tok_slot, const int* tok_pos, void* out, int ld_out, int T, int H, int Hkv, int dk, int dv, int BT,
                         float scale, int window, float out_scale, float softcap, int keep_first, const float* sink, const float* gate,
-                        int ld_gate, int* dev_err, cudaStream_t stream);
+                        int ld_gate, const float* slopes, int* dev_err, cudaStream_t stream);
 
 // The same attention on the tensor cores (attention_window_mma.cu; bfloat16): a CTA per key/value head, sequence and tile
 // of 64 (token, query head) rows, for prompt steps (rows seq_start[i] … of q are sequence i's new tokens, the first at
@@ -280,12 +285,12 @@ int vlrf_attn_window_mma(const void* q, int ldq, const void* Kc, const void* Vc,
                          const int* seq_slot, const int* seq_start, const int* seq_pos0, void* out, int ld_out, float* partials,
                          int n_seqs, int max_new, int H, int Hkv, int dk, int dv, int BT, float scale, int window, float out_scale,
                          int n_split, int* dev_err, cudaStream_t stream);
-// … with the cap, the kept first keys, the sinks and the gate per head of vlrf_attn_window_ex.
+// … with the cap, the kept first keys, the sinks, the gate per head and the slopes of vlrf_attn_window_ex.
 int vlrf_attn_window_mma_ex(const void* q, int ldq, const void* Kc, const void* Vc, const int* block_table, int max_blocks,
                             const int* seq_slot, const int* seq_start, const int* seq_pos0, void* out, int ld_out, float* partials,
                             int n_seqs, int max_new, int H, int Hkv, int dk, int dv, int BT, float scale, int window, float out_scale,
-                            int n_split, float softcap, int keep_first, const float* sink, const float* gate, int ld_gate, int* dev_err,
-                            cudaStream_t stream);
+                            int n_split, float softcap, int keep_first, const float* sink, const float* gate, int ld_gate,
+                            const float* slopes, int* dev_err, cudaStream_t stream);
 
 // ---- a state-space recurrence with a matrix state per head (ssd.cu) ----------------------------------------------------------
 // What a sequence keeps lies in `state`, float32 [slots][2][state_row]: per copy the heads' states [H][N][P] and, at
@@ -306,6 +311,34 @@ int vlrf_ssd_scan(const float* xbc, int channels, const float* proj, int ld, int
 // with row stride ld_out.
 int vlrf_ssd_gate_norm(const float* y, const float* proj, int ld, int z_off, const float* w, void* out, int out_dtype, int ld_out,
                        int n_rows, int d, int groups, float eps, float factor, cudaStream_t stream);
+
+// ---- recurrences with a matrix state per head (matrix_state.cu, matrix_state_rows.cu) ----------------------------------------
+// kind 0: S ← diag(a) S + k vᵀ; kind 1: S ← diag(a) S, u = sigmoid(s0)(v − Sᵀk), S ← S + k uᵀ (s1: k · q per group); kind 2: the
+// memory with exponential gates and a running maximum (s0, s1: raw input and forget gate logits, capped by `cap`).  o = Sᵀ q ·
+// q_scale into y [T][H·V]; kind 2 also (n · q · q_scale, exp(−m)) into den [T][H][2].  q, k [T][G·K], v [T][H·V], decay a [T][H·K]
+// float32 (column ranges of wider rows will do).  state float32 [slots][2][state_row], see the source for its layout.
+int vlrf_matrix_state_scan(int kind, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* decay,
+                           int ld_decay, const float* s0, int ld_s0, const float* s1, int ld_s1, float q_scale, float cap, float* state,
+                           int state_row, const int* seq_slot, const int* seq_start, const int* seq_pos0, float* y, int ldy, float* den,
+                           int n_seqs, int max_new, int H, int G, int K, int V, cudaStream_t stream);
+int vlrf_matrix_state_force_columns(int nc);
+// Convolution, x·sigmoid(x) and unit norms of q and k over columns [q: G·K | k: G·K | v: H·V] of the float32 rows `proj`; out
+// [T][2·G·K + H·V]; kq [T][G] = k · q; the kept inputs lie at conv_off of the state rows.
+int vlrf_conv_unit(const float* proj, int ld, int x_off, const float* w, int taps, float* state, int state_row, int conv_off,
+                   const int* seq_slot, const int* seq_start, const int* seq_pos0, float* out, float* kq, int n_seqs, int max_new, int H,
+                   int G, int K, int V, cudaStream_t stream);
+// out[t][c] = f(Σ_r a[t][r] · w[c][r] + bias[c]) for one or two (a1 not null) products; f kind 0: nothing, 1: sigmoid(z)^(1/tau),
+// 2: exp(−exp(a_log[c / per]) · softplus(z)).  a, out, bias, a_log float32; w of w_dtype [cols][rank].
+int vlrf_lowrank_rows(const float* a0, int lda0, int rank0, const void* w0, const float* bias0, const float* a_log0, int kind0, float tau0,
+                      int per0, float* out0, int ldo0, int cols0, const float* a1, int lda1, int rank1, const void* w1, const float* bias1,
+                      const float* a_log1, int kind1, float tau1, int per1, float* out1, int ldo1, int cols1, int w_dtype, int T,
+                      cudaStream_t stream);
+// A head's read-out: divided by (max(|den.x|, den.y) + 1e-6) where den is given, RMS norm over the head, weight, gate (silu or sigmoid).
+int vlrf_head_rows(const float* y, int ldy, const float* den, const float* w, int w_per_head, const float* gate, int ld_gate, int act,
+                   void* out, int out_dtype, int ld_out, int T, int H, int V, float eps, float factor, cudaStream_t stream);
+// x[r] (+)= factor · (RMSnorm(a[r]) · wa + RMSnorm(b[r]) · wb), float32 rows of d columns.
+int vlrf_norm_pair_add(const float* a, const float* b, const float* wa, const float* wb, float* x, int n_rows, int d, float eps, float factor,
+                       int accumulate, cudaStream_t stream);
 
 // ---- products per head and per group (gemm_heads.cu) ------------------------------------------------------------------
 // Y[m][h·y_hs …] = X[m][h·x_hs …] · W[h]ᵀ for every head h < H; W [H][N][K].
@@ -380,7 +413,8 @@ int vlrf_moe_route_scored(const float* z, int ld_z, int E, int top, int groups, 
 // offsets[e] = Σ counts[< e], E + 1 entries; counts are left zero.
 int vlrf_moe_plan(int* counts, int* offsets, int E, cudaStream_t stream);
 // sorted[offsets[ids[p]] + rank[p]] = h[p / top] for every pair p < T·top with an expert; row_of[p] = that row or −1.
-int vlrf_moe_gather(const void* h, int dtype, int width, const int* ids, const int* rank, const int* offsets, void* sorted,
+// With wts (float32 [T][top]; null: none) the copied row is multiplied by the pair's weight, rounded once.
+int vlrf_moe_gather(const void* h, int dtype, int width, const int* ids, const int* rank, const int* offsets, const float* wts, void* sorted,
                     int* row_of, int T, int top, cudaStream_t stream);
 // y[t] = Σ_j wts[t][j] · expert_out[row_of[t][j]] (+ (gate ? gate[t] : 1) · shared_out[t] if shared_out) (+ residual[t]
 // if residual, which may be y), float32.  With ids and h (the experts' input rows, of h_dtype [T][width]): a pair

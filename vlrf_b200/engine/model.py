@@ -97,9 +97,10 @@ class DecoderModel:
         def visit(obj):
             nonlocal total
             if isinstance(obj, torch.Tensor):
-                if obj.data_ptr() not in seen:
-                    seen.add(obj.data_ptr())
-                    total += obj.numel() * obj.element_size()
+                storage = obj.untyped_storage()          # (views of one tensor are counted once, whole)
+                if storage.data_ptr() not in seen:
+                    seen.add(storage.data_ptr())
+                    total += storage.nbytes()
             elif hasattr(obj, "__dict__"):
                 for v in vars(obj).values():
                     visit(v)

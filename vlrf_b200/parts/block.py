@@ -82,6 +82,95 @@ class PreNormBlock:
             ctx.ws.row_stats.forget()
 
 
+@register_part("block", "parallel_sublayers")
+class ParallelSublayersBlock:
+    """x += mixer(h) + ffn(h) with h = norm(x): one norm, both sublayers read its output.  The feed-forward may be absent.
+
+    Parts written in stages (`in_weight`, `in_bias`, `in_width`, `core`, `out_weight`, `merged_width`; a mixer without an output
+    matrix of its own has `from_projection`, a feed-forward with more to do than its staged part has `finish`) share their
+    products: one product of h gives the mixer's and the feed-forward's input columns, float32, each range beginning on a
+    multiple of eight columns; both write their inner rows side by side, and one product over the concatenated output
+    matrices adds the two sublayers to x.  Other parts run one after the other on the same h."""
+
+    leaves_row_stats = False
+
+    def __init__(self, norm1, mixer, feed_forward=None):
+        self.norm1, self.mixer, self.feed_forward = norm1, mixer, feed_forward
+        ff = feed_forward
+        self.joint_in = ff is not None and all(hasattr(p, "in_weight") and hasattr(p, "core") for p in (mixer, ff))
+        self.joint_out = self.joint_in and mixer.out_weight is not None and ff.out_weight is not None
+        if not self.joint_in:
+            return
+
+        def padded(w, b):
+            """The rows of an input product and their bias, with zero rows up to a multiple of eight."""
+            n = -(-w.shape[0] // 8) * 8
+            wp = torch.zeros((n, w.shape[1]), dtype=w.dtype, device=w.device)
+            wp[:w.shape[0]] = w
+            bp = torch.zeros(n, dtype=torch.float32, device=w.device)
+            if b is not None:
+                bp[:w.shape[0]] = b
+            return wp, bp
+        (wm, bm), (wf, bf) = padded(mixer.in_weight, mixer.in_bias), padded(ff.in_weight, ff.in_bias)
+        self.ff_at = wm.shape[0]
+        self.in_weight = torch.cat([wm, wf], dim=0).contiguous()
+        self.in_bias = torch.cat([bm, bf]).contiguous() if mixer.in_bias is not None or ff.in_bias is not None else None
+        # the parts go on with their places in the joint matrices and let go of their own
+        for part, at in ((mixer, 0), (ff, self.ff_at)):
+            rows = self.in_weight[at:at + part.in_width]
+            if hasattr(part, "adopt_in_weight"):
+                part.adopt_in_weight(rows)
+            else:
+                part.in_weight = rows
+        if self.joint_out:
+            m = mixer.merged_width
+            self.out_weight = torch.cat([mixer.out_weight, ff.out_weight], dim=1).contiguous()
+            for part, cols in ((mixer, self.out_weight[:, :m]), (ff, self.out_weight[:, m:])):
+                if hasattr(part, "adopt_out_weight"):
+                    part.adopt_out_weight(cols)
+                else:
+                    part.out_weight = cols
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, view, writes_cache: bool = True) -> None:
+        from ..csrc import ops
+        T, ws, mixer, ff = ctx.n_tokens, ctx.ws, self.mixer, self.feed_forward
+        ws.row_stats.forget()
+        h = ws.get("block_normed", T, x.shape[1], ctx.act_dtype)
+        self.norm1(x, h)
+        if not self.joint_in:
+            mixer.forward(h, x, ctx, view, writes_cache)
+            if ff is not None:
+                ff.forward(h, x, ctx)
+            return
+        n_ff = ff.leading_rows(T) if hasattr(ff, "leading_rows") else ff.in_width
+        n = min(-(-(self.ff_at + n_ff) // 8) * 8, self.in_weight.shape[0])
+        proj = ws.get("sublayers_in_proj", T, n, torch.float32)
+        ops.linear(h, self.in_weight[:n], self.in_bias[:n] if self.in_bias is not None else None, proj)
+        ff_proj = proj[:, self.ff_at:]
+        if self.joint_out:
+            m = mixer.merged_width
+            merged = ws.get("sublayers_merged", T, m + ff.merged_width, ctx.act_dtype)
+            mixer.core(proj[:, :mixer.in_width], merged[:, :m], ctx, view, writes_cache)
+            ff.core(ff_proj, merged[:, m:], ctx, h)
+            ops.linear(merged, self.out_weight, None, x, residual=x)
+        else:
+            if ff.out_weight is not None:
+                u = ws.get("sublayers_ff_inner", T, ff.merged_width, ctx.act_dtype)
+                ff.core(ff_proj, u, ctx, h)
+                ops.linear(u, ff.out_weight, None, x, residual=x)
+            if mixer.out_weight is None:
+                mixer.from_projection(proj[:, :mixer.in_width], x, ctx, view, writes_cache)
+            else:
+                merged = ws.get("sublayers_merged", T, mixer.merged_width, ctx.act_dtype)
+                mixer.core(proj[:, :mixer.in_width], merged, ctx, view, writes_cache)
+                ops.linear(merged, mixer.out_weight, None, x, residual=x)
+        if hasattr(ff, "finish"):
+            ff.finish(h, ff_proj, x, ctx)
+
+
 @register_part("block", "sublayer_norm")
 class SublayerNormBlock:
     """x += norm1(mixer(x)); x += norm2(ffn(x)): the norm acts on each sublayer's output, and the sublayers read the

@@ -26,7 +26,7 @@ class TokenEmbedding:
             if table.dim() != 2 or table.shape[0] < 2 or table.shape[1] != weight.shape[1] or table.dtype != weight.dtype:
                 raise ValueError("TokenEmbedding: the bigram table is [buckets + 1, width] in the embedding's dtype")
             if norm is not None or streams != 1 or getattr(position, "where", None) == "embedding":
-                raise ValueError("TokenEmbedding: a bigram table goes with one stream, no norm and no position table")
+                raise ValueError("TokenEmbedding: a bigram table goes with one stream, no norm and no positions at the embedding")
             buckets = int(table.shape[0]) - 1
             # (a multiplier enters the hash only through its remainder, which keeps every product inside 64 bits)
             self.bigram = (table, buckets, int(mul_prev) % buckets, int(mul_cur) % buckets)
@@ -35,6 +35,11 @@ class TokenEmbedding:
         self.scale, self.streams = float(scale), int(streams)
         if self.streams < 1:
             raise ValueError("TokenEmbedding: at least one stream")
+        self.sinusoid = position if hasattr(position, "frequencies") else None      # positions as sines and cosines, no table
+        if self.sinusoid is not None:
+            if self.sinusoid.width != self.width or self.streams != 1 or norm is not None:
+                raise ValueError("TokenEmbedding: sinusoidal positions of the embedding's width, one stream and no norm")
+            position = None
         if (self.scale != 1.0 or self.streams != 1) and (norm is not None or getattr(position, "where", None) == "embedding"):
             raise ValueError("TokenEmbedding: a scaled or copied embedding takes no norm and no position table")
         self.out_width = self.width * self.streams
@@ -57,12 +62,12 @@ class TokenEmbedding:
     def leaves_row_stats(self) -> bool:
         """The rows are written by a kernel that is handed the step's row statistics (see parts/block.py); a norm
         behind it rewrites them."""
-        return self.norm is None and self.scale == 1.0 and self.streams == 1 and self.bigram is None
+        return self.norm is None and self.scale == 1.0 and self.streams == 1 and self.bigram is None and self.sinusoid is None
 
     def emit_decode(self, program, x: torch.Tensor) -> None:
-        if self.scale != 1.0 or self.streams != 1 or self.bigram is not None:
+        if self.scale != 1.0 or self.streams != 1 or self.bigram is not None or self.sinusoid is not None:
             from .program import NotFusable
-            raise NotFusable("a scaled or copied embedding, or one with a bigram table, is not an operation of the decode program")
+            raise NotFusable("a scaled or copied embedding, or one with a bigram table or sinusoids, is not an operation of the decode program")
         if self.norm is not None:
             from .program import NotFusable
             raise NotFusable("an embedding with a norm behind it is not an operation of the decode program")
@@ -80,6 +85,10 @@ class TokenEmbedding:
             ops.embed_bigram(self.weight, table, buckets, mul_prev, mul_cur, self.scale, state, ctx, x, also=also)
             if also is not None:
                 ctx.ws.input_cast = (x.data_ptr(), ctx.n_tokens, id(ctx))
+            return x
+        if self.sinusoid is not None:
+            ctx.ws.row_stats.forget()
+            ops.embed_sinusoid(self.weight, self.sinusoid.frequencies, self.scale, ctx, x)
             return x
         if self.scale != 1.0 or self.streams != 1:
             ctx.ws.row_stats.forget()

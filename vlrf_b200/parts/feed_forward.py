@@ -73,15 +73,21 @@ class GatedMLP:
             raise ValueError(f"GatedMLP: gate '{activation}' is not one of {', '.join(GATES)}")
         if w_gate.shape != w_up.shape or w_down.shape[1] != w_gate.shape[0] or w_down.shape[0] != w_gate.shape[1]:
             raise ValueError("GatedMLP: the three matrices do not chain")
-        self.w_gate_up = torch.cat([w_gate, w_up], dim=0).contiguous()
-        self.w_down = w_down
+        # in stages, for blocks that join its products with another sublayer's: the rows of the input product, `core` from
+        # its float32 result to the inner rows, the output matrix
+        self.in_weight, self.in_bias, self.in_width = torch.cat([w_gate, w_up], dim=0).contiguous(), None, 2 * w_gate.shape[0]
+        self.out_weight, self.merged_width = w_down, w_gate.shape[0]
         self.activation = activation
         self.inner = w_gate.shape[0]
+
+    def core(self, proj, merged, ctx: StepContext, h=None) -> None:
+        ff = self.inner
+        ops.gate_mul(proj[:, :ff], proj[:, ff:2 * ff], merged, self.activation, ctx.n_tokens, ff)
 
     def forward(self, h, x: torch.Tensor, ctx: StepContext, norm=None, accumulate: bool = True) -> None:
         T, ff = ctx.n_tokens, self.inner
         gu = ctx.ws.get("ffn_gate_up", T, 2 * ff, torch.float32)
-        ops.linear(h, self.w_gate_up, None, gu)
+        ops.linear(h, self.in_weight, None, gu)
         u = ctx.ws.get("ffn_inner", T, ff, ctx.act_dtype)
-        ops.gate_mul(gu[:, :ff], gu[:, ff:], u, self.activation, T, ff)
-        ops.linear(u, self.w_down, None, x, residual=x if accumulate else None)
+        self.core(gu, u, ctx)
+        ops.linear(u, self.out_weight, None, x, residual=x if accumulate else None)

@@ -13,6 +13,7 @@ experts (`n_identity`): the router's last n_identity outputs stand for experts w
 input, so the router has n_identity more rows than there are expert matrices.  `scoring="sigmoid"`: the same rule with
 s = sigmoid(z), each output by itself.  `gate="clamped"` (with `limit`, `gate_alpha`): an expert is
 W_down (g · sigmoid(gate_alpha · g) · (u + 1)) with g = min(W_gate h, limit) and u = clamp(W_up h, −limit, limit).
+`weights_on="input"`: the output is Σ expert(weight · h) instead of Σ weight · expert(h).
 
 Nothing is decided on the host: the router's kernel counts each expert's rows, the tokens' inputs are copied into a
 buffer sorted by expert, and two grouped products (each row block with its expert's matrix) run over it with the gate
@@ -33,7 +34,7 @@ from .registry import register_part
 class RoutedExperts:
     def __init__(self, w_router, b_router, w_gate, w_up, w_down, *, top: int, shared=None, scoring: str = "softmax_chosen",
                  correction=None, groups: int = 1, keep: int = 1, weight_scale: float = 1.0, n_identity: int = 0,
-                 gate: str = "silu", limit: float | None = None, gate_alpha: float = 1.0):
+                 gate: str = "silu", limit: float | None = None, gate_alpha: float = 1.0, weights_on: str = "output"):
         """w_router [E + n_identity, width], b_router [E + n_identity] float32 or None; w_gate (or None), w_up [E, ff, width],
         w_down [E, width, ff]; shared: None or (w_gate [ffs, width], w_up [ffs, width], w_down [width, ffs], w_sg [1, width]
         or None); correction: float32 [E + n_identity] or None."""
@@ -51,6 +52,9 @@ class RoutedExperts:
             raise ValueError(f"routed experts: scoring '{scoring}' is none of 'softmax_chosen', 'softmax_all', 'sigmoid'")
         if gate not in ("silu", "clamped") or (gate == "clamped" and (w_gate is None or limit is None or not limit > 0.0)):
             raise ValueError("routed experts: the experts' gate is 'silu', or 'clamped' with gate matrices and a positive limit")
+        if weights_on not in ("output", "input") or (weights_on == "input" and n_identity):
+            raise ValueError("routed experts: a weight multiplies an expert's 'output' or its 'input' (and then no expert is the identity)")
+        self.weights_on = weights_on
         self.gate, self.limit, self.gate_alpha = gate, float(limit) if limit is not None else 0.0, float(gate_alpha)
         if scoring == "softmax_chosen" and (n_identity or correction is not None or groups != 1 or weight_scale != 1.0):
             raise ValueError("routed experts: identity experts, a correction, groups and a weight scale belong to scoring 'softmax_all'")
@@ -106,15 +110,61 @@ class RoutedExperts:
     fuses_norm = False
     leaves_row_stats = False
 
-    def forward(self, h, x: torch.Tensor, ctx: StepContext, norm=None, accumulate: bool = True) -> None:
+    # ---- in stages, for blocks that join this part's products with another sublayer's: `in_weight` (the router's rows, the
+    # shared expert's gate and up rows behind them), `core` (the shared expert's inner rows), `out_weight` (its down matrix),
+    # and `finish` (the routed experts, added to x).  A shared expert with a gate of its own has no such form.
+    @property
+    def in_weight(self):
+        return self.w_in
+
+    def adopt_in_weight(self, w) -> None:
+        self.w_in = w
+        if self.shared is not None:
+            at = self.n_logits
+            self.shared = (w[at:at + 2 * self.shared[2]], self.shared[1], self.shared[2])
+
+    def adopt_out_weight(self, w) -> None:
+        self.shared = (self.shared[0], w, self.shared[2])
+
+    @property
+    def in_bias(self):
+        return None if self._no_bias else self.b_in
+
+    @property
+    def in_width(self) -> int:
+        return self.w_in.shape[0]
+
+    def leading_rows(self, n_tokens: int) -> int:
+        """Rows of the input product that a step of n_tokens wants: with many rows the shared expert's are a product of
+        their own in the activation dtype, half the bytes."""
+        return self.n_logits if self.shared is not None and n_tokens > ops.SKINNY_MAX_ROWS else self.w_in.shape[0]
+
+    @property
+    def merged_width(self) -> int:
+        return self.shared[2] if self.shared is not None else 0
+
+    @property
+    def out_weight(self):
+        return self.shared[1] if self.shared is not None and not self.shared_gate else None
+
+    def core(self, proj, merged, ctx: StepContext, h=None) -> None:
+        """The shared expert's inner rows from the float32 columns of the input product (few rows), or from h (many)."""
+        T, (w_gu, _, ffs) = ctx.n_tokens, self.shared
+        if self.leading_rows(T) == self.n_logits:
+            su = ctx.ws.get("moe_shared_gate_up", T, 2 * ffs, ctx.act_dtype)
+            ops.linear(h, w_gu, None, su)
+            ops.gate_mul(su[:, :ffs], su[:, ffs:], merged, "silu", T, ffs)
+        else:
+            at = self.n_logits
+            ops.gate_mul(proj[:, at:at + ffs], proj[:, at + ffs:at + 2 * ffs], merged, "silu", T, ffs)
+
+    def finish(self, h, proj, x: torch.Tensor, ctx: StepContext, shared_out=None, accumulate: bool = True) -> None:
+        """The routed experts from the router's logits (the first columns of proj), weighted and summed into x, with the
+        shared expert's output where it is given."""
         T, ws, act = ctx.n_tokens, ctx.ws, ctx.act_dtype
         E, top, width, ff = self.n_experts, self.top, self.width, self.ff
         P = T * top
-        shared_apart = self.shared is not None and T > ops.SKINNY_MAX_ROWS
-        n_in = self.n_logits if shared_apart else self.w_in.shape[0]
-        inp = ws.get("moe_in_proj", T, n_in, torch.float32)
-        ops.linear(h, self.w_in[:n_in], None if self._no_bias else self.b_in[:n_in], inp)
-        z = inp
+        z = proj
         ids = ws.get("moe_ids", T, top, torch.int32)
         rank = ws.get("moe_rank", T, top, torch.int32)
         row_of = ws.get("moe_row_of", T, top, torch.int32)
@@ -129,7 +179,8 @@ class RoutedExperts:
             ops.moe_route(z, E, top, self.shared_gate, ctx.tok_slot, ids, wts, rank, gate, counts, T)
         ops.moe_plan(counts, offsets, max(E, 1))
         rows = ws.get("moe_sorted", P, width, act)
-        ops.moe_gather(h, ids, rank, offsets, rows, row_of, T, top)
+        on_input = self.weights_on == "input"
+        ops.moe_gather(h, ids, rank, offsets, rows, row_of, T, top, wts=wts if on_input else None)
         out = ws.get("moe_expert_out", P, width, torch.float32)
         if E > 0:
             a = ws.get("moe_inner", P, ff, act)
@@ -143,20 +194,21 @@ class RoutedExperts:
             else:
                 ops.linear_grouped(rows, self.w_gate_up, a, offsets, P, act="relu2")     # (the activation in the product's epilogue)
             ops.linear_grouped(a, self.w_down, out, offsets, P)
+        residual = x if accumulate else None
+        if self.n_identity:
+            ops.moe_combine(out, row_of, wts, top, shared_out, gate, x, T, residual=residual, ids=ids, h=h)
+        else:
+            ops.moe_combine(out, row_of, None if on_input else wts, top, shared_out, gate, x, T, residual=residual)
+
+    def forward(self, h, x: torch.Tensor, ctx: StepContext, norm=None, accumulate: bool = True) -> None:
+        T, ws = ctx.n_tokens, ctx.ws
+        n_in = self.leading_rows(T)
+        inp = ws.get("moe_in_proj", T, n_in, torch.float32)
+        ops.linear(h, self.w_in[:n_in], None if self._no_bias else self.b_in[:n_in], inp)
         shared_out = None
         if self.shared is not None:
-            w_gu, w_d, ffs = self.shared
-            sa = ws.get("moe_shared_inner", T, ffs, act)
-            if shared_apart:
-                su = ws.get("moe_shared_gate_up", T, 2 * ffs, act)
-                ops.linear(h, w_gu, None, su)
-                ops.gate_mul(su[:, :ffs], su[:, ffs:], sa, "silu", T, ffs)
-            else:
-                at = self.n_logits
-                ops.gate_mul(inp[:, at:at + ffs], inp[:, at + ffs:at + 2 * ffs], sa, "silu", T, ffs)
-            shared_out = ws.get("moe_shared_out", T, width, torch.float32)
-            ops.linear(sa, w_d, None, shared_out)
-        if self.n_identity:
-            ops.moe_combine(out, row_of, wts, top, shared_out, gate, x, T, residual=x if accumulate else None, ids=ids, h=h)
-        else:
-            ops.moe_combine(out, row_of, wts, top, shared_out, gate, x, T, residual=x if accumulate else None)
+            sa = ws.get("moe_shared_inner", T, self.shared[2], ctx.act_dtype)
+            self.core(inp, sa, ctx, h)
+            shared_out = ws.get("moe_shared_out", T, self.width, torch.float32)
+            ops.linear(sa, self.shared[1], None, shared_out)
+        self.finish(h, inp, x, ctx, shared_out, accumulate)

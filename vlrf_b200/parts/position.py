@@ -26,6 +26,22 @@ class LearnedAbsolutePositions:
         self.max_positions = table.shape[0]
 
 
+@register_part("position", "sinusoidal")
+class SinusoidalPositions:
+    """Entry 2i of a token's embedding grows by sin(p · f_i) and entry 2i + 1 by cos(p · f_i), f_i = base^(−2i/width).  The
+    part holds the frequencies in 64-bit; the embedding's kernel forms the angle in 64-bit, brings it into one turn and takes
+    the 32-bit sine and cosine, so a far position loses nothing.  No table, so nothing bounds a sequence's length."""
+
+    where = "embedding"
+
+    def __init__(self, width: int, device, base: float = 10000.0):
+        if width <= 0 or not base > 0.0:
+            raise ValueError(f"SinusoidalPositions: width {width} and base {base} must be positive")
+        self.width, self.base = int(width), float(base)
+        f = [self.base ** (-2.0 * i / width) for i in range((width + 1) // 2)]
+        self.frequencies = torch.tensor(f, dtype=torch.float64).to(device).contiguous()
+
+
 @register_part("position", "rotary")
 class RotaryPositions:
     """Rotation of queries and keys by position.  Of a vector's first `dims` entries, entry i is paired with entry

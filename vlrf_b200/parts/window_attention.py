@@ -14,12 +14,13 @@ What else is a parameter, each absent by default:
   w_k None (and w_v None)  the layer has no keys and values of its own: it attends another layer's cache with its own
                            queries (the model's schedule says whose), and keeps nothing
   qk_norm "head" | "all"   an RMS norm of queries and of keys ahead of the rotation: every head by itself with one weight
-                           vector of `dim` entries for all heads, or the whole projection as one row; weights `q_norm`,
-                           `k_norm`, `norm_eps`
+                           vector of `dim` entries for all heads (or, without `q_norm` and `k_norm`, no weight), or the
+                           whole projection as one row; weights `q_norm`, `k_norm`, `norm_eps`
   rotary                   its pairing (halves or neighbours), its frequency table and its factor on cosines and sines
   softcap c                score ← c · tanh(score / c) after the scale
   keep_first n             with a window: keys at positions below n stay visible to every later query
   sink [heads]             one more term exp(sink_h) in the denominator of head h's softmax, with nothing in the numerator
+  slopes [heads]           a distance bias: slopes_h · (i − j) is taken off every score (behind the cap, ahead of the softmax)
   w_gate [heads, width]    head h's result is multiplied by sigmoid(w_gate_h · input) ahead of the output projection; the
                            gate's logits ride in the input product as `heads` more float32 columns
 
@@ -41,7 +42,8 @@ from .registry import register_part
 class WindowAttention:
     def __init__(self, w_q, w_k, w_v, w_out, *, n_heads: int, n_kv_heads: int, dim: int, vdim: int, scale: float,
                  b_q=None, b_k=None, b_v=None, window: int = 0, rotary=None, qk_norm: str | None = None, q_norm=None, k_norm=None,
-                 norm_eps: float = 0.0, softcap: float | None = None, keep_first: int = 0, sink=None, w_gate=None):
+                 norm_eps: float = 0.0, softcap: float | None = None, keep_first: int = 0, sink=None, w_gate=None,
+                 slopes=None):
         H, G = int(n_heads), int(n_kv_heads)
         if H <= 0 or G <= 0 or H % G != 0:
             raise ValueError(f"window attention: {H} heads cannot share {G} key/value heads")
@@ -68,11 +70,15 @@ class WindowAttention:
         if qk_norm not in (None, "head", "all"):
             raise ValueError(f"window attention: a norm of queries and keys is 'head' or 'all', not '{qk_norm}'")
         if qk_norm is not None:
+            if qk_norm == "head" and q_norm is None and k_norm is None:      # a norm without weights
+                q_norm = k_norm = torch.ones(dim, dtype=torch.float32, device=w_q.device)
             nq, nk = (dim, dim) if qk_norm == "head" else (H * dim, G * dim)
             if q_norm is None or q_norm.numel() != nq or (self.own_kv and (k_norm is None or k_norm.numel() != nk)) or not norm_eps > 0.0:
                 raise ValueError("window attention: the norm of queries and keys needs its weights and a positive eps")
         if sink is not None and sink.numel() != H:
             raise ValueError("window attention: one sink per query head")
+        if slopes is not None and slopes.numel() != H:
+            raise ValueError("window attention: one slope per query head")
         if w_gate is not None and tuple(w_gate.shape) != (H, w_q.shape[1]):
             raise ValueError("window attention: the gate per head is [heads, width]")
         weights = [w_q] + ([w_k] if w_k is not None else []) + ([w_v] if w_v is not None else [])
@@ -88,6 +94,7 @@ class WindowAttention:
         self.k_norm = k_norm.float().contiguous() if qk_norm is not None and self.own_kv else None
         self.softcap, self.keep_first = float(softcap) if softcap is not None else 0.0, int(keep_first)
         self.sink = sink.float().contiguous() if sink is not None else None
+        self.slopes = slopes.float().contiguous() if slopes is not None else None
         self.q_off, self.k_off = 0, H * dim
         self.v_off = self.k_off if self.values_are_keys else H * dim + G * dim
         width_kv = (G * dim if w_k is not None else 0) + (G * vdim if w_v is not None else 0)
@@ -127,6 +134,7 @@ class WindowAttention:
                             magnitude=float(getattr(self.rotary, "magnitude", 1.0)))
         ops.attention_window_step(q, view.k, view.v, view.block_table, merged, ctx, H, G, self.dim, self.vdim, self.scale,
                                   self.window, factor, softcap=self.softcap, keep_first=self.keep_first, sink=self.sink,
+                                  slopes=self.slopes,
                                   # head h times sigmoid of its gate logit (a float32 column of the input product), applied by
                                   # the attention kernel where it writes the head's result
                                   gate=proj[:, self.gate_off:self.gate_off + H] if self.gate_off is not None else None)

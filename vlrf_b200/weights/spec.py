@@ -17,6 +17,14 @@ from .safetensors_io import WeightError
 
 
 @dataclasses.dataclass(frozen=True)
+class FreeSize:
+    """A size that no configuration key gives: the checkpoint's tensors say it (every tensor that names it alike), and
+    random weights are drawn with `default`."""
+    name: str
+    default: int
+
+
+@dataclasses.dataclass(frozen=True)
 class TensorSpec:
     name: str
     shape: tuple
@@ -25,6 +33,11 @@ class TensorSpec:
     #: "table": integer table (kept int32)
     kind: str = "matrix"
     optional: bool = False
+
+    @property
+    def drawn_shape(self) -> tuple:
+        """The shape that random weights get."""
+        return tuple(n.default if isinstance(n, FreeSize) else n for n in self.shape)
 
 
 @dataclasses.dataclass
@@ -50,6 +63,7 @@ def check_tensors(found: dict, specs: list, *, prefixes: tuple = ("",), ignore: 
     used = set()
     matched: dict[str, torch.Tensor] = {}
     missing, wrong = [], []
+    free: dict[str, int] = {}
     for spec in specs:
         hit = None
         for p in prefixes:
@@ -58,13 +72,16 @@ def check_tensors(found: dict, specs: list, *, prefixes: tuple = ("",), ignore: 
                 break
         if hit is None:
             if not spec.optional:
-                missing.append(f"{spec.name} {list(spec.shape)}")
+                missing.append(f"{spec.name} {[n.name if isinstance(n, FreeSize) else n for n in spec.shape]}")
             continue
         used.add(hit)
         t = found[hit]
-        if tuple(t.shape) != tuple(spec.shape):
-            wrong.append(f"{hit}: expected {list(spec.shape)}, found {list(t.shape)}")
+        # a free size is settled by the first tensor that has it; the others must agree
+        expected = tuple(free.get(n.name, n) if isinstance(n, FreeSize) else n for n in spec.shape)
+        if len(t.shape) != len(expected) or any((f <= 0) if isinstance(n, FreeSize) else f != n for f, n in zip(t.shape, expected)):
+            wrong.append(f"{hit}: expected {[n.name if isinstance(n, FreeSize) else n for n in expected]}, found {list(t.shape)}")
             continue
+        free.update({n.name: int(f) for f, n in zip(t.shape, expected) if isinstance(n, FreeSize)})
         if spec.kind == "table" and t.is_floating_point():
             wrong.append(f"{hit}: expected an integer table, found {t.dtype}")
             continue
