@@ -1030,9 +1030,231 @@ def suposun_kernels(z: dict, hbm_gbs: float, bf16_tflops: float) -> dict:
     return out
 
 
+#: Pelenex at two sizes that resemble a real model's layers, beside a Kotisun of the same width, depth, attention heads and
+#: dense inner size and a recurrent state of about the same size (its closest relative in the framework: windowed attention
+#: beside a recurrence with a matrix state per head), without streams and loop.  Layers: attention beside the decayed memory +
+#: dense; stabilized memory + experts; delta memory + dense; stabilized memory + experts.
+PELENEX_SIZES = {
+    "s": dict(width=1024, heads=16, kv_heads=4, dim=64, window=512, keep=64, gla=(16, 64, 128), lstm=(8, 64, 256), delta=(8, 4, 128, 128),
+              ff_gated=2816, experts=16, top=2, expert_ff=1024, shared_ff=1024, r_heads=32, r_vdim=64, state=64, groups=4, vocab=32000),
+    "m": dict(width=2048, heads=16, kv_heads=2, dim=128, window=1024, keep=128, gla=(32, 128, 128), lstm=(16, 128, 256), delta=(32, 16, 128, 128),
+              ff_gated=5632, experts=32, top=4, expert_ff=1408, shared_ff=2816, r_heads=32, r_vdim=128, state=128, groups=8, vocab=32000),
+}
+
+
+def pelenex_config(z: dict) -> dict:
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+            "mask": {"size": z["window"], "keep_first": z["keep"]}}
+    gh, gk, gv = z["gla"]
+    lh, lk, lv = z["lstm"]
+    dh, dg, dk, dv = z["delta"]
+    dense = {"kind": "dense", "ff": z["ff_gated"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}, "shared": {"ff": z["shared_ff"]}}
+    lstm = {"type": "mlstm", "mixer": {"heads": lh, "dim": lk, "vdim": lv, "gate_cap": 15.0}, "mlp": moe}
+    layers = [{"type": "parallel", "mixer": {"left": left, "right": {"heads": gh, "dim": gk, "vdim": gv, "tau": 16.0}}, "mlp": dense}, lstm,
+              {"type": "channel_delta", "mixer": {"heads": dh, "kv_heads": dg, "dim": dk, "vdim": dv, "conv": 4}, "mlp": dense}, lstm]
+    return {"architecture": "Pelenex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5, "groups": 4}, "logit_softcap": 30.0,
+            "layers": layers}
+
+
+def kotisun_config_like(z: dict) -> dict:
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+            "mask": {"size": z["window"]}}
+    right = {"heads": z["r_heads"], "vdim": z["r_vdim"], "state": z["state"], "groups": z["groups"], "conv": 4, "norm_groups": z["groups"]}
+    layer = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.7},
+             "mlp": {"kind": "dense", "ff": z["ff_gated"]}}
+    return {"architecture": "Kotisun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "logit_softcap": 30.0, "layers": [layer] * 4}
+
+
+def pelenex_kernels(z: dict, hbm_gbs: float, bf16_tflops: float) -> dict:
+    """Pelenex's own kernels alone, each beside the like kernel of a model that was there (20 launches replayed as one graph,
+    inputs rotated over more than L2): the three recurrences beside Kotisun's; the convolution with its unit norms beside
+    Kotisun's convolution; a head's read-out beside Kotisun's gate and norm; the low-rank decays beside a product of the
+    same shape; attention with slopes and kept first keys beside a plain window; the preparation of queries and keys beside
+    Kotisun's; the pair of normed outputs beside Kuvusun's norm added to the residual; the embedding beside a scaled one."""
+    import types
+    import torch
+    from vlrf_b200.csrc import ops
+    from vlrf_b200.parts import get_part
+    from vlrf_b200.parts.context import Workspace
+    dev, bf = "cuda", torch.bfloat16
+    width = z["width"]
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)   # noqa: E731
+
+    def timed(fn, reps=20):
+        for i in range(3):
+            fn(i)
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for i in range(reps):
+                fn(i)
+        graph.replay()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        graph.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / reps * 1e3
+
+    def bytes_point(us, nbytes, flops=0.0):
+        pt = {"us": round(us, 1), "gb_s": round(nbytes / us / 1e3, 1), "frac_hbm": round(nbytes / us / 1e3 / hbm_gbs, 3), "mib": round(nbytes / 2**20, 1)}
+        return dict(pt, tflops=round(flops / us / 1e6, 2)) if flops else pt
+
+    def flops_point(us, fl):
+        return {"us": round(us, 1), "tflops": round(fl / us / 1e6, 1), "frac_tensor": round(fl / us / 1e6 / bf16_tflops, 4)}
+
+    def rotated(make, nbytes):
+        """Enough tensors that together they exceed L2."""
+        return [make() for _ in range(max(2, min(64, int(300e6 // max(nbytes, 1)) + 1)))]
+
+    warm = torch.zeros(4096, 4096, device=dev)
+    t_end = time.time() + 0.2
+    while time.time() < t_end:
+        warm.add_(1.0)
+        torch.cuda.synchronize()
+    del warm
+    out = {}
+    S, L, B = 2, 1024, 64
+    err = torch.zeros(1, dtype=torch.int32, device=dev)
+
+    def step(n_seq, n_new, ctx_len):
+        return types.SimpleNamespace(n_tokens=n_seq * n_new, n_seqs=n_seq, max_new=n_new, max_context=ctx_len, ws=Workspace(dev), dev_err=err,
+                                     seq_slot=i32(list(range(n_seq))), seq_start=i32([i * n_new for i in range(n_seq + 1)]),
+                                     seq_pos0=i32([ctx_len - n_new] * n_seq), tok_slot=i32([s for s in range(n_seq) for _ in range(n_new)]),
+                                     tok_pos=i32([ctx_len - n_new + j for _ in range(n_seq) for j in range(n_new)]))
+    rnd = lambda *sh: torch.randn(*sh, device=dev)   # noqa: E731
+    for label, c in (("prompt", step(S, L, L)), ("decode", step(B, 1, L))):
+        T, n_seq = c.n_tokens, c.n_seqs
+        # -- the recurrences ----------------------------------------------------------------------------------------------------
+        kinds = {"decayed": (z["gla"][0], z["gla"][0], z["gla"][1], z["gla"][2]), "delta": z["delta"],
+                 "stabilized": (z["lstm"][0], z["lstm"][0], z["lstm"][1], z["lstm"][2])}
+        for kind, (H, G, K, V) in kinds.items():
+            numbers = H * (V + 1) * (K + 1) if kind == "stabilized" else H * K * V
+            row = -(-numbers // 4) * 4
+            states = rotated(lambda: torch.zeros(n_seq, 2, row, device=dev), n_seq * row * 8) if label == "decode" else [torch.zeros(n_seq, 2, row, device=dev)]
+            q, k, v = rnd(T, G * K), rnd(T, G * K) * K ** -0.5, rnd(T, H * V)
+            decay, s0, s1 = torch.rand(T, H * K, device=dev) * 0.1 + 0.9, rnd(T, H), rnd(T, H)
+            y, den = torch.zeros(T, H * V, device=dev), torch.zeros(T, 2 * H, device=dev)
+            more = {"decayed": dict(decay=decay), "delta": dict(decay=decay, s0=s0, s1=s1), "stabilized": dict(s0=s0, s1=s1, cap=15.0, den=den)}[kind]
+            us = timed(lambda i: ops.matrix_state_scan(kind, q, k, v, states[i % len(states)], c, y, H, G, K, V, q_scale=0.1, **more), reps=10)
+            nbytes = n_seq * 2 * numbers * 4 + T * (2 * G * K + 2 * H * V + (0 if kind == "stabilized" else H * K)) * 4
+            # multiply-adds of the equations: decay, write and read-out (delta: also the read ahead of the write), two flops each
+            out[f"scan_{kind}_{label}"] = {"pelenex": bytes_point(us, nbytes, 2.0 * T * H * K * V * (3 if kind == "delta" else 2))}
+            del states
+        Hs, P, N, Gs, taps = z["r_heads"], z["r_vdim"], z["state"], z["groups"], 4
+        inner, ch = Hs * P, Hs * P + 2 * Gs * N
+        ld, srow = 2 * inner + 2 * Gs * N + Hs, Hs * N * P + (taps - 1) * ch
+        states = rotated(lambda: torch.zeros(n_seq, 2, srow, device=dev), n_seq * srow * 8)
+        proj, xbc, y = rnd(T, ld) * 0.5, torch.zeros(T, ch, device=dev), torch.zeros(T, inner, device=dev)
+        conv_w, conv_b = rnd(ch, taps) * 0.3, torch.zeros(ch, device=dev)
+        dtb, al, dsk, nw = torch.full((Hs,), -1.0, device=dev), torch.zeros(Hs, device=dev), torch.ones(Hs, device=dev), torch.ones(inner, device=dev)
+        us = timed(lambda i: ops.ssd_scan_step(xbc, proj, inner + ch, dtb, al, dsk, states[i % len(states)], c, y, Hs, Gs, N, P), reps=10)
+        like = bytes_point(us, n_seq * 2 * Hs * N * P * 4 + T * (ch + inner) * 4, 2.0 * T * Hs * N * P * 2)
+        for kind in kinds:
+            out[f"scan_{kind}_{label}"]["kotisun"] = like
+        # -- convolution (+ unit norms), read-out -------------------------------------------------------------------------------
+        projs = rotated(lambda: rnd(T, ld) * 0.5, T * ld * 4)
+        us = timed(lambda i: ops.ssd_conv(projs[i % len(projs)], inner, conv_w, conv_b, states[0], Hs * N * P, c.seq_slot, c.seq_start, c.seq_pos0, xbc, n_seq, c.max_new))
+        out["conv_" + label] = {"kotisun": bytes_point(us, T * ch * 8)}
+        merged = torch.zeros(T, inner, dtype=bf, device=dev)
+        ys = rotated(lambda: rnd(T, inner), T * inner * 4)
+        us = timed(lambda i: ops.ssd_gate_norm(ys[i % len(ys)], projs[i % len(projs)], 0, nw, Gs, 1e-5, 1.0, merged, T))
+        out["read_out_" + label] = {"kotisun": bytes_point(us, T * inner * 10)}
+        del projs, states, ys
+        H, G, K, V = z["delta"]
+        ch = 2 * G * K + H * V
+        projs = rotated(lambda: rnd(T, ch), T * ch * 4)
+        st, cw = torch.zeros(n_seq, 2, 3 * ch, device=dev), rnd(ch, 4) * 0.3
+        qkv, kq = torch.zeros(T, ch, device=dev), torch.zeros(T, G, device=dev)
+        us = timed(lambda i: ops.conv_unit(projs[i % len(projs)], 0, cw, st, 0, c, qkv, kq, H, G, K, V))
+        out["conv_" + label]["pelenex"] = bytes_point(us, T * ch * 8)
+        ys, gs = rotated(lambda: rnd(T, H * V), T * H * V * 4), rotated(lambda: rnd(T, H * V), T * H * V * 4)
+        m, w = torch.zeros(T, H * V, dtype=bf, device=dev), torch.ones(V, device=dev)
+        us = timed(lambda i: ops.head_rows(ys[i % len(ys)], w, gs[i % len(gs)], "sigmoid", m, T, H, V, 1e-5))
+        out["read_out_" + label]["pelenex"] = bytes_point(us, T * H * V * 10)
+        del projs, ys
+        # -- low-rank decays and gates --------------------------------------------------------------------------------------------
+        rank = max(8, width // 16)
+        a1, w2, bias, alog = rnd(T, 2 * rank), (rnd(H * K, rank) * rank ** -0.5).to(bf), rnd(H * K), torch.zeros(H, device=dev)
+        wg = (rnd(H * V, rank) * rank ** -0.5).to(bf)
+        decays = rotated(lambda: torch.zeros(T, H * K, device=dev), T * H * K * 4)
+        us = timed(lambda i: ops.lowrank_rows([(a1[:, :rank], w2, decays[i % len(decays)], "softplus_decay", dict(bias=bias, a_log=alog, per=K)),
+                                               (a1[:, rank:], wg, gs[i % len(gs)], "plain", {})], T))
+        moved = T * (2 * rank + H * K + H * V) * 4 + (H * K + H * V) * rank * 2
+        out["lowrank_" + label] = {"pelenex": bytes_point(us, moved)}
+        a16 = a1[:, :rank].to(bf).contiguous()
+        both = torch.cat([w2, wg]).contiguous()
+        outs = rotated(lambda: torch.zeros(T, H * (K + V), device=dev), T * H * (K + V) * 4)
+        us = timed(lambda i: ops.linear(a16, both, None, outs[i % len(outs)]))
+        out["lowrank_" + label]["product"] = bytes_point(us, T * (rank * 2 + H * (K + V) * 4) + (H * K + H * V) * rank * 2)
+        del decays, gs, outs
+        # -- attention over a paged cache whose blocks are dealt at random ---------------------------------------------------------
+        H, G, dk, window, keep = z["heads"], z["kv_heads"], z["dim"], z["window"], z["keep"]
+        per = L // 64
+        caches = rotated(lambda: (rnd(n_seq * per, G, 64, dk).to(bf), rnd(n_seq * per, G, 64, dk).to(bf)), n_seq * per * G * 64 * dk * 4 if label == "decode" else 2e8)
+        table = torch.randperm(n_seq * per, device=dev).to(torch.int32).view(n_seq, per).contiguous()
+        q, o = rnd(T, H * dk).to(bf), torch.zeros(T, H * dk, dtype=bf, device=dev)
+        slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)], device=dev)
+        run = lambda i, **kw: ops.attention_window_step(q, *caches[i % len(caches)], table, o, c, H, G, dk, dk, dk ** -0.5, window, 1.0, **kw)  # noqa: E731
+        us_new, us_old = timed(lambda i: run(i, keep_first=keep, slopes=slopes)), timed(lambda i: run(i))
+        if label == "decode":
+            out["attention_decode"] = {"pelenex": bytes_point(us_new, n_seq * G * min(L, window + keep) * dk * 4),
+                                       "plain_window": bytes_point(us_old, n_seq * G * min(L, window) * dk * 4)}
+        else:
+            pairs = lambda extra: sum(min(p + 1, window) + min(extra, max(0, p + 1 - window)) for p in range(L))   # noqa: E731
+            out["attention_prompt"] = {"pelenex": flops_point(us_new, 4.0 * n_seq * H * dk * pairs(keep)),
+                                       "plain_window": flops_point(us_old, 4.0 * n_seq * H * dk * pairs(0))}
+        projs = rotated(lambda: rnd(T, (H + G) * dk), T * (H + G) * dk * 4)
+        ones, freq = torch.ones(dk, device=dev), torch.ones(dk // 4, device=dev)
+        moved = T * (H + G) * dk * 4 + T * (H + 2 * G) * dk * 2
+        prep = lambda i, f, rot, **kw: ops.qkv_rope_append(projs[i % len(projs)], 0, H * dk, H * dk, f, rot, o, *caches[0], table, c.tok_slot, c.tok_pos, T, H, G,  # noqa: E731
+                                                           dk, dk, True, err, **kw)
+        us = timed(lambda i: prep(i, None, 0, norm="head", q_norm=ones, k_norm=ones, eps=1e-5))
+        out["prepare_" + label] = {"pelenex": bytes_point(us, moved)}
+        us = timed(lambda i: prep(i, freq, dk // 2))
+        out["prepare_" + label]["rotation"] = bytes_point(us, moved)
+        del caches, projs
+        # -- the pair of normed outputs; the layer's norm; the embedding -------------------------------------------------------------
+        yas, ybs = rotated(lambda: rnd(T, width), T * width * 4), rotated(lambda: rnd(T, width), T * width * 4)
+        x, w, h = rnd(T, width), torch.ones(width, device=dev), torch.zeros(T, width, dtype=bf, device=dev)
+        us = timed(lambda i: ops.norm_pair_add(yas[i % len(yas)], ybs[i % len(ybs)], w, w, x, T, 1e-5, 0.5))
+        out["norm_pair_" + label] = {"pelenex": bytes_point(us, T * width * 16)}
+        us = timed(lambda i: ops.group_rmsnorm(yas[i % len(yas)], w, 1e-5, 1, x, accumulate=True, also=h))
+        out["norm_pair_" + label]["norm_add"] = bytes_point(us, T * width * 14)
+        us = timed(lambda i: ops.group_rmsnorm(yas[i % len(yas)], w, 1e-5, 4, h))
+        out["norm_" + label] = {"pelenex": bytes_point(us, T * width * 6)}
+        us = timed(lambda i: ops.layernorm(yas[i % len(yas)], w, w, 1e-5, h))
+        out["norm_" + label]["layernorm"] = bytes_point(us, T * width * 6)
+        table_e, freqs = rnd(z["vocab"], width).to(bf), get_part("position", "sinusoidal")(width, dev).frequencies
+        toks = [torch.randint(0, z["vocab"], (T,), dtype=torch.int32, device=dev) for _ in range(4)]
+
+        def emb(i):
+            c.tokens = toks[i % 4]
+            ops.embed_sinusoid(table_e, freqs, 1.0, c, x)
+        us = timed(emb)
+        out["embed_" + label] = {"pelenex": bytes_point(us, T * width * 6)}
+        us = timed(lambda i: ops.embed_streams(table_e, toks[i % 4], x, 1, 2.0, err))
+        out["embed_" + label]["scaled"] = bytes_point(us, T * width * 6)
+        # -- the experts' input rows, multiplied by their weights --------------------------------------------------------------------
+        E, top = z["experts"], z["top"]
+        ids, rank_ = torch.randint(0, E, (T, top), dtype=torch.int32, device=dev), torch.zeros(T, top, dtype=torch.int32, device=dev)
+        offs, rows, row_of = torch.arange(E + 1, dtype=torch.int32, device=dev) * 0, torch.zeros(T * top, width, dtype=bf, device=dev), torch.zeros(T, top, dtype=torch.int32, device=dev)
+        rank_.copy_(torch.randperm(T * top, device=dev).view(T, top))
+        hs, wts = rotated(lambda: rnd(T, width).to(bf), T * width * 2), torch.rand(T, top, device=dev)
+        us = timed(lambda i: ops.moe_gather(hs[i % len(hs)], ids, rank_, offs, rows, row_of, T, top, wts=wts))
+        out["gather_" + label] = {"pelenex": bytes_point(us, T * width * 2 * (1 + top))}
+        us = timed(lambda i: ops.moe_gather(hs[i % len(hs)], ids, rank_, offs, rows, row_of, T, top))
+        out["gather_" + label]["unweighted"] = bytes_point(us, T * width * 2 * (1 + top))
+        del yas, ybs, hs
+    return out
+
+
 def design_bench(args) -> int:
     """`--design NAME`: the design at sizes like a real model's layers (random weights) beside its closest existing
-    model of equal size (GPT-2; for Rakelorn, Kuvusun): prefill and decode throughput, and each kernel's time.  One JSON line."""
+    model of equal size (GPT-2; for Rakelorn and Suposun, Kuvusun; for Pelenex, Kotisun): prefill and decode throughput, and each kernel's time.  One JSON line."""
     import vlrf_b200.models  # noqa: F401
     from vlrf_b200.weights import write_random_model
     hbm_gbs, bf16_tflops, peak_src = peaks()
@@ -1041,8 +1263,10 @@ def design_bench(args) -> int:
     sizes, config_of, kernels_of = {"kuvusun": (DESIGN_SIZES, kuvusun_config, design_kernels),
                                     "kotisun": (KOTISUN_SIZES, kotisun_config, kotisun_kernels),
                                     "rakelorn": (RAKELORN_SIZES, rakelorn_config, rakelorn_kernels),
-                                    "suposun": (SUPOSUN_SIZES, suposun_config, suposun_kernels)}[args.design]
-    beside, beside_of = {"rakelorn": ("kuvusun", kuvusun_config_like), "suposun": ("kuvusun", kuvusun_config)}.get(args.design, ("gpt2", gpt2_config_like))
+                                    "suposun": (SUPOSUN_SIZES, suposun_config, suposun_kernels),
+                                    "pelenex": (PELENEX_SIZES, pelenex_config, pelenex_kernels)}[args.design]
+    beside, beside_of = {"rakelorn": ("kuvusun", kuvusun_config_like), "suposun": ("kuvusun", kuvusun_config),
+                         "pelenex": ("kotisun", kotisun_config_like)}.get(args.design, ("gpt2", gpt2_config_like))
     line["beside"] = beside
     for name in args.design_sizes.split(","):
         z = sizes[name]
@@ -1103,7 +1327,7 @@ def main() -> int:
                     help="with --only decode or prefill and VLRF_B200_KERNEL_TRACE=1: print where the last step's kernels spent their time")
     ap.add_argument("--only", default="all", choices=["all", "decode", "prefill"],
                     help="measure one part only and print a short line (for profiling runs); the full line needs 'all'")
-    ap.add_argument("--design", default=None, choices=["kuvusun", "kotisun", "rakelorn", "suposun"],
+    ap.add_argument("--design", default=None, choices=["kuvusun", "kotisun", "rakelorn", "suposun", "pelenex"],
                     help="instead of the default workload: this design at sizes like a real model's layers beside its closest "
                          "existing model of equal size (GPT-2; for rakelorn and suposun, Kuvusun)")
     ap.add_argument("--design-sizes", default="s,m", help="with --design: which of the sizes %s" % ",".join(DESIGN_SIZES))

@@ -179,11 +179,11 @@ def gated_ff(h, w, p):
 def route(h, w, p, ml, margins=None):
     """(chosen experts [T, top], their scores [T, top]): scores sigmoid(W_router h), the largest chosen, not renormalized."""
     top = ml["router"]["top"]
-    s = torch.sigmoid(h @ w[p + "router"].T)
-    order = torch.sort(s, dim=-1, descending=True, stable=True)
-    if margins is not None and s.shape[1] > top:
+    z = h @ w[p + "router"].T
+    order = torch.sort(z, dim=-1, descending=True, stable=True)
+    if margins is not None and z.shape[1] > top:
         margins.append(order.values[:, top - 1] - order.values[:, top])
-    return order.indices[:, :top], order.values[:, :top]
+    return order.indices[:, :top], torch.sigmoid(order.values[:, :top])
 
 
 def routed_ff(h, w, p, ml, margins=None):
@@ -229,8 +229,9 @@ def logits_all_positions(cfg, w, ids):
     return forward(cfg, w, ids)
 
 
-def decided_prefix(cfg, w, ids, least=0.02):
-    """Positions before the first token whose routing (in any layer) is closer to another outcome than `least`."""
+def decided_prefix(cfg, w, ids, least=0.05):
+    """Positions before the first token whose routing (in any layer) has two logits closer together than `least` where the
+    chosen end."""
     margins = []
     forward(cfg, w, ids, margins=margins)
     if not margins:
