@@ -90,6 +90,7 @@ def state_numbers(kind, H, K, V):
 @pytest.mark.parametrize("kind", ["decayed", "delta", "stabilized"])
 def test_recurrence_over_steps(kind, H, G, K, V, columns):
     from vlrf_b200.csrc import call_host
+    warps = {0: 0, 1: 2, 2: 1, 4: 4}[columns]
     if kind != "delta":
         G = H
     seqs = draw_recurrence(kind, H, G, K, V, TOTAL, K * 7 + V)
@@ -108,11 +109,11 @@ def test_recurrence_over_steps(kind, H, G, K, V, columns):
             assert torch.equal(torch.nan_to_num(again), torch.nan_to_num(out))
         return out
 
-    call_host("vlrf_matrix_state_force_columns", columns)
+    call_host("vlrf_matrix_state_force", columns, warps)
     try:
         got = run_steps(fn, [0, 0, 0], 8, None, None)
     finally:
-        call_host("vlrf_matrix_state_force_columns", 0)
+        call_host("vlrf_matrix_state_force", 0, 0)
     for i in range(3):
         close(got[i], want[i], 2e-5, f"{kind}, sequence {i}")
     assert torch.isnan(state[[s for s in range(8) if s not in SLOTS]]).all(), "a state of another slot was written"

@@ -132,7 +132,7 @@ _SIGNATURES = {
         "vlrf_matrix_state_scan": [_c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int,
         _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_float, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
         _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
-        "vlrf_matrix_state_force_columns": [_c_int],
+        "vlrf_matrix_state_force": [_c_int, _c_int],
         "vlrf_conv_unit": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p,
         _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
         "vlrf_lowrank_rows": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_float, _c_int,

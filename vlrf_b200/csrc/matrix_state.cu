@@ -25,6 +25,7 @@
 // the read-outs of eight tokens are summed together, seven exchanges for all eight, and lane r ends up with token r's.
 // Prompts and single tokens run the same arithmetic in the same order.
 #include "common.cuh"
+#include <type_traits>
 
 namespace {
 constexpr int MS_WARPS = 4;
@@ -55,19 +56,137 @@ struct MatrixStateArgs {
     float* y;
     int ldy;
     float* den;
-    int H, G, K, V, col_blocks, batch, vec_rows, vec_v, vec_state;
+    int H, G, K, V, col_blocks, batch, vec_rows, vec_v, vec_state, max_new, warps;
 };
 
 // log sigmoid(x), stable at both ends
 __device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 
+// A lane's part of the state: rows 4·(8j + r) … + 3 for j < NR/4 (as pairs) of NC columns from `my_col` on, from or into a copy
+// of the state.  Rows and columns that do not exist are zero and stay so.
+template <int NR, int NC>
+__device__ __forceinline__ void load_state(f32x2 (&S)[NC][NR / 2], const float* base, int my_col, int VT, int K, int r, int vec) {
+#pragma unroll
+    for (int e = 0; e < NC; ++e) {
+        const bool has = my_col + e < VT;
+        const float* col = base + (size_t)(my_col + e) * K;
+#pragma unroll
+        for (int j = 0; j < NR / 4; ++j) {
+            const int row = 4 * (8 * j + r);
+            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (has) {
+                if (vec) { if (row < K) x = *reinterpret_cast<const float4*>(col + row); }
+                else {
+                    if (row < K) x.x = col[row];
+                    if (row + 1 < K) x.y = col[row + 1];
+                    if (row + 2 < K) x.z = col[row + 2];
+                    if (row + 3 < K) x.w = col[row + 3];
+                }
+            }
+            S[e][2 * j] = pk2(x.x, x.y);
+            S[e][2 * j + 1] = pk2(x.z, x.w);
+        }
+    }
+}
+template <int NR, int NC>
+__device__ __forceinline__ void store_state(const f32x2 (&S)[NC][NR / 2], float* base, int my_col, int VT, int K, int r, int vec) {
+#pragma unroll
+    for (int e = 0; e < NC; ++e) {
+        if (my_col + e >= VT) continue;
+        float* col = base + (size_t)(my_col + e) * K;
+#pragma unroll
+        for (int j = 0; j < NR / 4; ++j) {
+            const int row = 4 * (8 * j + r);
+            float x[4];
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(x[0]), "=f"(x[1]) : "l"(S[e][2 * j]));
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(x[2]), "=f"(x[3]) : "l"(S[e][2 * j + 1]));
+            if (vec) { if (row < K) *reinterpret_cast<float4*>(col + row) = make_float4(x[0], x[1], x[2], x[3]); }
+            else {
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    if (row + q < K) col[row + q] = x[q];
+            }
+        }
+    }
+}
+
+// A token's rows as a lane holds them: k, q and (kinds 0 and 1) the decay at the lane's rows.
+template <int NR> struct TokenRows { ulonglong2 k[NR / 4], q[NR / 4], d[NR / 4]; };
+
+// One token: S moves on, and p gets the lane's share (its rows) of the read-outs.  a, b: kind 1 (b, k · q), kind 2 (what stays, what
+// comes); v: the columns' values.
+template <int MODE, int NR, int NC>
+__device__ __forceinline__ void advance(f32x2 (&S)[NC][NR / 2], const TokenRows<NR>& X, const float (&v)[NC], float a, float b, int r, float (&p)[NC]) {
+    constexpr int NV = NR / 4, NP = NR / 2;
+    f32x2 dq[NC][2];
+#pragma unroll
+    for (int e = 0; e < NC; ++e) dq[e][0] = dq[e][1] = 0ull;
+    if (MODE == MS_DELTA) {
+        f32x2 dk[NC][2];
+#pragma unroll
+        for (int e = 0; e < NC; ++e) dk[e][0] = dk[e][1] = 0ull;
+#pragma unroll
+        for (int j = 0; j < NV; ++j)
+#pragma unroll
+            for (int e = 0; e < NC; ++e) {
+                S[e][2 * j] = mul2(X.d[j].x, S[e][2 * j]);
+                S[e][2 * j + 1] = mul2(X.d[j].y, S[e][2 * j + 1]);
+                dk[e][0] = fma2(X.k[j].x, S[e][2 * j], dk[e][0]);
+                dk[e][1] = fma2(X.k[j].y, S[e][2 * j + 1], dk[e][1]);
+            }
+        float d[NC];
+#pragma unroll
+        for (int e = 0; e < NC; ++e) d[e] = sum2(add2(dk[e][0], dk[e][1]));
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+            for (int e = 0; e < NC; ++e) d[e] += __shfl_xor_sync(0xffffffffu, d[e], o);
+        // Sᵀq of the state before the write, while the exchanges are under way
+#pragma unroll
+        for (int j = 0; j < NV; ++j)
+#pragma unroll
+            for (int e = 0; e < NC; ++e) {
+                dq[e][0] = fma2(X.q[j].x, S[e][2 * j], dq[e][0]);
+                dq[e][1] = fma2(X.q[j].y, S[e][2 * j + 1], dq[e][1]);
+            }
+#pragma unroll
+        for (int e = 0; e < NC; ++e) {
+            const float u = a * (v[e] - d[e]);
+            const f32x2 uu = pk2(u, u);
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                S[e][2 * j] = fma2(X.k[j].x, uu, S[e][2 * j]);
+                S[e][2 * j + 1] = fma2(X.k[j].y, uu, S[e][2 * j + 1]);
+            }
+            p[e] = sum2(add2(dq[e][0], dq[e][1])) + (r == 0 ? u * b : 0.f);
+        }
+    } else {
+        const f32x2 keep = pk2(a, a);
+#pragma unroll
+        for (int e = 0; e < NC; ++e) {
+            const float w = MODE == MS_STABILIZED ? v[e] * b : v[e];
+            const f32x2 ww = pk2(w, w);
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                S[e][2 * j] = fma2(X.k[j].x, ww, mul2(MODE == MS_DECAYED ? X.d[j].x : keep, S[e][2 * j]));
+                S[e][2 * j + 1] = fma2(X.k[j].y, ww, mul2(MODE == MS_DECAYED ? X.d[j].y : keep, S[e][2 * j + 1]));
+                dq[e][0] = fma2(X.q[j].x, S[e][2 * j], dq[e][0]);
+                dq[e][1] = fma2(X.q[j].y, S[e][2 * j + 1], dq[e][1]);
+            }
+            p[e] = sum2(add2(dq[e][0], dq[e][1]));
+        }
+        (void)NP;
+    }
+}
+
 // NR: rows of a column that a lane holds (K ≤ 8·NR; a multiple of 4); NC: columns a lane
 template <int MODE, int NR, int NC>
-__global__ void __launch_bounds__(MS_WARPS * 32)
+__global__ void __launch_bounds__(MS_WARPS * 32, 1)
 matrix_state_scan_kernel(const MatrixStateArgs A) {
-    constexpr int KP = 8 * NR, NP = NR / 2, NV = NR / 4, CW = MS_WARPS * 4 * NC;
+    constexpr int KP = 8 * NR, NV = NR / 4;
     constexpr bool DECAY = MODE != MS_STABILIZED;
     constexpr int ROWS = DECAY ? 3 : 2;             // k, q (, decay)
+    constexpr bool AHEAD = NR <= 16;                // a token's rows are fetched from shared memory while the one before is worked on
     pdl_wait();
     pdl_launch_dependents();
     extern __shared__ __align__(16) float ms_sm[];
@@ -75,7 +194,8 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
     const int slot = A.seq_slot[s];
     if (slot < 0) return;                           // padding (the whole CTA)
     const int start = A.seq_start[s], n = A.seq_start[s + 1] - start, pos0 = A.seq_pos0[s];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane & 7, c = lane >> 3;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane & 7, c = lane >> 3, n_thr = blockDim.x;
+    const int CW = (n_thr >> 5) * 4 * NC;           // columns of the CTA
     const int K = A.K, V = A.V, VT = V + (MODE == MS_STABILIZED ? 1 : 0), B = A.batch;
     const int g = h / (A.H / A.G);
     const int col0 = pb * CW + warp * 4 * NC;       // the warp's first column
@@ -90,7 +210,7 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
 
     // rows K … KP − 1 stay zero in both stages
     if (K < KP) {
-        for (int i = threadIdx.x; i < 2 * B * ROWS * (KP - K); i += MS_WARPS * 32) {
+        for (int i = threadIdx.x; i < 2 * B * ROWS * (KP - K); i += n_thr) {
             const int row = i / (KP - K), cc = K + i - row * (KP - K);       // row: stage-major over [2][ROWS][B]
             const int st = row / (ROWS * B);
             ms_sm[st * stage_floats + (row - st * ROWS * B) * KP + cc] = 0.f;
@@ -105,14 +225,14 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
         const size_t t0 = (size_t)(start + i0);
         if (A.vec_rows) {
             const int q4 = K / 4;
-            for (int i = threadIdx.x; i < nb * q4; i += MS_WARPS * 32) {
+            for (int i = threadIdx.x; i < nb * q4; i += n_thr) {
                 const int ii = i / q4, cc = (i - ii * q4) * 4;
                 ms_cp16(ks + ii * KP + cc, A.k + (t0 + ii) * A.ldk + g * K + cc);
                 ms_cp16(qs + ii * KP + cc, A.q + (t0 + ii) * A.ldq + g * K + cc);
                 if (DECAY) ms_cp16(ds + ii * KP + cc, A.decay + (t0 + ii) * A.ld_decay + h * K + cc);
             }
         } else {
-            for (int i = threadIdx.x; i < nb * K; i += MS_WARPS * 32) {
+            for (int i = threadIdx.x; i < nb * K; i += n_thr) {
                 const int ii = i / K, cc = i - ii * K;
                 ms_cp4(ks + ii * KP + cc, A.k + (t0 + ii) * A.ldk + g * K + cc);
                 ms_cp4(qs + ii * KP + cc, A.q + (t0 + ii) * A.ldq + g * K + cc);
@@ -120,12 +240,12 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
             }
         }
         if (A.vec_v) {                              // (V a multiple of 4: a group of four columns is whole or not there)
-            for (int i = threadIdx.x; i < nb * (CW / 4); i += MS_WARPS * 32) {
+            for (int i = threadIdx.x; i < nb * (CW / 4); i += n_thr) {
                 const int ii = i / (CW / 4), cc = (i - ii * (CW / 4)) * 4;
                 if (pb * CW + cc < V) ms_cp16(vs + ii * CW + cc, A.v + (t0 + ii) * A.ldv + h * V + pb * CW + cc);
             }
         } else {
-            for (int i = threadIdx.x; i < nb * CW; i += MS_WARPS * 32) {
+            for (int i = threadIdx.x; i < nb * CW; i += n_thr) {
                 const int ii = i / CW, cc = i - ii * CW;
                 if (pb * CW + cc < V) ms_cp4(vs + i, A.v + (t0 + ii) * A.ldv + h * V + pb * CW + cc);
             }
@@ -133,30 +253,8 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
     };
     fetch(0, 0);
     asm volatile("cp.async.commit_group;" ::: "memory");
-
-    // the lane's part of the state: rows 4·(8j + r) … + 3 for j < NV, of columns my_col … + NC − 1
-    f32x2 S[NC][NP];
-#pragma unroll
-    for (int e = 0; e < NC; ++e) {
-        const bool has = my_col + e < VT;
-        const float* col = A.state + copy_in + head_at + (size_t)(my_col + e) * K;
-#pragma unroll
-        for (int j = 0; j < NV; ++j) {
-            const int row = 4 * (8 * j + r);
-            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (has) {
-                if (A.vec_state) { if (row < K) x = *reinterpret_cast<const float4*>(col + row); }
-                else {
-                    if (row < K) x.x = col[row];
-                    if (row + 1 < K) x.y = col[row + 1];
-                    if (row + 2 < K) x.z = col[row + 2];
-                    if (row + 3 < K) x.w = col[row + 3];
-                }
-            }
-            S[e][2 * j] = pk2(x.x, x.y);
-            S[e][2 * j + 1] = pk2(x.z, x.w);
-        }
-    }
+    f32x2 S[NC][NR / 2];
+    load_state<NR, NC>(S, A.state + copy_in + head_at, my_col, VT, K, r, A.vec_state);
     // numbers of the batch's tokens: lane ii asks for token ii's, a batch ahead
     float m_run = 0.f, raw0 = 0.f, raw1 = 0.f;
     if (MODE == MS_STABILIZED && active) m_run = A.state[copy_in + max_at + col0];
@@ -193,89 +291,36 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
         __syncwarp();
         if (!active) continue;                      // (whole warps)
         const float* ks = ms_sm + st * stage_floats + 4 * r;
-        const float* qs = ks + B * KP;
-        const float* ds = qs + B * KP;
         const float* vs = ms_sm + st * stage_floats + ROWS * B * KP + warp * 4 * NC + c * NC;
-        for (int e0 = 0; e0 < nb; e0 += 8) {
-            float p[NC][8];                         // this lane's share of the read-outs of eight tokens
+        auto rows_of = [&](int ii, TokenRows<NR>& X) {
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                X.k[j] = *reinterpret_cast<const ulonglong2*>(ks + ii * KP + 32 * j);
+                if (DECAY) X.d[j] = *reinterpret_cast<const ulonglong2*>(ks + (2 * B + ii) * KP + 32 * j);
+                X.q[j] = *reinterpret_cast<const ulonglong2*>(ks + (B + ii) * KP + 32 * j);
+            }
+        };
+        TokenRows<NR> X[AHEAD ? 2 : 1];
+        if (AHEAD) rows_of(0, X[0]);
+        // eight tokens from e0 on; FULL: all eight are there (nothing then stands between one token's loads and the next's)
+        auto eight = [&](int e0, auto full) {
+            constexpr bool FULL = decltype(full)::value;
+            float p[8][NC];                         // this lane's share of the read-outs of eight tokens
 #pragma unroll
             for (int t = 0; t < 8; ++t) {
                 const int ii = e0 + t;
-                if (ii < nb) {                      // (uniform over the CTA)
-                    const float* kt = ks + ii * KP;
-                    const float* qt = qs + ii * KP;
-                    const float* dt = ds + ii * KP;
+                if (FULL || ii < nb) {              // (uniform over the CTA)
+                    if (AHEAD) rows_of((FULL && t < 7) || ii + 1 < nb ? ii + 1 : ii, X[(t + 1) & 1]);
+                    else rows_of(ii, X[0]);
                     float v[NC];
 #pragma unroll
                     for (int e = 0; e < NC; ++e) v[e] = my_col + e < V ? vs[ii * CW + e] : (MODE == MS_STABILIZED && my_col + e == V) ? 1.f : 0.f;
-                    if (MODE == MS_DELTA) {
-                        const float2 bk = *reinterpret_cast<const float2*>(scal + 2 * ii);      // (b, k · q)
-                        f32x2 dk[NC][2], dq[NC][2], kr[NP];
-#pragma unroll
-                        for (int e = 0; e < NC; ++e) { dk[e][0] = dk[e][1] = dq[e][0] = dq[e][1] = 0ull; }
-#pragma unroll
-                        for (int j = 0; j < NV; ++j) {
-                            const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(kt + 32 * j);
-                            const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(qt + 32 * j);
-                            const ulonglong2 d4 = *reinterpret_cast<const ulonglong2*>(dt + 32 * j);
-                            kr[2 * j] = k4.x; kr[2 * j + 1] = k4.y;
-#pragma unroll
-                            for (int e = 0; e < NC; ++e) {
-                                S[e][2 * j] = mul2(d4.x, S[e][2 * j]);
-                                S[e][2 * j + 1] = mul2(d4.y, S[e][2 * j + 1]);
-                                dk[e][0] = fma2(k4.x, S[e][2 * j], dk[e][0]);
-                                dk[e][1] = fma2(k4.y, S[e][2 * j + 1], dk[e][1]);
-                                dq[e][0] = fma2(q4.x, S[e][2 * j], dq[e][0]);
-                                dq[e][1] = fma2(q4.y, S[e][2 * j + 1], dq[e][1]);
-                            }
-                        }
-                        float d[NC];
-#pragma unroll
-                        for (int e = 0; e < NC; ++e) d[e] = sum2(add2(dk[e][0], dk[e][1]));
-#pragma unroll
-                        for (int o = 4; o > 0; o >>= 1)
-#pragma unroll
-                            for (int e = 0; e < NC; ++e) d[e] += __shfl_xor_sync(0xffffffffu, d[e], o);
-#pragma unroll
-                        for (int e = 0; e < NC; ++e) {
-                            const float u = bk.x * (v[e] - d[e]);
-                            const f32x2 uu = pk2(u, u);
-#pragma unroll
-                            for (int j = 0; j < NP; ++j) S[e][j] = fma2(kr[j], uu, S[e][j]);
-                            p[e][t] = sum2(add2(dq[e][0], dq[e][1])) + (r == 0 ? u * bk.y : 0.f);
-                        }
-                    } else {
-                        f32x2 acc[NC][2], keep = 0ull;
-                        if (MODE == MS_STABILIZED) {
-                            const float2 ab = *reinterpret_cast<const float2*>(scal + 2 * ii);  // (what stays, what comes)
-                            keep = pk2(ab.x, ab.x);
-#pragma unroll
-                            for (int e = 0; e < NC; ++e) v[e] *= ab.y;
-                        }
-                        f32x2 vv[NC];
-#pragma unroll
-                        for (int e = 0; e < NC; ++e) { vv[e] = pk2(v[e], v[e]); acc[e][0] = acc[e][1] = 0ull; }
-#pragma unroll
-                        for (int j = 0; j < NV; ++j) {
-                            const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(kt + 32 * j);
-                            const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(qt + 32 * j);
-                            ulonglong2 d4;
-                            if (DECAY) d4 = *reinterpret_cast<const ulonglong2*>(dt + 32 * j);
-                            else { d4.x = keep; d4.y = keep; }
-#pragma unroll
-                            for (int e = 0; e < NC; ++e) {
-                                S[e][2 * j] = fma2(k4.x, vv[e], mul2(d4.x, S[e][2 * j]));
-                                S[e][2 * j + 1] = fma2(k4.y, vv[e], mul2(d4.y, S[e][2 * j + 1]));
-                                acc[e][0] = fma2(q4.x, S[e][2 * j], acc[e][0]);
-                                acc[e][1] = fma2(q4.y, S[e][2 * j + 1], acc[e][1]);
-                            }
-                        }
-#pragma unroll
-                        for (int e = 0; e < NC; ++e) p[e][t] = sum2(add2(acc[e][0], acc[e][1]));
-                    }
+                    float2 ab = make_float2(0.f, 0.f);
+                    if (MODE != MS_DECAYED) ab = *reinterpret_cast<const float2*>(scal + 2 * ii);
+                    advance<MODE, NR, NC>(S, X[AHEAD ? (t & 1) : 0], v, ab.x, ab.y, r, p[t]);
                 } else {
 #pragma unroll
-                    for (int e = 0; e < NC; ++e) p[e][t] = 0.f;
+                    for (int e = 0; e < NC; ++e) p[t][e] = 0.f;
                 }
             }
             // eight sums over eight lanes: each exchange halves the tokens a lane is responsible for
@@ -287,15 +332,15 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
                     const bool up = r & w;
 #pragma unroll
                     for (int t = 0; t < w; ++t) {
-                        const float give = up ? p[e][t] : p[e][t + w], mine = up ? p[e][t + w] : p[e][t];
-                        p[e][t] = mine + __shfl_xor_sync(0xffffffffu, give, w);
+                        const float give = up ? p[t][e] : p[t + w][e], mine = up ? p[t + w][e] : p[t][e];
+                        p[t][e] = mine + __shfl_xor_sync(0xffffffffu, give, w);
                     }
                 }
-                o[e] = p[e][0] * A.q_scale;
+                o[e] = p[0][e] * A.q_scale;
             }
             const int ii = e0 + r;
             const float em = MODE == MS_STABILIZED ? __shfl_sync(0xffffffffu, floor_mine, ii & 31) : 0.f;
-            if (ii < nb) {
+            if (FULL || ii < nb) {
                 const size_t row = (size_t)(start + i0 + ii);
 #pragma unroll
                 for (int e = 0; e < NC; ++e) {
@@ -306,37 +351,109 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
                     }
                 }
             }
+        };
+        for (int e0 = 0; e0 < nb; e0 += 8) {
+            if (nb - e0 >= 8) eight(e0, std::true_type{});
+            else eight(e0, std::false_type{});
         }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     if (!active) return;
+    store_state<NR, NC>(S, A.state + copy_out + head_at, my_col, VT, K, r, A.vec_state);
+    if (MODE == MS_STABILIZED && r == 0) {
 #pragma unroll
-    for (int e = 0; e < NC; ++e) {
-        if (my_col + e >= VT) continue;
-        float* col = A.state + copy_out + head_at + (size_t)(my_col + e) * K;
+        for (int e = 0; e < NC; ++e)
+            if (my_col + e < VT) A.state[copy_out + max_at + my_col + e] = m_run;
+    }
+}
+
+// A step of single tokens: a warp takes 4·NC columns of a head of a sequence, straight from and into device memory (no other
+// warp shares enough of a token's rows to be worth a stage in shared memory).  The same arithmetic in the same order.
+template <int MODE, int NR, int NC>
+__global__ void __launch_bounds__(MS_WARPS * 32)
+matrix_state_step_kernel(const MatrixStateArgs A) {
+    constexpr int NV = NR / 4;
+    constexpr bool DECAY = MODE != MS_STABILIZED;
+    pdl_wait();
+    pdl_launch_dependents();
+    const int s = blockIdx.y, slot = A.seq_slot[s];
+    if (slot < 0) return;                           // padding
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane & 7, c = lane >> 3;
+    const int unit = blockIdx.x * MS_WARPS + warp;
+    const int h = unit / A.col_blocks;
+    if (h >= A.H) return;                           // (whole warps; no block-wide barrier below)
+    const int K = A.K, V = A.V, VT = V + (MODE == MS_STABILIZED ? 1 : 0), g = h / (A.H / A.G);
+    const int col0 = (unit - h * A.col_blocks) * 4 * NC, my_col = col0 + c * NC;
+    const int pos0 = A.seq_pos0[s];
+    const size_t t = (size_t)A.seq_start[s];
+    const size_t copy_in = ((size_t)slot * 2 + (pos0 & 1)) * A.state_row, copy_out = ((size_t)slot * 2 + ((pos0 + 1) & 1)) * A.state_row;
+    const size_t head_at = (size_t)h * VT * K, max_at = (size_t)A.H * VT * K + (size_t)h * VT;
+    f32x2 S[NC][NR / 2];
+    load_state<NR, NC>(S, A.state + copy_in + head_at, my_col, VT, K, r, A.vec_state);
+    TokenRows<NR> X;
+    auto row_of = [&](const float* base, ulonglong2 (&out)[NV]) {
 #pragma unroll
         for (int j = 0; j < NV; ++j) {
             const int row = 4 * (8 * j + r);
-            float x[4];
-            asm("mov.b64 {%0, %1}, %2;" : "=f"(x[0]), "=f"(x[1]) : "l"(S[e][2 * j]));
-            asm("mov.b64 {%0, %1}, %2;" : "=f"(x[2]), "=f"(x[3]) : "l"(S[e][2 * j + 1]));
-            if (A.vec_state) { if (row < K) *reinterpret_cast<float4*>(col + row) = make_float4(x[0], x[1], x[2], x[3]); }
+            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (A.vec_rows) { if (row < K) x = *reinterpret_cast<const float4*>(base + row); }
             else {
-#pragma unroll
-                for (int q = 0; q < 4; ++q)
-                    if (row + q < K) col[row + q] = x[q];
+                if (row < K) x.x = base[row];
+                if (row + 1 < K) x.y = base[row + 1];
+                if (row + 2 < K) x.z = base[row + 2];
+                if (row + 3 < K) x.w = base[row + 3];
             }
+            out[j].x = pk2(x.x, x.y);
+            out[j].y = pk2(x.z, x.w);
         }
-        if (MODE == MS_STABILIZED && r == 0) A.state[copy_out + max_at + my_col + e] = m_run;
+    };
+    row_of(A.k + t * A.ldk + (size_t)g * K, X.k);
+    row_of(A.q + t * A.ldq + (size_t)g * K, X.q);
+    if (DECAY) row_of(A.decay + t * A.ld_decay + (size_t)h * K, X.d);
+    float v[NC], p[NC];
+#pragma unroll
+    for (int e = 0; e < NC; ++e)
+        v[e] = my_col + e < V ? A.v[t * A.ldv + (size_t)h * V + my_col + e] : (MODE == MS_STABILIZED && my_col + e == V) ? 1.f : 0.f;
+    float a = 0.f, b = 0.f, m_new = 0.f;
+    if (MODE == MS_DELTA) {
+        a = sigmoid_f(A.s0[t * A.ld_s0 + h]);
+        b = A.s1[t * A.ld_s1 + g];
+    } else if (MODE == MS_STABILIZED) {
+        const float m_run = A.state[copy_in + max_at + col0];
+        const float log_i = A.cap * tanhf(A.s0[t * A.ld_s0 + h] / A.cap), log_f = log_sigmoid(A.cap * tanhf(A.s1[t * A.ld_s1 + h] / A.cap));
+        m_new = fmaxf(log_f + m_run, log_i);
+        a = expf(log_f + m_run - m_new);
+        b = expf(log_i - m_new);
+    }
+    advance<MODE, NR, NC>(S, X, v, a, b, r, p);
+    store_state<NR, NC>(S, A.state + copy_out + head_at, my_col, VT, K, r, A.vec_state);
+#pragma unroll
+    for (int e = 0; e < NC; ++e) {
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) p[e] += __shfl_xor_sync(0xffffffffu, p[e], o);
+        if (r != 0) continue;
+        if (my_col + e < V) A.y[t * A.ldy + (size_t)h * V + my_col + e] = p[e] * A.q_scale;
+        else if (MODE == MS_STABILIZED && my_col + e == V) {
+            A.den[(t * A.H + h) * 2] = p[e] * A.q_scale;
+            A.den[(t * A.H + h) * 2 + 1] = expf(-m_new);
+        }
+        if (MODE == MS_STABILIZED && my_col + e < VT) A.state[copy_out + max_at + my_col + e] = m_new;
     }
 }
 
 template <int MODE, int NR, int NC> int launch_scan(MatrixStateArgs& A, int n_seqs, cudaStream_t stream) {
-    constexpr int KP = 8 * NR, CW = MS_WARPS * 4 * NC, ROWS = MODE == MS_STABILIZED ? 2 : 3;
-    const int VT = A.V + (MODE == MS_STABILIZED ? 1 : 0);
-    A.col_blocks = (VT + CW - 1) / CW;
+    constexpr int KP = 8 * NR, ROWS = MODE == MS_STABILIZED ? 2 : 3;
+    const int VT = A.V + (MODE == MS_STABILIZED ? 1 : 0), chunks = (VT + 4 * NC - 1) / (4 * NC);
+    if (A.max_new == 1) {
+        A.col_blocks = chunks;
+        launch_chained(matrix_state_step_kernel<MODE, NR, NC>, dim3((A.H * chunks + MS_WARPS - 1) / MS_WARPS, n_seqs), dim3(MS_WARPS * 32), (size_t)0,
+                       stream, A);
+        return vlrf_check_launch("matrix_state_step");
+    }
+    const int warps = A.warps, CW = warps * 4 * NC;
+    A.col_blocks = (chunks + warps - 1) / warps;
     // tokens a batch: as many as the step's longest run has, at most 16, fewer where the rows are long
-    const auto bytes = [&](int b) { return (size_t)(2 * b * (ROWS * KP + CW) + MS_WARPS * b * 2) * sizeof(float); };
+    const auto bytes = [&](int b) { return (size_t)(2 * b * (ROWS * KP + CW) + warps * b * 2) * sizeof(float); };
     while (A.batch > 1 && bytes(A.batch) > 110 * 1024) A.batch /= 2;
     const size_t smem = bytes(A.batch);
     static size_t allowed = 48 * 1024;
@@ -345,7 +462,7 @@ template <int MODE, int NR, int NC> int launch_scan(MatrixStateArgs& A, int n_se
         if (e != cudaSuccess) return vlrf_fail(VLRF_ERR_CUDA, "matrix_state_scan: %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
         allowed = smem;
     }
-    launch_chained(matrix_state_scan_kernel<MODE, NR, NC>, dim3(A.H * A.col_blocks, n_seqs), dim3(MS_WARPS * 32), smem, stream, A);
+    launch_chained(matrix_state_scan_kernel<MODE, NR, NC>, dim3(A.H * A.col_blocks, n_seqs), dim3(warps * 32), smem, stream, A);
     return vlrf_check_launch("matrix_state_scan");
 }
 
@@ -360,13 +477,15 @@ template <int MODE> int pick_scan(MatrixStateArgs& A, int nc, int n_seqs, cudaSt
 }
 
 bool on16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
-int ms_forced_columns = 0;
+int ms_forced_columns = 0, ms_forced_warps = 0;
 }  // namespace
 
-// For measurements: a lane's columns (1, 2 or 4; 0: chosen by the step's size).
-extern "C" int vlrf_matrix_state_force_columns(int nc) {
-    VLRF_REQUIRE(nc == 0 || nc == 1 || nc == 2 || nc == 4, "matrix_state_scan: a lane takes 1, 2 or 4 columns, not %d", nc);
-    ms_forced_columns = nc;
+// For measurements and tests: a lane's columns (1, 2 or 4) and a CTA's warps (1, 2 or 4); 0: chosen by the step's size.
+extern "C" int vlrf_matrix_state_force(int columns, int warps) {
+    VLRF_REQUIRE(columns == 0 || columns == 1 || columns == 2 || columns == 4, "matrix_state_scan: a lane takes 1, 2 or 4 columns, not %d", columns);
+    VLRF_REQUIRE(warps == 0 || warps == 1 || warps == 2 || warps == 4, "matrix_state_scan: a CTA has 1, 2 or 4 warps, not %d", warps);
+    ms_forced_columns = columns;
+    ms_forced_warps = warps;
     return VLRF_OK;
 }
 
@@ -391,16 +510,18 @@ extern "C" int vlrf_matrix_state_scan(int kind, const float* q, int ldq, const f
     A.q_scale = q_scale; A.cap = cap; A.state = state; A.state_row = state_row;
     A.seq_slot = seq_slot; A.seq_start = seq_start; A.seq_pos0 = seq_pos0;
     A.y = y; A.ldy = ldy; A.den = den; A.H = H; A.G = G; A.K = K; A.V = V; A.col_blocks = 1;
+    A.max_new = max_new; A.warps = ms_forced_warps ? ms_forced_warps : 4;
     A.batch = max_new < MS_MAX_BATCH ? max_new : MS_MAX_BATCH;
     A.vec_rows = K % 4 == 0 && on16(q) && on16(k) && ldq % 4 == 0 && ldk % 4 == 0 && (decay == nullptr || (on16(decay) && ld_decay % 4 == 0));
     A.vec_v = V % 4 == 0 && on16(v) && ldv % 4 == 0;
     A.vec_state = K % 4 == 0 && on16(state) && state_row % 4 == 0;
-    // columns a lane: few where the step has few columns in all (every SM gets warps), more where it has plenty
+    // columns a lane (measured): single tokens 2; prompts 1 where the step's columns are fewer than warps for every scheduler of
+    // the GPU, else 2; 4 for the decayed kind with columns in plenty (it has the most rows to read from shared memory)
     int sms = 148, dev = 0;
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     const long long warps1 = (long long)n_seqs * H * ((V + 3) / 4);
-    int nc = ms_forced_columns ? ms_forced_columns : warps1 > 16LL * sms ? 4 : warps1 > 8LL * sms ? 2 : 1;
+    int nc = ms_forced_columns ? ms_forced_columns : max_new == 1 ? 2 : warps1 <= 4LL * sms ? 1 : (kind == MS_DECAYED && warps1 > 8LL * sms) ? 4 : 2;
     if (K > 128 && nc > 2) nc = 2;
     switch (kind) {
         case MS_DECAYED: return pick_scan<MS_DECAYED>(A, nc, n_seqs, stream);

@@ -194,36 +194,69 @@ __device__ __forceinline__ float lr_apply(const LowRankPart& P, float z, int col
     return z;
 }
 
-// a tile of 64 tokens by 64 columns; bfloat16 weights on mma.sync with the float32 rows as the sum of two bfloat16 rows
+// a tile of 64 tokens by CT columns; bfloat16 weights on mma.sync with the float32 rows as the sum of two bfloat16 rows.  VEC: ranks
+// of a multiple of 8 and rows on 16-byte boundaries, eight weights and four row entries a load
+constexpr int LR_K = 64;                            // of the rank at a time
+template <int CT, bool VEC>
 __global__ void __launch_bounds__(128)
 lowrank_mma_kernel(const LowRankPart P0, const LowRankPart P1, int T) {
     pdl_wait();
     pdl_launch_dependents();
     const bool second = (int)blockIdx.x >= P0.tiles;
     const LowRankPart& P = second ? P1 : P0;
-    const int c0 = (blockIdx.x - (second ? P0.tiles : 0)) * 64, t0 = blockIdx.y * 64;
-    constexpr int LD = 40;                          // 32 of the rank at a time, rows padded against bank conflicts
-    __shared__ __align__(16) __nv_bfloat16 hi[64 * LD], lo[64 * LD], ws[64 * LD];
+    const int c0 = (blockIdx.x - (second ? P0.tiles : 0)) * CT, t0 = blockIdx.y * 64;
+    constexpr int LD = LR_K + 8;                    // rows padded against bank conflicts
+    __shared__ __align__(16) __nv_bfloat16 hi[64 * LD], lo[64 * LD], ws[CT * LD];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-    float acc[8][4];
+    const int rank = P.rank, lda = P.lda, cols = P.cols;
+    float acc[CT / 8][4];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    for (int j = 0; j < CT / 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
     const __nv_bfloat16* W = (const __nv_bfloat16*)P.w;
-    for (int r0 = 0; r0 < P.rank; r0 += 32) {
+    for (int r0 = 0; r0 < rank; r0 += LR_K) {
         if (r0 > 0) __syncthreads();
-        for (int i = threadIdx.x; i < 64 * 32; i += 128) {
-            const int row = i >> 5, rr = i & 31;
-            const bool in = r0 + rr < P.rank;
-            const float x = (in && t0 + row < T) ? P.a[(size_t)(t0 + row) * P.lda + r0 + rr] : 0.f;
-            const __nv_bfloat16 h = __float2bfloat16_rn(x);
-            hi[row * LD + rr] = h;
-            lo[row * LD + rr] = __float2bfloat16_rn(x - __bfloat162float(h));
-            ws[row * LD + rr] = (in && c0 + row < P.cols) ? W[(size_t)(c0 + row) * P.rank + r0 + rr] : __float2bfloat16_rn(0.f);
+        const int kn = min(LR_K, (rank - r0 + 15) & ~15);       // entries that the products of this pass read
+        if (VEC) {
+            float4 x[64 * LR_K / 4 / 128];
+            uint4 y[CT * LR_K / 8 / 128];
+#pragma unroll
+            for (int q = 0; q < CT * LR_K / 8 / 128; ++q) {
+                const int i = threadIdx.x + q * 128, row = i / (LR_K / 8), rr = (i % (LR_K / 8)) * 8;
+                y[q] = (r0 + rr < rank && c0 + row < cols) ? *reinterpret_cast<const uint4*>(W + (size_t)(c0 + row) * rank + r0 + rr) : make_uint4(0, 0, 0, 0);
+            }
+#pragma unroll
+            for (int q = 0; q < 64 * LR_K / 4 / 128; ++q) {
+                const int i = threadIdx.x + q * 128, row = i / (LR_K / 4), rr = (i % (LR_K / 4)) * 4;
+                x[q] = (r0 + rr < rank && t0 + row < T) ? *reinterpret_cast<const float4*>(P.a + (size_t)(t0 + row) * lda + r0 + rr) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int q = 0; q < CT * LR_K / 8 / 128; ++q) {
+                const int i = threadIdx.x + q * 128, row = i / (LR_K / 8), rr = (i % (LR_K / 8)) * 8;
+                *reinterpret_cast<uint4*>(ws + row * LD + rr) = y[q];
+            }
+#pragma unroll
+            for (int q = 0; q < 64 * LR_K / 4 / 128; ++q) {
+                const int i = threadIdx.x + q * 128, row = i / (LR_K / 4), rr = (i % (LR_K / 4)) * 4;
+                const __nv_bfloat162 h0 = __floats2bfloat162_rn(x[q].x, x[q].y), h1 = __floats2bfloat162_rn(x[q].z, x[q].w);
+                const __nv_bfloat162 l0 = __floats2bfloat162_rn(x[q].x - __low2float(h0), x[q].y - __high2float(h0));
+                const __nv_bfloat162 l1 = __floats2bfloat162_rn(x[q].z - __low2float(h1), x[q].w - __high2float(h1));
+                *reinterpret_cast<uint2*>(hi + row * LD + rr) = make_uint2(*reinterpret_cast<const uint32_t*>(&h0), *reinterpret_cast<const uint32_t*>(&h1));
+                *reinterpret_cast<uint2*>(lo + row * LD + rr) = make_uint2(*reinterpret_cast<const uint32_t*>(&l0), *reinterpret_cast<const uint32_t*>(&l1));
+            }
+        } else {
+            for (int i = threadIdx.x; i < 64 * kn; i += 128) {
+                const int row = i / kn, rr = i - row * kn;
+                const float x = (r0 + rr < rank && t0 + row < T) ? P.a[(size_t)(t0 + row) * lda + r0 + rr] : 0.f;
+                const __nv_bfloat16 h = __float2bfloat16_rn(x);
+                hi[row * LD + rr] = h;
+                lo[row * LD + rr] = __float2bfloat16_rn(x - __bfloat162float(h));
+                if (row < CT) ws[row * LD + rr] = (r0 + rr < rank && c0 + row < cols) ? W[(size_t)(c0 + row) * rank + r0 + rr] : __float2bfloat16_rn(0.f);
+            }
         }
         __syncthreads();
 #pragma unroll
-        for (int ks = 0; ks < 2; ++ks) {
-            if (r0 + 16 * ks >= P.rank) break;
+        for (int ks = 0; ks < LR_K / 16; ++ks) {
+            if (16 * ks >= kn) break;
             uint32_t ah[4], al[4];
             const int rb = warp * 16 + g, kb = ks * 16 + 2 * t;
 #pragma unroll
@@ -233,7 +266,7 @@ lowrank_mma_kernel(const LowRankPart P0, const LowRankPart P1, int T) {
                 al[q] = *reinterpret_cast<const uint32_t*>(lo + at);
             }
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
+            for (int j = 0; j < CT / 8; ++j) {
                 const uint32_t b0 = *reinterpret_cast<const uint32_t*>(ws + (j * 8 + g) * LD + kb);
                 const uint32_t b1 = *reinterpret_cast<const uint32_t*>(ws + (j * 8 + g) * LD + kb + 8);
 #define LR_MMA(A) asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n" \
@@ -245,16 +278,21 @@ lowrank_mma_kernel(const LowRankPart P0, const LowRankPart P1, int T) {
             }
         }
     }
+    const bool pairs = (P.ldo & 1) == 0 && (cols & 1) == 0 && (reinterpret_cast<uintptr_t>(P.out) & 7) == 0;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
         const int row = t0 + warp * 16 + g + half * 8;
         if (row >= T) continue;
         float* o = P.out + (size_t)row * P.ldo;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
+        for (int j = 0; j < CT / 8; ++j) {
             const int col = c0 + j * 8 + 2 * t;
-            if (col < P.cols) o[col] = lr_apply(P, acc[j][2 * half], col);
-            if (col + 1 < P.cols) o[col + 1] = lr_apply(P, acc[j][2 * half + 1], col + 1);
+            if (pairs) {
+                if (col < cols) *reinterpret_cast<float2*>(o + col) = make_float2(lr_apply(P, acc[j][2 * half], col), lr_apply(P, acc[j][2 * half + 1], col + 1));
+            } else {
+                if (col < cols) o[col] = lr_apply(P, acc[j][2 * half], col);
+                if (col + 1 < cols) o[col + 1] = lr_apply(P, acc[j][2 * half + 1], col + 1);
+            }
         }
     }
 }
@@ -451,7 +489,19 @@ extern "C" int vlrf_lowrank_rows(const float* a0, int lda0, int rank0, const voi
     VLRF_REQUIRE(T >= 0 && T <= 64 * 65535, "lowrank_rows: too many rows");
     if (T == 0) return VLRF_OK;
     const dim3 grid(P0.tiles + P1.tiles, (T + 63) / 64);
-    if (w_dtype == VLRF_BF16) launch_chained(lowrank_mma_kernel, grid, dim3(128), (size_t)0, stream, P0, P1, T);
+    if (w_dtype == VLRF_BF16) {
+        // few rows: narrower tiles, so that more of the GPU takes part
+        const int ct = T <= 64 ? 32 : 64;
+        P0.tiles = (P0.cols + ct - 1) / ct;
+        P1.tiles = a1 != nullptr ? (P1.cols + ct - 1) / ct : 0;
+        const dim3 g(P0.tiles + P1.tiles, (T + 63) / 64);
+        const auto fits = [](const LowRankPart& P) { return P.rank % 8 == 0 && P.lda % 4 == 0 && rows16(P.a) && rows16(P.w); };
+        const bool vec = fits(P0) && fits(P1);
+        if (ct == 32) { if (vec) launch_chained(lowrank_mma_kernel<32, true>, g, dim3(128), (size_t)0, stream, P0, P1, T);
+                        else launch_chained(lowrank_mma_kernel<32, false>, g, dim3(128), (size_t)0, stream, P0, P1, T); }
+        else { if (vec) launch_chained(lowrank_mma_kernel<64, true>, g, dim3(128), (size_t)0, stream, P0, P1, T);
+               else launch_chained(lowrank_mma_kernel<64, false>, g, dim3(128), (size_t)0, stream, P0, P1, T); }
+    }
     else if (w_dtype == VLRF_F32) launch_chained(lowrank_fma_kernel, grid, dim3(128), (size_t)0, stream, P0, P1, T);
     else return vlrf_fail(VLRF_ERR_INVALID_ARG, "lowrank_rows: unknown weight dtype %d", w_dtype);
     return vlrf_check_launch("lowrank_rows");

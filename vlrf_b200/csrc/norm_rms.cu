@@ -272,6 +272,50 @@ rmsnorm_shift_kernel(const float* __restrict__ x, int ld_x, const float* __restr
     }
 }
 
+// group_rmsnorm for rows on 16-byte boundaries whose groups are whole runs of 128 columns: a thread holds NV quads of its row in
+// registers, a warp sums the run of 128 columns that it holds of each, and a group's sum is that of its runs, in order.
+template <typename OT, bool ACC, int NV>
+__global__ void __launch_bounds__(256)
+group_rmsnorm_quads_kernel(const float* y, int ld_y, const int* __restrict__ rows, const float* __restrict__ w, OT* out, int ld_out, int d,
+                           int groups, float eps, __nv_bfloat16* also) {
+    pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
+    pdl_launch_dependents();
+    __shared__ float run_sm[NV * 8];
+    const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float* yr = y + (size_t)(rows ? rows[r] : r) * ld_y;
+    float4 v[NV];
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = 4 * (threadIdx.x + 256 * k);
+        v[k] = i < d ? *reinterpret_cast<const float4*>(yr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const float s = warp_sum(fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, v[k].w * v[k].w))));
+        if (lane == 0) run_sm[8 * k + warp] = s;
+    }
+    __syncthreads();
+    const int gs = d / groups, per = gs / 128;      // runs of a group
+    OT* o = out + (size_t)r * ld_out;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = 4 * (threadIdx.x + 256 * k);
+        if (i >= d) break;
+        const int first = (8 * k + warp) / per * per;
+        float s = 0.f;
+        for (int q = 0; q < per; ++q) s += run_sm[first + q];
+        const float inv = 1.f / sqrtf(s / (float)gs + eps);
+        const float4 g = *reinterpret_cast<const float4*>(w + i);
+        float4 x = make_float4(v[k].x * inv * g.x, v[k].y * inv * g.y, v[k].z * inv * g.z, v[k].w * inv * g.w);
+        if (ACC) {
+            const float4 old = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(o) + i);
+            x.x += old.x; x.y += old.y; x.z += old.z; x.w += old.w;
+        }
+        store4<OT>(o + i, x.x, x.y, x.z, x.w);
+        if (also != nullptr) store4<__nv_bfloat16>(also + (size_t)r * d + i, x.x, x.y, x.z, x.w);   // what the next sublayer reads of the row
+    }
+}
+
 // rmsnorm_shift with a CTA per token, for rows on 16-byte boundaries: a thread holds NV groups of four columns of its
 // row and of the row before in registers (both asked for at once), the two sums of squares are reduced together, and
 // nothing is read twice.  The CTA of a sequence's first token of the step also norms and keeps the sequence's last row.
@@ -418,6 +462,18 @@ extern "C" int vlrf_group_rmsnorm(const float* y, int ld_y, const int* rows, con
     VLRF_REQUIRE(ld_y >= d && ld_out >= d, "group_rmsnorm: leading sizes are smaller than the row");
     VLRF_REQUIRE(!accumulate || out_dtype == VLRF_F32, "group_rmsnorm: only float32 rows can be added to");
     if (n_rows == 0) return VLRF_OK;
+    const auto on = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
+    if ((d / groups) % 128 == 0 && d <= 8192 && (out_dtype == VLRF_F32 || out_dtype == VLRF_BF16) && ld_y % 4 == 0 && ld_out % 4 == 0 && on(y, 16) &&
+        on(w, 16) && on(out, out_dtype == VLRF_BF16 ? 8 : 16) && on(also_bf16, 8)) {
+#define QUADS(OT, ACC, NV) launch_chained(group_rmsnorm_quads_kernel<OT, ACC, NV>, dim3(n_rows), dim3(256), (size_t)(0), stream, y, ld_y, rows, w, (OT*)out, ld_out, d, groups, eps, (__nv_bfloat16*)also_bf16)
+#define QUADS_NV(OT, ACC) do { if (d <= 1024) QUADS(OT, ACC, 1); else if (d <= 2048) QUADS(OT, ACC, 2); else if (d <= 4096) QUADS(OT, ACC, 4); else QUADS(OT, ACC, 8); } while (0)
+        if (out_dtype == VLRF_BF16) QUADS_NV(__nv_bfloat16, false);
+        else if (accumulate) QUADS_NV(float, true);
+        else QUADS_NV(float, false);
+#undef QUADS_NV
+#undef QUADS
+        return vlrf_check_launch("group_rmsnorm");
+    }
     if (out_dtype == VLRF_F32) {
         if (accumulate) launch_chained(group_rmsnorm_kernel<float, true>, dim3(n_rows), dim3(NORM_THREADS), (size_t)(0), stream, y, ld_y, rows, w, (float*)out, ld_out, d, groups, eps, (__nv_bfloat16*)also_bf16);
         else launch_chained(group_rmsnorm_kernel<float, false>, dim3(n_rows), dim3(NORM_THREADS), (size_t)(0), stream, y, ld_y, rows, w, (float*)out, ld_out, d, groups, eps, (__nv_bfloat16*)also_bf16);

@@ -321,7 +321,7 @@ int vlrf_matrix_state_scan(int kind, const float* q, int ldq, const float* k, in
                            int ld_decay, const float* s0, int ld_s0, const float* s1, int ld_s1, float q_scale, float cap, float* state,
                            int state_row, const int* seq_slot, const int* seq_start, const int* seq_pos0, float* y, int ldy, float* den,
                            int n_seqs, int max_new, int H, int G, int K, int V, cudaStream_t stream);
-int vlrf_matrix_state_force_columns(int nc);
+int vlrf_matrix_state_force(int columns, int warps);    // for measurements and tests: columns a lane, warps a CTA (0: chosen)
 // Convolution, x·sigmoid(x) and unit norms of q and k over columns [q: G·K | k: G·K | v: H·V] of the float32 rows `proj`; out
 // [T][2·G·K + H·V]; kq [T][G] = k · q; the kept inputs lie at conv_off of the state rows.
 int vlrf_conv_unit(const float* proj, int ld, int x_off, const float* w, int taps, float* state, int state_row, int conv_off,
