@@ -279,10 +279,11 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
         } else if (MODE == MS_STABILIZED) {
             const float log_i = A.cap * tanhf(raw0 / A.cap), log_f = log_sigmoid(A.cap * tanhf(raw1 / A.cap));
             float before = 0.f, behind = 0.f;
-            for (int ii = 0; ii < nb; ++ii) {
+#pragma unroll
+            for (int ii = 0; ii < MS_MAX_BATCH; ++ii) {     // (written out, so that only the sum and the maximum wait for one another)
                 const float m_new = fmaxf(__shfl_sync(0xffffffffu, log_f, ii) + m_run, __shfl_sync(0xffffffffu, log_i, ii));
                 if (lane == ii) { before = m_run; behind = m_new; }
-                m_run = m_new;
+                if (ii < nb) m_run = m_new;
             }
             if (lane < B) { scal[2 * lane] = expf(log_f + before - behind); scal[2 * lane + 1] = expf(log_i - behind); }
             floor_mine = expf(-behind);

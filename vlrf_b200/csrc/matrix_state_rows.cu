@@ -16,6 +16,7 @@
 //   numbers for all heads or of H·V numbers; act sigmoid(z) or z · sigmoid(z); rounded to the activation dtype.
 // norm_pair_add: x[t] += factor · (RMSnorm(a[t]) · wa + RMSnorm(b[t]) · wb), float32; the rows fit registers.
 #include "common.cuh"
+#include <type_traits>
 
 namespace {
 constexpr float UNIT_EPS = 1e-6f, DEN_EPS = 1e-6f;
@@ -187,10 +188,15 @@ struct LowRankPart {
 };
 
 __device__ __forceinline__ float lr_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float lr_apply(const LowRankPart& P, float z, int col) {
-    if (P.bias != nullptr) z += P.bias[col];
-    if (P.kind == LR_POWER) return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * P.inv_tau);
-    if (P.kind == LR_SOFTPLUS) return expf(-expf(P.a_log[col / P.per]) * lr_softplus(z));
+// What f needs of a column: its bias, and for the softplus decay minus its rate.
+__device__ __forceinline__ float2 lr_column(const LowRankPart& P, int col) {
+    const bool in = col < P.cols;
+    return make_float2(in && P.bias != nullptr ? P.bias[col] : 0.f, in && P.kind == LR_SOFTPLUS ? -expf(P.a_log[col / P.per]) : P.inv_tau);
+}
+template <int KIND> __device__ __forceinline__ float lr_apply(float z, float2 c) {
+    z += c.x;
+    if (KIND == LR_POWER) return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * c.y);      // log sigmoid(z) / tau
+    if (KIND == LR_SOFTPLUS) return expf(c.y * lr_softplus(z));
     return z;
 }
 
@@ -203,7 +209,7 @@ lowrank_mma_kernel(const LowRankPart P0, const LowRankPart P1, int T) {
     pdl_wait();
     pdl_launch_dependents();
     const bool second = (int)blockIdx.x >= P0.tiles;
-    const LowRankPart& P = second ? P1 : P0;
+    const LowRankPart P = second ? P1 : P0;
     const int c0 = (blockIdx.x - (second ? P0.tiles : 0)) * CT, t0 = blockIdx.y * 64;
     constexpr int LD = LR_K + 8;                    // rows padded against bank conflicts
     __shared__ __align__(16) __nv_bfloat16 hi[64 * LD], lo[64 * LD], ws[CT * LD];
@@ -278,23 +284,33 @@ lowrank_mma_kernel(const LowRankPart P0, const LowRankPart P1, int T) {
             }
         }
     }
-    const bool pairs = (P.ldo & 1) == 0 && (cols & 1) == 0 && (reinterpret_cast<uintptr_t>(P.out) & 7) == 0;
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-        const int row = t0 + warp * 16 + g + half * 8;
-        if (row >= T) continue;
-        float* o = P.out + (size_t)row * P.ldo;
+    float* out = P.out;
+    const int ldo = P.ldo;
+    const bool pairs = (ldo & 1) == 0 && (cols & 1) == 0 && (reinterpret_cast<uintptr_t>(out) & 7) == 0;
+    auto finish = [&](auto kind) {
+        constexpr int KIND = decltype(kind)::value;
 #pragma unroll
         for (int j = 0; j < CT / 8; ++j) {
             const int col = c0 + j * 8 + 2 * t;
-            if (pairs) {
-                if (col < cols) *reinterpret_cast<float2*>(o + col) = make_float2(lr_apply(P, acc[j][2 * half], col), lr_apply(P, acc[j][2 * half + 1], col + 1));
-            } else {
-                if (col < cols) o[col] = lr_apply(P, acc[j][2 * half], col);
-                if (col + 1 < cols) o[col + 1] = lr_apply(P, acc[j][2 * half + 1], col + 1);
+            if (col >= cols) break;
+            const float2 k0 = lr_column(P, col), k1 = lr_column(P, col + 1);
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int row = t0 + warp * 16 + g + half * 8;
+                if (row >= T) continue;
+                float* o = out + (size_t)row * ldo + col;
+                const float x0 = lr_apply<KIND>(acc[j][2 * half], k0), x1 = lr_apply<KIND>(acc[j][2 * half + 1], k1);
+                if (pairs) *reinterpret_cast<float2*>(o) = make_float2(x0, x1);
+                else {
+                    o[0] = x0;
+                    if (col + 1 < cols) o[1] = x1;
+                }
             }
         }
-    }
+    };
+    if (P.kind == LR_SOFTPLUS) finish(std::integral_constant<int, LR_SOFTPLUS>{});
+    else if (P.kind == LR_POWER) finish(std::integral_constant<int, LR_POWER>{});
+    else finish(std::integral_constant<int, LR_PLAIN>{});
 }
 
 // float32 weights: the same tile, four by eight results a thread
@@ -334,7 +350,10 @@ lowrank_fma_kernel(const LowRankPart P0, const LowRankPart P1, int T) {
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int col = c0 + tx + 16 * j;
-            if (col < P.cols) P.out[(size_t)row * P.ldo + col] = lr_apply(P, acc[i][j], col);
+            if (col >= P.cols) continue;
+            const float2 c = lr_column(P, col);
+            P.out[(size_t)row * P.ldo + col] = P.kind == LR_SOFTPLUS ? lr_apply<LR_SOFTPLUS>(acc[i][j], c)
+                                               : P.kind == LR_POWER ? lr_apply<LR_POWER>(acc[i][j], c) : lr_apply<LR_PLAIN>(acc[i][j], c);
         }
     }
 }

@@ -90,7 +90,8 @@ class ParallelSublayersBlock:
     matrix of its own has `from_projection`, a feed-forward with more to do than its staged part has `finish`) share their
     products: one product of h gives the mixer's and the feed-forward's input columns, float32, each range beginning on a
     multiple of eight columns; both write their inner rows side by side, and one product over the concatenated output
-    matrices adds the two sublayers to x.  Other parts run one after the other on the same h."""
+    matrices adds the two sublayers to x.  Whatever of the two needs nothing of the other (the routed experts and the mixer's
+    recurrence) is enqueued on two streams.  Other parts run one after the other on the same h."""
 
     leaves_row_stats = False
 
@@ -153,22 +154,35 @@ class ParallelSublayersBlock:
         if self.joint_out:
             m = mixer.merged_width
             merged = ws.get("sublayers_merged", T, m + ff.merged_width, ctx.act_dtype)
-            mixer.core(proj[:, :mixer.in_width], merged[:, :m], ctx, view, writes_cache)
-            ff.core(ff_proj, merged[:, m:], ctx, h)
+            if hasattr(ff, "finish"):
+                # what the feed-forward does besides its staged part runs beside the mixer
+                with ws.beside():
+                    mixer.core(proj[:, :mixer.in_width], merged[:, :m], ctx, view, writes_cache)
+                ff.core(ff_proj, merged[:, m:], ctx, h)
+                ff.finish(h, ff_proj, x, ctx)
+                ws.join()
+            else:
+                mixer.core(proj[:, :mixer.in_width], merged[:, :m], ctx, view, writes_cache)
+                ff.core(ff_proj, merged[:, m:], ctx, h)
             ops.linear(merged, self.out_weight, None, x, residual=x)
-        else:
+            return
+
+        def feed_forward():
             if ff.out_weight is not None:
                 u = ws.get("sublayers_ff_inner", T, ff.merged_width, ctx.act_dtype)
                 ff.core(ff_proj, u, ctx, h)
                 ops.linear(u, ff.out_weight, None, x, residual=x)
-            if mixer.out_weight is None:
-                mixer.from_projection(proj[:, :mixer.in_width], x, ctx, view, writes_cache)
-            else:
-                merged = ws.get("sublayers_merged", T, mixer.merged_width, ctx.act_dtype)
+            if hasattr(ff, "finish"):
+                ff.finish(h, ff_proj, x, ctx)
+        if mixer.out_weight is None:
+            mixer.from_projection(proj[:, :mixer.in_width], x, ctx, view, writes_cache, meanwhile=feed_forward)
+        else:
+            merged = ws.get("sublayers_merged", T, mixer.merged_width, ctx.act_dtype)
+            with ws.beside():
                 mixer.core(proj[:, :mixer.in_width], merged, ctx, view, writes_cache)
-                ops.linear(merged, mixer.out_weight, None, x, residual=x)
-        if hasattr(ff, "finish"):
-            ff.finish(h, ff_proj, x, ctx)
+            feed_forward()
+            ws.join()
+            ops.linear(merged, mixer.out_weight, None, x, residual=x)
 
 
 @register_part("block", "sublayer_norm")

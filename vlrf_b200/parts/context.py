@@ -7,6 +7,7 @@ decoded tokens.
 """
 from __future__ import annotations
 
+import contextlib
 import dataclasses
 
 import torch
@@ -20,6 +21,7 @@ class Workspace:
     def __init__(self, device):
         self.device = torch.device(device)
         self._bufs: dict[str, torch.Tensor] = {}
+        self._side = None        # the second stream of `beside`
         self._views: dict = {}   # (name, rows, cols, dtype) -> the view handed out last time (making one costs 2 to 3 us)
         self.frozen = False  # set while a captured graph depends on the addresses
         self.generation = 0  # counts (re)allocations: captured steps are valid for one generation only
@@ -68,6 +70,21 @@ class Workspace:
             self._bufs[name] = buf
             self.generation += 1
         return buf[:n]
+
+    @contextlib.contextmanager
+    def beside(self):
+        """What the body enqueues runs on a second stream, behind everything enqueued so far and beside whatever the caller
+        enqueues next, until `join`.  The two may share nothing but what both only read.  (In a captured step: a fork of the
+        graph.)  Not nested."""
+        if self._side is None:
+            self._side = torch.cuda.Stream(device=self.device)
+        self._side.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(self._side):
+            yield
+
+    def join(self) -> None:
+        """Everything enqueued from here on runs behind what `beside` enqueued."""
+        torch.cuda.current_stream().wait_stream(self._side)
 
     def bytes(self) -> int:
         return sum(b.numel() * b.element_size() for b in self._bufs.values())

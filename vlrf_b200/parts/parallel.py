@@ -74,22 +74,31 @@ class ParallelMixer:
         self.right.core(proj[:, nl:self.in_width], merged[:, ml:self.merged_width], ctx, view.parts[1], writes_cache,
                         factor * self.right_scale)
 
-    def from_projection(self, proj, x: torch.Tensor, ctx: StepContext, view, writes_cache: bool = True, accumulate: bool = True) -> None:
-        """From the input product's float32 result to the residual."""
+    def from_projection(self, proj, x: torch.Tensor, ctx: StepContext, view, writes_cache: bool = True, accumulate: bool = True,
+                        meanwhile=None) -> None:
+        """From the input product's float32 result to the residual.  With normed outputs the branches run beside each other;
+        `meanwhile` (a function, or None) enqueues what else may run then, and may add to x."""
         T, ws, width = ctx.n_tokens, ctx.ws, x.shape[1]
         if self.out_norms is None:
+            if meanwhile is not None:
+                meanwhile()
             merged = ws.get("parallel_merged", T, self.merged_width, ctx.act_dtype)
             self.core(proj, merged, ctx, view, writes_cache)
             ops.linear(merged, self.out_weight, None, x, residual=x if accumulate else None)
             return
         nl = self.left.in_width
-        outs = []
-        for name, branch, cols, part in (("left", self.left, proj[:, :nl], view.parts[0]),
-                                         ("right", self.right, proj[:, nl:self.in_width], view.parts[1])):
+        outs = [ws.get("parallel_out_" + name, T, width, torch.float32) for name in ("left", "right")]
+
+        def run(name, branch, cols, part, out):
             merged = ws.get("parallel_merged_" + name, T, branch.merged_width, ctx.act_dtype)
             branch.core(cols, merged, ctx, part, writes_cache)
-            outs.append(ws.get("parallel_out_" + name, T, width, torch.float32))
-            ops.linear(merged, branch.out_weight, None, outs[-1])
+            ops.linear(merged, branch.out_weight, None, out)
+        with ws.beside():
+            run("right", self.right, proj[:, nl:self.in_width], view.parts[1], outs[1])
+        run("left", self.left, proj[:, :nl], view.parts[0], outs[0])
+        if meanwhile is not None:
+            meanwhile()
+        ws.join()
         w_left, w_right, eps = self.out_norms
         ops.norm_pair_add(outs[0], outs[1], w_left, w_right, x, T, eps, self.left_scale, accumulate)
 
