@@ -29,7 +29,7 @@
 
 namespace {
 constexpr int MS_WARPS = 4;
-constexpr int MS_MAX_BATCH = 16;
+constexpr int MS_MAX_BATCH = 32;       // a lane per token works out a batch's gates
 constexpr int MS_DECAYED = 0, MS_DELTA = 1, MS_STABILIZED = 2;
 
 typedef unsigned long long f32x2;
@@ -216,6 +216,13 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
             ms_sm[st * stage_floats + (row - st * ROWS * B) * KP + cc] = 0.f;
         }
     }
+    // who copies what: a thread's first token, column and step in tokens, for rows of K and of CW numbers in quads
+    const bool whole_rows = A.vec_rows && n_thr % (K / 4) == 0;
+    const int ii0 = whole_rows ? threadIdx.x / (K / 4) : 0, ii_step = whole_rows ? n_thr / (K / 4) : 1, q_col = (threadIdx.x - ii0 * (K / 4)) * 4;
+    const int v0 = threadIdx.x / (CW / 4), v_step = n_thr / (CW / 4), v_col = (threadIdx.x - v0 * (CW / 4)) * 4;
+    if (MODE == MS_STABILIZED && pb * CW <= V && V < pb * CW + CW) {        // the column of n takes k itself: its value is always 1
+        for (int i = threadIdx.x; i < 2 * B; i += n_thr) ms_sm[(i / B) * stage_floats + ROWS * B * KP + (i % B) * CW + (V - pb * CW)] = 1.f;
+    }
     auto fetch = [&](int i0, int st) {              // all threads: the inputs of the batch that begins at token i0
         const int nb = min(B, n - i0);
         float* ks = ms_sm + st * stage_floats;
@@ -223,7 +230,13 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
         float* ds = qs + B * KP;
         float* vs = ms_sm + st * stage_floats + ROWS * B * KP;
         const size_t t0 = (size_t)(start + i0);
-        if (A.vec_rows) {
+        if (whole_rows) {                           // a thread's quads lie in one column of quads: no division here
+            for (int ii = ii0; ii < nb; ii += ii_step) {
+                ms_cp16(ks + ii * KP + q_col, A.k + (t0 + ii) * A.ldk + g * K + q_col);
+                ms_cp16(qs + ii * KP + q_col, A.q + (t0 + ii) * A.ldq + g * K + q_col);
+                if (DECAY) ms_cp16(ds + ii * KP + q_col, A.decay + (t0 + ii) * A.ld_decay + h * K + q_col);
+            }
+        } else if (A.vec_rows) {
             const int q4 = K / 4;
             for (int i = threadIdx.x; i < nb * q4; i += n_thr) {
                 const int ii = i / q4, cc = (i - ii * q4) * 4;
@@ -240,10 +253,8 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
             }
         }
         if (A.vec_v) {                              // (V a multiple of 4: a group of four columns is whole or not there)
-            for (int i = threadIdx.x; i < nb * (CW / 4); i += n_thr) {
-                const int ii = i / (CW / 4), cc = (i - ii * (CW / 4)) * 4;
-                if (pb * CW + cc < V) ms_cp16(vs + ii * CW + cc, A.v + (t0 + ii) * A.ldv + h * V + pb * CW + cc);
-            }
+            if (pb * CW + v_col < V)
+                for (int ii = v0; ii < nb; ii += v_step) ms_cp16(vs + ii * CW + v_col, A.v + (t0 + ii) * A.ldv + h * V + pb * CW + v_col);
         } else {
             for (int i = threadIdx.x; i < nb * CW; i += n_thr) {
                 const int ii = i / CW, cc = i - ii * CW;
@@ -278,13 +289,18 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
             if (lane < B) { scal[2 * lane] = sigmoid_f(raw0); scal[2 * lane + 1] = raw1; }
         } else if (MODE == MS_STABILIZED) {
             const float log_i = A.cap * tanhf(raw0 / A.cap), log_f = log_sigmoid(A.cap * tanhf(raw1 / A.cap));
-            float before = 0.f, behind = 0.f;
+            // m of every token by a scan over the lanes: from m before lane's token and the ones ahead of it, m becomes
+            // max(sum_f + m, top), and two such steps one after the other are a step of the same form
+            float sum_f = lane < nb ? log_f : 0.f, top = lane < nb ? log_i : -INFINITY;
 #pragma unroll
-            for (int ii = 0; ii < MS_MAX_BATCH; ++ii) {     // (written out, so that only the sum and the maximum wait for one another)
-                const float m_new = fmaxf(__shfl_sync(0xffffffffu, log_f, ii) + m_run, __shfl_sync(0xffffffffu, log_i, ii));
-                if (lane == ii) { before = m_run; behind = m_new; }
-                if (ii < nb) m_run = m_new;
+            for (int o = 1; o < 32; o <<= 1) {
+                const float pf = __shfl_up_sync(0xffffffffu, sum_f, o), pt = __shfl_up_sync(0xffffffffu, top, o);
+                if (lane >= o) { top = fmaxf(pt + sum_f, top); sum_f += pf; }
             }
+            const float behind = fmaxf(sum_f + m_run, top);
+            float before = __shfl_up_sync(0xffffffffu, behind, 1);
+            if (lane == 0) before = m_run;
+            m_run = __shfl_sync(0xffffffffu, behind, 31);
             if (lane < B) { scal[2 * lane] = expf(log_f + before - behind); scal[2 * lane + 1] = expf(log_i - behind); }
             floor_mine = expf(-behind);
         }
@@ -315,7 +331,7 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
                     else rows_of(ii, X[0]);
                     float v[NC];
 #pragma unroll
-                    for (int e = 0; e < NC; ++e) v[e] = my_col + e < V ? vs[ii * CW + e] : (MODE == MS_STABILIZED && my_col + e == V) ? 1.f : 0.f;
+                    for (int e = 0; e < NC; ++e) v[e] = vs[ii * CW + e];     // (columns that do not exist: anything, it goes nowhere)
                     float2 ab = make_float2(0.f, 0.f);
                     if (MODE != MS_DECAYED) ab = *reinterpret_cast<const float2*>(scal + 2 * ii);
                     advance<MODE, NR, NC>(S, X[AHEAD ? (t & 1) : 0], v, ab.x, ab.y, r, p[t]);
