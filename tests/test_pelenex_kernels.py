@@ -211,7 +211,7 @@ def test_convolution_and_unit_norms_over_steps(H, G, K, V, taps):
 
 
 @pytest.mark.parametrize("dt", DT)
-@pytest.mark.parametrize("T,rank,rank2,H,K,V", [(1, 16, 24, 2, 32, 16), (70, 5, 33, 3, 24, 10), (64, 64, 8, 4, 33, 40), (3, 1, 128, 1, 130, 7), (129, 40, 40, 2, 64, 64)])
+@pytest.mark.parametrize("T,rank,rank2,H,K,V", [(1, 16, 24, 2, 32, 16), (200, 256, 24, 1, 200, 40), (90, 264, 8, 1, 60, 24), (70, 5, 33, 3, 24, 10), (64, 64, 8, 4, 33, 40), (3, 1, 128, 1, 130, 7), (129, 40, 40, 2, 64, 64)])
 def test_low_rank_decays_and_gates(T, rank, rank2, H, K, V, dt):
     from vlrf_b200.csrc import ops
     g = torch.Generator().manual_seed(T + rank)
