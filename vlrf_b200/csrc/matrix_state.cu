@@ -19,11 +19,13 @@
 //
 // The kernel: eight lanes share the rows of a column and a warp takes 4·NC columns, its part of the state in registers as
 // pairs of rows (`fma.rn.f32x2`: two multiply-adds an instruction); a CTA of four warps takes 16·NC columns of a
-// head of a sequence.  k, q, a and v of up to 16 tokens at a time arrive in shared memory by `cp.async` a batch ahead.  The
+// head of a sequence.  k, q, a and v of up to 32 tokens at a time arrive in shared memory by `cp.async` a batch ahead, and a
+// token's rows are fetched from there while the token before is worked on.  The
 // columns of a state never meet.  Sums over rows: kind 1 needs Sᵀk before it can go on (three exchanges among the eight
 // lanes a token, with Sᵀq taken of the state before the write and u (k · q) added, so the read-out waits for nothing);
 // the read-outs of eight tokens are summed together, seven exchanges for all eight, and lane r ends up with token r's.
-// Prompts and single tokens run the same arithmetic in the same order.
+// A step of single tokens has a kernel of its own (matrix_state_step) that reads and writes memory directly; both run the same
+// arithmetic in the same order.
 #include "common.cuh"
 #include <type_traits>
 
