@@ -92,7 +92,7 @@ _SIGNATURES = {
                            _c_float, _c_int, _c_void_p, _c_void_p],
     "vlrf_cast_rows": [_c_void_p, _c_void_p, _c_int, ctypes.c_longlong, _c_void_p],
     "vlrf_gate_mul": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-                      _c_void_p],
+                      _c_float, _c_void_p],
     "vlrf_embed_streams": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p],
     "vlrf_streams_read_norm": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float,
                                _c_void_p],
@@ -107,13 +107,14 @@ _SIGNATURES = {
                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_float, _c_void_p, _c_void_p],
     "vlrf_qkv_norm_rope_append": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p,
                                   _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                  _c_int, _c_void_p, _c_void_p, _c_float, _c_int, _c_float, _c_void_p, _c_void_p],
+                                  _c_int, _c_int, _c_void_p, _c_void_p, _c_float, _c_int, _c_float, _c_void_p, _c_void_p],
     "vlrf_attn_window_ex": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_float, _c_float, _c_int, _c_void_p,
-                            _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p],
+                            _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_float, _c_void_p, _c_void_p],
     "vlrf_attn_window_mma_ex": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                                 _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_float,
-                                _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p],
+                                _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_float, _c_void_p,
+                                _c_void_p],
     "vlrf_embed_bigram": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
                           _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p],
     "vlrf_scale_values": [_c_void_p, ctypes.c_longlong, _c_float, _c_void_p],
@@ -131,7 +132,7 @@ _SIGNATURES = {
                            _c_float, _c_float, _c_void_p],
         "vlrf_matrix_state_scan": [_c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int,
         _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_float, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
-        _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+        _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
         "vlrf_matrix_state_force": [_c_int, _c_int],
         "vlrf_conv_unit": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p,
         _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
@@ -148,26 +149,26 @@ _SIGNATURES = {
                         _c_int, _c_int, _c_void_p],
     "vlrf_gemm_grouped": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                           _c_int, _c_void_p],
-    "vlrf_latent_append": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_void_p, _c_int, _c_int, _c_void_p, _c_int,
+    "vlrf_latent_append": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_void_p, _c_int, _c_int, _c_float, _c_void_p, _c_int,
                            _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p],
-    "vlrf_latent_q_rows": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int,
+    "vlrf_latent_q_rows": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p, _c_void_p, _c_int,
                            _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "vlrf_attn_latent": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p,
-                         _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p],
+                         _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p],
     "vlrf_latent_gather": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
                            _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p],
     "vlrf_attn_rows_takes": [_c_int] * 9,
     "vlrf_attn_rows": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p,
-                       _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p],
+                       _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_float, _c_void_p],
     "vlrf_attn_latent_mma_takes": [_c_int, _c_int, _c_int, _c_int, _c_int],
     "vlrf_attn_latent_mma_group": [_c_int, _c_int],
     "vlrf_attn_latent_mma_ctas_per_sm": [_c_int, _c_int],
     "vlrf_attn_latent_mma": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p,
                              _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p,
-                             _c_void_p, _c_void_p],
+                             _c_void_p, _c_float, _c_void_p, _c_void_p],
     "vlrf_moe_route": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
                        _c_void_p, _c_int, _c_void_p],
-    "vlrf_moe_route_scored": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p,
+    "vlrf_moe_route_scored": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p,
                               _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p],
     "vlrf_moe_plan": [_c_void_p, _c_void_p, _c_int, _c_void_p],
     "vlrf_moe_gather": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,

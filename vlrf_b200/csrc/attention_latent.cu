@@ -18,7 +18,10 @@
 // Rotation: of a vector's first `dims` entries, entry i is paired with entry i + dims/2 ("rotate half" pairing), or,
 // with `interleaved`, entry 2i with entry 2i + 1; the pair (u, v) at position p becomes (u cos a − v sin a,
 // v cos a + u sin a), a = p · inv_freq[i]; entries beyond `dims` pass unchanged.  inv_freq is a float32 table from the
-// caller.
+// caller; `magnitude` multiplies every cosine and sine.
+//
+// Attention's further parameters: window (position i sees j with i − j < window), sink (a float32 per head, or null: exp(sink_h)
+// is one more term of the softmax's denominator, with nothing in the numerator), out_scale (a factor on the result).
 //
 // The cache of one layer is [block][BT][row_w] with row_w ≥ C + R; block_table as for the key/value cache.
 #include "common.cuh"
@@ -27,10 +30,12 @@ namespace {
 constexpr int LAT_WARPS = 4;
 constexpr int LAT_MAX_C = 1024;          // latent width the general kernel holds in registers (32 a lane)
 
-__device__ __forceinline__ void rotate_pair(float u, float v, float pos, float f, float& ou, float& ov) {
+__device__ __forceinline__ void rotate_pair(float u, float v, float pos, float f, float magnitude, float& ou, float& ov) {
     const float a = pos * f;
     float s, c;
     sincosf(a, &s, &c);
+    s *= magnitude;
+    c *= magnitude;
     ou = u * c - v * s;
     ov = v * c + u * s;
 }
@@ -38,7 +43,7 @@ __device__ __forceinline__ void rotate_pair(float u, float v, float pos, float f
 template <typename ET>
 __global__ void __launch_bounds__(128)
 latent_append_kernel(const float* __restrict__ proj, int ld, int C, int R, const float* __restrict__ norm_w, float eps,
-                     const float* __restrict__ inv_freq, int rot_dims, int interleaved, ET* __restrict__ cache, int row_w,
+                     const float* __restrict__ inv_freq, int rot_dims, int interleaved, float magnitude, ET* __restrict__ cache, int row_w,
                      const int* __restrict__ block_table, int max_blocks, const int* __restrict__ tok_slot,
                      const int* __restrict__ tok_pos, int BT, int* __restrict__ dev_err) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
@@ -67,7 +72,7 @@ latent_append_kernel(const float* __restrict__ proj, int ld, int C, int R, const
     for (int i = threadIdx.x; i < half; i += 128) {
         const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
         float ou, ov;
-        rotate_pair(src[C + a], src[C + b], (float)pos, inv_freq[i], ou, ov);
+        rotate_pair(src[C + a], src[C + b], (float)pos, inv_freq[i], magnitude, ou, ov);
         ElemIO<ET>::store(dst + C + a, ou);
         ElemIO<ET>::store(dst + C + b, ov);
     }
@@ -77,7 +82,7 @@ latent_append_kernel(const float* __restrict__ proj, int ld, int C, int R, const
 template <typename ET>
 __global__ void __launch_bounds__(128)
 latent_q_rows_kernel(const float* __restrict__ q, int ld_q, int H, int dim, int R, const float* __restrict__ inv_freq,
-                     int rot_dims, int interleaved, const int* __restrict__ tok_pos, ET* __restrict__ qn, int ld_qn,
+                     int rot_dims, int interleaved, float magnitude, const int* __restrict__ tok_pos, ET* __restrict__ qn, int ld_qn,
                      ET* __restrict__ qp, int ld_qp, int C) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
@@ -94,7 +99,7 @@ latent_q_rows_kernel(const float* __restrict__ q, int ld_q, int H, int dim, int 
         const float* s = src + h * per + dim;
         const int a = interleaved ? 2 * c : c, b = interleaved ? 2 * c + 1 : c + half;
         float ou, ov;
-        rotate_pair(s[a], s[b], pos, inv_freq[c], ou, ov);
+        rotate_pair(s[a], s[b], pos, inv_freq[c], magnitude, ou, ov);
         ET* d = qp + (size_t)t * ld_qp + (size_t)h * (C + R) + C;
         ElemIO<ET>::store(d + a, ou);
         ElemIO<ET>::store(d + b, ov);
@@ -131,7 +136,7 @@ __global__ void __launch_bounds__(LAT_WARPS * 32)
 attn_latent_kernel(const ET* __restrict__ qp, int ld_q, const ET* __restrict__ cache, int row_w, int C, int R,
                    const int* __restrict__ block_table, int max_blocks, const int* __restrict__ tok_slot,
                    const int* __restrict__ tok_pos, ET* __restrict__ out, int ld_out, int H, int BT, float scale,
-                   int window, int* __restrict__ dev_err) {
+                   int window, const float* __restrict__ sink, float out_scale, int* __restrict__ dev_err) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
     extern __shared__ float q_sm[];                            // [LAT_WARPS][C + R]
@@ -192,7 +197,13 @@ attn_latent_kernel(const ET* __restrict__ qp, int ld_q, const ET* __restrict__ c
         m = m_new;
     }
     if (lost && lane == 0) atomicOr(dev_err, VLRF_DEVERR_NO_BLOCK);
-    const float inv = (l > 0.f) ? 1.f / l : 0.f;
+    float f = out_scale;
+    if (sink != nullptr) {                                     // exp(sink) joins the denominator: no key, no value
+        const float sk = sink[h], m_new = fmaxf(m, sk), corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
+        l = l * corr + expf(sk - m_new);
+        f *= corr;
+    }
+    const float inv = (l > 0.f) ? f / l : 0.f;
 #pragma unroll
     for (int i = 0; i < LAT_MAX_C / 32; ++i) {
         const int c = i * 32 + lane;
@@ -202,7 +213,7 @@ attn_latent_kernel(const ET* __restrict__ qp, int ld_q, const ET* __restrict__ c
 }  // namespace
 
 extern "C" int vlrf_latent_append(const float* proj, int ld, int C, int R, const float* norm_w, float eps,
-                                  const float* inv_freq, int rot_dims, int interleaved, void* cache, int dtype, int row_w,
+                                  const float* inv_freq, int rot_dims, int interleaved, float magnitude, void* cache, int dtype, int row_w,
                                   const int* block_table, int max_blocks, const int* tok_slot, const int* tok_pos,
                                   int T, int BT, int* dev_err, cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && C > 0 && R >= 0 && ld >= C + R && row_w >= C + R && BT > 0 && max_blocks > 0, "latent_append: bad sizes");
@@ -211,24 +222,24 @@ extern "C" int vlrf_latent_append(const float* proj, int ld, int C, int R, const
     VLRF_REQUIRE(norm_w != nullptr && dev_err != nullptr, "latent_append: needs the norm's weight and the device error word");
     if (T == 0) return VLRF_OK;
     if (dtype == VLRF_F32)
-        launch_chained(latent_append_kernel<float>, dim3(T), dim3(128), (size_t)(0), stream, proj, ld, C, R, norm_w, eps, inv_freq, rot_dims, interleaved, (float*)cache, row_w, block_table, max_blocks, tok_slot, tok_pos, BT, dev_err);
+        launch_chained(latent_append_kernel<float>, dim3(T), dim3(128), (size_t)(0), stream, proj, ld, C, R, norm_w, eps, inv_freq, rot_dims, interleaved, magnitude, (float*)cache, row_w, block_table, max_blocks, tok_slot, tok_pos, BT, dev_err);
     else if (dtype == VLRF_BF16)
-        launch_chained(latent_append_kernel<__nv_bfloat16>, dim3(T), dim3(128), (size_t)(0), stream, proj, ld, C, R, norm_w, eps, inv_freq, rot_dims, interleaved, (__nv_bfloat16*)cache, row_w, block_table, max_blocks, tok_slot, tok_pos, BT, dev_err);
+        launch_chained(latent_append_kernel<__nv_bfloat16>, dim3(T), dim3(128), (size_t)(0), stream, proj, ld, C, R, norm_w, eps, inv_freq, rot_dims, interleaved, magnitude, (__nv_bfloat16*)cache, row_w, block_table, max_blocks, tok_slot, tok_pos, BT, dev_err);
     else return vlrf_fail(VLRF_ERR_INVALID_ARG, "latent_append: unknown dtype %d", dtype);
     return vlrf_check_launch("latent_append");
 }
 
 extern "C" int vlrf_latent_q_rows(const float* q, int ld_q, int H, int dim, int R, const float* inv_freq, int rot_dims, int interleaved,
-                                  const int* tok_pos, void* qn, int ld_qn, void* qp, int ld_qp, int C, int dtype, int T,
+                                  float magnitude, const int* tok_pos, void* qn, int ld_qn, void* qp, int ld_qp, int C, int dtype, int T,
                                   cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && H > 0 && dim > 0 && R >= 0 && C >= 0, "latent_q_rows: bad sizes");
     VLRF_REQUIRE(ld_q >= H * (dim + R) && ld_qn >= H * dim && ld_qp >= H * (C + R), "latent_q_rows: leading sizes are too small");
     VLRF_REQUIRE(rot_dims >= 0 && rot_dims <= R && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq != nullptr), "latent_q_rows: bad rotation");
     if (T == 0) return VLRF_OK;
     if (dtype == VLRF_F32)
-        launch_chained(latent_q_rows_kernel<float>, dim3(T), dim3(128), (size_t)(0), stream, q, ld_q, H, dim, R, inv_freq, rot_dims, interleaved, tok_pos, (float*)qn, ld_qn, (float*)qp, ld_qp, C);
+        launch_chained(latent_q_rows_kernel<float>, dim3(T), dim3(128), (size_t)(0), stream, q, ld_q, H, dim, R, inv_freq, rot_dims, interleaved, magnitude, tok_pos, (float*)qn, ld_qn, (float*)qp, ld_qp, C);
     else if (dtype == VLRF_BF16)
-        launch_chained(latent_q_rows_kernel<__nv_bfloat16>, dim3(T), dim3(128), (size_t)(0), stream, q, ld_q, H, dim, R, inv_freq, rot_dims, interleaved, tok_pos, (__nv_bfloat16*)qn, ld_qn, (__nv_bfloat16*)qp, ld_qp, C);
+        launch_chained(latent_q_rows_kernel<__nv_bfloat16>, dim3(T), dim3(128), (size_t)(0), stream, q, ld_q, H, dim, R, inv_freq, rot_dims, interleaved, magnitude, tok_pos, (__nv_bfloat16*)qn, ld_qn, (__nv_bfloat16*)qp, ld_qp, C);
     else return vlrf_fail(VLRF_ERR_INVALID_ARG, "latent_q_rows: unknown dtype %d", dtype);
     return vlrf_check_launch("latent_q_rows");
 }
@@ -251,8 +262,8 @@ extern "C" int vlrf_latent_gather(const void* cache, int dtype, int row_w, int C
 
 extern "C" int vlrf_attn_latent(const void* qp, int dtype, int ld_q, const void* cache, int row_w, int C, int R,
                                 const int* block_table, int max_blocks, const int* tok_slot, const int* tok_pos,
-                                void* out, int ld_out, int T, int H, int BT, float scale, int window, int* dev_err,
-                                cudaStream_t stream) {
+                                void* out, int ld_out, int T, int H, int BT, float scale, int window, const float* sink,
+                                float out_scale, int* dev_err, cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && H > 0 && C > 0 && R >= 0 && max_blocks > 0, "attn_latent: bad sizes");
     VLRF_REQUIRE(C <= LAT_MAX_C, "attn_latent: a latent of %d numbers is wider than %d", C, LAT_MAX_C);
     VLRF_REQUIRE(row_w >= C + R && ld_q >= H * (C + R) && ld_out >= H * C, "attn_latent: leading sizes are too small");
@@ -262,9 +273,9 @@ extern "C" int vlrf_attn_latent(const void* qp, int dtype, int ld_q, const void*
     dim3 grid(T, (H + LAT_WARPS - 1) / LAT_WARPS);
     const size_t smem = (size_t)LAT_WARPS * (C + R) * sizeof(float);
     if (dtype == VLRF_F32)
-        launch_chained(attn_latent_kernel<float>, dim3(grid), dim3(LAT_WARPS * 32), (size_t)(smem), stream, (const float*)qp, ld_q, (const float*)cache, row_w, C, R, block_table, max_blocks, tok_slot, tok_pos, (float*)out, ld_out, H, BT, scale, window, dev_err);
+        launch_chained(attn_latent_kernel<float>, dim3(grid), dim3(LAT_WARPS * 32), (size_t)(smem), stream, (const float*)qp, ld_q, (const float*)cache, row_w, C, R, block_table, max_blocks, tok_slot, tok_pos, (float*)out, ld_out, H, BT, scale, window, sink, out_scale, dev_err);
     else if (dtype == VLRF_BF16)
-        launch_chained(attn_latent_kernel<__nv_bfloat16>, dim3(grid), dim3(LAT_WARPS * 32), (size_t)(smem), stream, (const __nv_bfloat16*)qp, ld_q, (const __nv_bfloat16*)cache, row_w, C, R, block_table, max_blocks, tok_slot, tok_pos, (__nv_bfloat16*)out, ld_out, H, BT, scale, window, dev_err);
+        launch_chained(attn_latent_kernel<__nv_bfloat16>, dim3(grid), dim3(LAT_WARPS * 32), (size_t)(smem), stream, (const __nv_bfloat16*)qp, ld_q, (const __nv_bfloat16*)cache, row_w, C, R, block_table, max_blocks, tok_slot, tok_pos, (__nv_bfloat16*)out, ld_out, H, BT, scale, window, sink, out_scale, dev_err);
     else return vlrf_fail(VLRF_ERR_INVALID_ARG, "attn_latent: unknown dtype %d", dtype);
     return vlrf_check_launch("attn_latent");
 }

@@ -14,6 +14,9 @@
 // and sum, meet in a second kernel).  Tiles arrive by `cp.async` into two buffers; rows behind the last visible one are
 // filled with zeros, so nothing unwritten is ever multiplied.
 //
+// A sink's term joins a row's denominator where its parts are complete (in the kernel, or in the merge of a cut context), and
+// the result is multiplied by out_scale there.
+//
 // Sizes taken: C a multiple of 32 up to 512, R a multiple of 16, cache rows of a multiple of 8 numbers, blocks of a
 // multiple of 32 tokens.  Others go to attention_latent.cu.
 #include "common.cuh"
@@ -52,7 +55,7 @@ attn_latent_mma_kernel(const __nv_bfloat16* __restrict__ qp, int ld_q, const __n
                        int C, int R, const int* __restrict__ block_table, int max_blocks, const int* __restrict__ seq_slot,
                        const int* __restrict__ seq_start, const int* __restrict__ seq_pos0, int tiles_per_seq,
                        __nv_bfloat16* __restrict__ out, int ld_out, int H, int BT, float scale, int window, int n_split,
-                       float* __restrict__ partials, int* __restrict__ dev_err) {
+                       float* __restrict__ partials, const float* __restrict__ sink, float out_scale, int* __restrict__ dev_err) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char lm_raw[];
@@ -242,7 +245,18 @@ attn_latent_mma_kernel(const __nv_bfloat16* __restrict__ qp, int ld_q, const __n
     if (!active) return;
     const int tok = row0 + grp;
     if (n_split == 1) {
-        const float inv0 = l_run[0] > 0.f ? 1.f / l_run[0] : 0.f, inv1 = l_run[1] > 0.f ? 1.f / l_run[1] : 0.f;
+        float f[2] = {out_scale, out_scale};
+        if (sink != nullptr) {                                     // exp(sink) joins the denominator
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                if (g + 8 * r >= heads_here) continue;
+                const float sk = sink[hg * 16 + g + 8 * r], m2 = fmaxf(m_run[r], sk);
+                const float corr = (m_run[r] == -INFINITY) ? 0.f : expf(m_run[r] - m2);
+                l_run[r] = l_run[r] * corr + expf(sk - m2);
+                f[r] *= corr;
+            }
+        }
+        const float inv0 = l_run[0] > 0.f ? f[0] / l_run[0] : 0.f, inv1 = l_run[1] > 0.f ? f[1] / l_run[1] : 0.f;
 #pragma unroll
         for (int nt = 0; nt < LM_NT_MAX; ++nt) {
             if (nt < nt_cnt) {
@@ -274,7 +288,7 @@ attn_latent_mma_kernel(const __nv_bfloat16* __restrict__ qp, int ld_q, const __n
 // the parts of every (token, head) into one: weights exp(m_s − max m) on the parts' unnormalised sums
 __global__ void __launch_bounds__(128)
 attn_latent_merge_kernel(const float* __restrict__ partials, const int* __restrict__ tok_slot, __nv_bfloat16* __restrict__ out,
-                         int ld_out, int H, int C, int n_split) {
+                         int ld_out, int H, int C, int n_split, const float* __restrict__ sink, float out_scale) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
     const int tok = blockIdx.x, h = blockIdx.y;
@@ -286,14 +300,14 @@ attn_latent_merge_kernel(const float* __restrict__ partials, const int* __restri
     }
     const float* base = partials + ((size_t)tok * hgs + hg) * n_split * 16 * (C + 2) + (size_t)r * (C + 2);
     const size_t stride = (size_t)16 * (C + 2);
-    float m = -INFINITY;
+    float m = sink != nullptr ? sink[h] : -INFINITY;
     for (int s = 0; s < n_split; ++s) m = fmaxf(m, base[s * stride + C]);
-    float denom = 0.f;
+    float denom = sink != nullptr ? expf(sink[h] - m) : 0.f;
     for (int s = 0; s < n_split; ++s) {
         const float ms = base[s * stride + C];
         if (ms != -INFINITY) denom += expf(ms - m) * base[s * stride + C + 1];
     }
-    const float inv = denom > 0.f ? 1.f / denom : 0.f;
+    const float inv = denom > 0.f ? out_scale / denom : 0.f;
     for (int c = threadIdx.x; c < C; c += 128) {
         float v = 0.f;
         for (int s = 0; s < n_split; ++s) {
@@ -333,8 +347,8 @@ extern "C" int vlrf_attn_latent_mma_group(int C, int R) {
 extern "C" int vlrf_attn_latent_mma(const void* qp, int ld_q, const void* cache, int row_w, int C, int R,
                                     const int* block_table, int max_blocks, const int* seq_slot, const int* seq_start,
                                     const int* seq_pos0, void* out, int ld_out, int n_seqs, int max_new, int H, int BT,
-                                    float scale, int window, int n_split, float* partials, int* dev_err,
-                                    cudaStream_t stream) {
+                                    float scale, int window, int n_split, float* partials, const float* sink, float out_scale,
+                                    int* dev_err, cudaStream_t stream) {
     VLRF_REQUIRE(vlrf_attn_latent_mma_takes(C, R, row_w, BT, ld_q), "attn_latent_mma: does not take C=%d R=%d row=%d BT=%d ld_q=%d", C, R, row_w, BT, ld_q);
     VLRF_REQUIRE(n_seqs >= 0 && max_new >= 1 && H > 0 && max_blocks > 0 && window >= 0 && dev_err != nullptr, "attn_latent_mma: bad arguments");
     VLRF_REQUIRE(ld_q >= H * (C + R) && ld_out >= H * C && ld_out % 2 == 0, "attn_latent_mma: leading sizes are too small");
@@ -355,9 +369,9 @@ extern "C" int vlrf_attn_latent_mma(const void* qp, int ld_q, const void* cache,
     }
     launch_chained(kern, dim3(grid), dim3(G * 128), (size_t)(smem), stream, (const __nv_bfloat16*)qp, ld_q, (const __nv_bfloat16*)cache, row_w, C, R, block_table,
                                           max_blocks, seq_slot, seq_start, seq_pos0, tiles_per_seq, (__nv_bfloat16*)out, ld_out, H,
-                                          BT, scale, window, n_split, partials, dev_err);
+                                          BT, scale, window, n_split, partials, sink, out_scale, dev_err);
     int st = vlrf_check_launch("attn_latent_mma");
     if (st != VLRF_OK || n_split == 1) return st;
-    launch_chained(attn_latent_merge_kernel, dim3(dim3(n_seqs, H)), dim3(128), (size_t)(0), stream, partials, seq_slot, (__nv_bfloat16*)out, ld_out, H, C, n_split);
+    launch_chained(attn_latent_merge_kernel, dim3(dim3(n_seqs, H)), dim3(128), (size_t)(0), stream, partials, seq_slot, (__nv_bfloat16*)out, ld_out, H, C, n_split, sink, out_scale);
     return vlrf_check_launch("attn_latent_merge");
 }

@@ -6,13 +6,14 @@
 // other path.  Queries and keys have two parts that are stored apart: a part per head (dim columns: qn [T][H·dim],
 // kn [T][H·dim]) and a part whose key all heads share (R columns: qr [T][H·R], kr [T][≥ R] with a row stride of its
 // own; R may be 0).  The score of query i and key j ≤ i of the same sequence is (qn_h(i)·kn_h(j) + qr_h(i)·kr(j))·scale;
-// softmax in float32; values v [T][H·vdim]; out [T][H·vdim].
+// softmax in float32; values v [T][H·vdim]; out [T][H·vdim].  With window w > 0 query i sees keys i − w < j ≤ i; sink (a float32
+// per head, or null) adds exp(sink_h) to the softmax's denominator and nothing to its numerator; out_scale multiplies the result.
 //
 // A CTA takes 64 consecutive queries of one sequence and one head: four warps of 16 query rows each, whose MMA
 // operands stay in registers.  Tiles of 32 keys ([kn | kr] rows) and values arrive by `cp.async` in two buffers;
 // a warp multiplies its queries by the tile, keeps maximum and sum of its rows in registers, and adds P·V to its
-// accumulators (the scores' fragments are the next MMA's operands as they are).  Tiles wholly above a warp's rows are
-// skipped.  Sizes: dim + R one of 32, 64, 96, 128, 192, 256; dim and R multiples of 8; vdim a multiple of 8 up to 128.
+// accumulators (the scores' fragments are the next MMA's operands as they are).  Tiles wholly above a warp's rows or
+// wholly ahead of their windows are skipped.  Sizes: dim + R one of 32, 64, 96, 128, 192, 256; dim and R multiples of 8; vdim a multiple of 8 up to 128.
 #include "common.cuh"
 
 namespace {
@@ -43,7 +44,8 @@ __global__ void __launch_bounds__(128)
 attn_rows_kernel(const __nv_bfloat16* __restrict__ qn, int ld_qn, const __nv_bfloat16* __restrict__ qr, int ld_qr,
                  const __nv_bfloat16* __restrict__ kn, int ld_kn, const __nv_bfloat16* __restrict__ kr, int ld_kr,
                  const __nv_bfloat16* __restrict__ v, int ld_v, const int* __restrict__ seq_start, int n_seqs, int tiles_per_seq,
-                 __nv_bfloat16* __restrict__ out, int ld_out, int dim, int R, int vdim, float scale) {
+                 __nv_bfloat16* __restrict__ out, int ld_out, int dim, int R, int vdim, float scale, int window,
+                 const float* __restrict__ sink, float out_scale) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char ar_raw[];
@@ -97,21 +99,22 @@ attn_rows_kernel(const __nv_bfloat16* __restrict__ qn, int ld_qn, const __nv_bfl
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    const int n_tiles = q_last / AR_KT + 1;
+    const int tile0 = window > 0 ? max(0, q0 - window + 1) / AR_KT : 0, n_tiles = q_last / AR_KT + 1;
     const int my_q0 = q0 + 16 * w;                                 // this warp's rows: my_q0 + g and my_q0 + g + 8
     const int nt_cnt = vdim >> 3;
     float acc[AR_NT_MAX][4];
 #pragma unroll
     for (int i = 0; i < AR_NT_MAX; ++i) { acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f; }
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-    fetch(0, 0);
-    for (int tile = 0; tile < n_tiles; ++tile) {
+    fetch(tile0, tile0 & 1);
+    for (int tile = tile0; tile < n_tiles; ++tile) {
         const int buf = tile & 1;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                           // the tile has landed; the other buffer is free
         if (tile + 1 < n_tiles) fetch(tile + 1, buf ^ 1);
         const int key0 = tile * AR_KT;
         if (key0 > my_q0 + 15 || my_q0 >= len) continue;           // wholly above this warp's rows, or no rows at all
+        if (window > 0 && key0 + AR_KT - 1 <= my_q0 - window) continue;      // wholly ahead of its windows
         const __nv_bfloat16* kt = k_sm + (size_t)buf * AR_KT * LDK;
         const __nv_bfloat16* vt = v_sm + (size_t)buf * AR_KT * ldv;
         float s[4][4];
@@ -136,7 +139,7 @@ attn_rows_kernel(const __nv_bfloat16* __restrict__ qn, int ld_qn, const __nv_bfl
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = key0 + 8 * nt + 2 * t4 + (e & 1), q = my_q0 + g + 8 * (e >> 1);
-                s[nt][e] = key <= q ? s[nt][e] * scale : -INFINITY;
+                s[nt][e] = key <= q && (window == 0 || q - key < window) ? s[nt][e] * scale : -INFINITY;
                 mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
             }
         float corr[2];
@@ -195,7 +198,13 @@ attn_rows_kernel(const __nv_bfloat16* __restrict__ qn, int ld_qn, const __nv_bfl
     for (int r = 0; r < 2; ++r) {
         const int q = my_q0 + g + 8 * r;
         if (q >= len) continue;
-        const float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
+        float f = out_scale;
+        if (sink != nullptr) {                                     // exp(sink) joins the denominator
+            const float sk = sink[h], m2 = fmaxf(m_run[r], sk), c = m_run[r] == -INFINITY ? 0.f : expf(m_run[r] - m2);
+            l_run[r] = l_run[r] * c + expf(sk - m2);
+            f *= c;
+        }
+        const float inv = l_run[r] > 0.f ? f / l_run[r] : 0.f;
         __nv_bfloat16* dst = out + (size_t)(row0 + q) * ld_out + (size_t)h * vdim;
 #pragma unroll
         for (int nt = 0; nt < AR_NT_MAX; ++nt)
@@ -220,9 +229,10 @@ extern "C" int vlrf_attn_rows_takes(int dim, int R, int vdim, int ld_qn, int ld_
 
 extern "C" int vlrf_attn_rows(const void* qn, int ld_qn, const void* qr, int ld_qr, const void* kn, int ld_kn, const void* kr,
                               int ld_kr, const void* v, int ld_v, const int* seq_start, void* out, int ld_out, int n_seqs,
-                              int max_new, int H, int dim, int R, int vdim, float scale, cudaStream_t stream) {
+                              int max_new, int H, int dim, int R, int vdim, float scale, int window, const float* sink,
+                              float out_scale, cudaStream_t stream) {
     VLRF_REQUIRE(vlrf_attn_rows_takes(dim, R, vdim, ld_qn, ld_qr, ld_kn, ld_kr, ld_v, ld_out), "attn_rows: does not take dim=%d R=%d vdim=%d", dim, R, vdim);
-    VLRF_REQUIRE(n_seqs >= 0 && max_new >= 1 && H > 0 && H <= 65535 && seq_start != nullptr, "attn_rows: bad arguments");
+    VLRF_REQUIRE(n_seqs >= 0 && max_new >= 1 && H > 0 && H <= 65535 && seq_start != nullptr && window >= 0, "attn_rows: bad arguments");
     VLRF_REQUIRE(((reinterpret_cast<uintptr_t>(qn) | reinterpret_cast<uintptr_t>(kn) | reinterpret_cast<uintptr_t>(v) |
                    reinterpret_cast<uintptr_t>(qr) | reinterpret_cast<uintptr_t>(kr)) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 3) == 0,
                  "attn_rows: rows must start on 16-byte boundaries");
@@ -240,7 +250,7 @@ extern "C" int vlrf_attn_rows(const void* qn, int ld_qn, const void* qr, int ld_
         }                                                                                                                      \
         launch_chained(attn_rows_kernel<KQ>, grid, dim3(128), smem, stream, (const __nv_bfloat16*)qn, ld_qn, (const __nv_bfloat16*)qr, \
                        ld_qr, (const __nv_bfloat16*)kn, ld_kn, (const __nv_bfloat16*)kr, ld_kr, (const __nv_bfloat16*)v, ld_v,  \
-                       seq_start, n_seqs, tiles_per_seq, (__nv_bfloat16*)out, ld_out, dim, R, vdim, scale);                            \
+                       seq_start, n_seqs, tiles_per_seq, (__nv_bfloat16*)out, ld_out, dim, R, vdim, scale, window, sink, out_scale);                            \
     }
     switch ((dim + R) / 16) {
         case 2: AR_GO(2) break;

@@ -25,6 +25,9 @@
 //   positions); gate (float32 [T][ld_gate], a logit per query head) multiplies head h's result by sigmoid(gate[t][h]);
 //   slopes (a float32 per query head) take slope_h · (query position − key position) off every score, behind the cap;
 //   sink (one float32 a query head) adds the term exp(sink_h) to the softmax's denominator and nothing to its numerator.
+// maps 2 (both kernels): differential attention.  A query or key head is two maps of dk numbers, [map 1 | map 2] (the cache's key
+//   rows hold both, K [block][kv_head][BT][2·dk]); each map is a softmax of its own over the same values, and
+//   o = a₁ − map_factor · a₂ is divided by sqrt(mean(o²) + head_eps) over the head's dv numbers before out_scale.
 #include "common.cuh"
 
 namespace {
@@ -36,14 +39,17 @@ __global__ void __launch_bounds__(128)
 qkv_rope_append_kernel(const float* __restrict__ proj, int ld, int q_off, int k_off, int v_off, const float* __restrict__ freq,
                        int rot, ET* __restrict__ q_out, int ldq, ET* __restrict__ Kc, ET* __restrict__ Vc,
                        const int* __restrict__ block_table, int max_blocks, const int* __restrict__ tok_slot,
-                       const int* __restrict__ tok_pos, int H, int Hkv, int dk, int dv, int BT, int write_cache,
+                       const int* __restrict__ tok_pos, int H, int Hkv, int Hv, int dk, int dv, int BT, int write_cache,
                        int norm, const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int pairing,
                        float magnitude, int* __restrict__ dev_err) {
+    // H, Hkv: query and key heads as they are rotated and normed, maps counted one by one; Hv: value heads.  Key heads that share
+    // a value head (the maps of a head) lie side by side in the cache's rows.
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
     const int slot = tok_slot[t];
     if (slot < 0) return;  // padding row (the whole CTA leaves: no barrier is missed)
+    const int maps = Hkv / Hv;
     const int pos = tok_pos[t];
     const float* row = proj + (size_t)t * ld;
     const int half = rot / 2;
@@ -94,6 +100,10 @@ qkv_rope_append_kernel(const float* __restrict__ proj, int ld, int q_off, int k_
     auto normed = [&](const float* head, const float* w, float inv, int c) -> float {
         return norm ? head[c] * inv * w[c] : head[c];
     };
+    auto key_at = [&](int blk, int h) -> ET* {
+        const int hv = maps == 1 ? h : h / maps;
+        return Kc + ((((size_t)blk * Hv + hv) * BT + (pos % BT)) * maps + (h - hv * maps)) * dk;
+    };
     auto rotated = [&](const float* head, const float* w, float inv, int c) -> float {
         const float x = normed(head, w, inv, c);
         if (c >= rot) return x;
@@ -121,7 +131,7 @@ qkv_rope_append_kernel(const float* __restrict__ proj, int ld, int q_off, int k_
             const bool isq = h < H;
             const float* head = isq ? row + q_off + h * dk : row + k_off + (h - H) * dk;
             const float* w = isq ? q_norm : k_norm;
-            ET* dst = isq ? q_out + (size_t)t * ldq + h * dk : Kc + (((size_t)blk * Hkv + (h - H)) * BT + (pos % BT)) * dk;
+            ET* dst = isq ? q_out + (size_t)t * ldq + h * dk : key_at(blk, h - H);
             float xa[4], xb[4];
             int ia[4], ib[4];
             float ss = 0.f;
@@ -153,9 +163,9 @@ qkv_rope_append_kernel(const float* __restrict__ proj, int ld, int q_off, int k_
             }
         }
         if (blk < 0) return;
-        for (int i = threadIdx.x; i < Hkv * dv; i += blockDim.x) {
+        for (int i = threadIdx.x; i < Hv * dv; i += blockDim.x) {
             const int h = i / dv, c = i - h * dv;
-            ElemIO<ET>::store(Vc + (((size_t)blk * Hkv + h) * BT + (pos % BT)) * dv + c, row[v_off + i]);
+            ElemIO<ET>::store(Vc + (((size_t)blk * Hv + h) * BT + (pos % BT)) * dv + c, row[v_off + i]);
         }
         return;
     }
@@ -201,7 +211,7 @@ qkv_rope_append_kernel(const float* __restrict__ proj, int ld, int q_off, int k_
             int ia, ib;
             float oa, ob;
             pair_of(row + k_off + h * dk, norm == 2 ? k_norm + h * dk : k_norm, norm ? inv_sm[H + h] : 1.f, u, ia, ib, oa, ob);
-            ET* dst = Kc + (((size_t)blk * Hkv + h) * BT + (pos % BT)) * dk;
+            ET* dst = key_at(blk, h);
             ElemIO<ET>::store(dst + ia, oa);
             ElemIO<ET>::store(dst + ib, ob);
         }
@@ -209,23 +219,24 @@ qkv_rope_append_kernel(const float* __restrict__ proj, int ld, int q_off, int k_
         for (int i = threadIdx.x; i < Hkv * dk; i += blockDim.x) {
             const int h = i / dk, c = i - h * dk;
             const float* w = norm == 2 ? k_norm + h * dk : k_norm;
-            ElemIO<ET>::store(Kc + (((size_t)blk * Hkv + h) * BT + (pos % BT)) * dk + c,
+            ElemIO<ET>::store(key_at(blk, h) + c,
                               rotated(row + k_off + h * dk, w, norm ? inv_sm[H + h] : 1.f, c));
         }
     }
-    for (int i = threadIdx.x; i < Hkv * dv; i += blockDim.x) {
+    for (int i = threadIdx.x; i < Hv * dv; i += blockDim.x) {
         const int h = i / dv, c = i - h * dv;
-        ElemIO<ET>::store(Vc + (((size_t)blk * Hkv + h) * BT + (pos % BT)) * dv + c, row[v_off + i]);
+        ElemIO<ET>::store(Vc + (((size_t)blk * Hv + h) * BT + (pos % BT)) * dv + c, row[v_off + i]);
     }
 }
 
-template <typename ET>
+template <typename ET, int MAPS>
 __global__ void __launch_bounds__(AW_WARPS * 32)
 attn_window_kernel(const ET* __restrict__ q_in, int ldq, const ET* __restrict__ Kc, const ET* __restrict__ Vc,
                    const int* __restrict__ block_table, int max_blocks, const int* __restrict__ tok_slot,
                    const int* __restrict__ tok_pos, ET* __restrict__ out, int ld_out, int H, int Hkv, int dk, int dv, int BT,
                    float scale, int window, float out_scale, float softcap, int keep_first, const float* __restrict__ sink,
-                   const float* __restrict__ gate, int ld_gate, const float* __restrict__ slopes, int* __restrict__ dev_err) {
+                   const float* __restrict__ gate, int ld_gate, const float* __restrict__ slopes, float map_factor, float head_eps,
+                   int* __restrict__ dev_err) {
     pdl_wait();
     pdl_launch_dependents();
     extern __shared__ float q_sm[];  // [AW_WARPS][dk]
@@ -237,14 +248,6 @@ attn_window_kernel(const ET* __restrict__ q_in, int ldq, const ET* __restrict__ 
     const int pos = tok_pos[t];
     const int hk = h / (H / Hkv);
     float* q = q_sm + warp * dk;
-    const ET* qsrc = q_in + (size_t)t * ldq + (size_t)h * dk;
-    for (int i = lane; i < dk; i += 32) q[i] = ElemIO<ET>::load(qsrc + i) * scale;
-    __syncwarp();
-
-    float acc[AW_MAX / 32];
-#pragma unroll
-    for (int i = 0; i < AW_MAX / 32; ++i) acc[i] = 0.f;
-    float m = -INFINITY, l = 0.f;
     const float slope = slopes != nullptr ? slopes[h] : 0.f;     // what a step of distance takes off a score
     const int first = (window > 0) ? max(0, pos - window + 1) : 0;
     const int* table = block_table + (size_t)slot * max_blocks;
@@ -253,56 +256,85 @@ attn_window_kernel(const ET* __restrict__ q_in, int ldq, const ET* __restrict__ 
     // the keys kept whatever the window (positions below keep_first that the window no longer reaches), then the window
     const int n_kept = (window > 0 && keep_first > 0) ? min(keep_first, first) : 0;
     const int kept_end = ((n_kept + 31) / 32) * 32, win_begin = (first / 32) * 32;
-    for (int k0 = n_kept > 0 ? 0 : win_begin; k0 <= pos; k0 += 32) {
-        if (k0 >= kept_end && k0 < win_begin) { k0 = win_begin - 32; continue; }   // (the chunks between the two ranges)
-        const int blk = table[k0 / BT];
-        if (blk < 0) { lost = true; break; }
-        const size_t kbase = (((size_t)blk * Hkv + hk) * BT + (k0 % BT)) * dk;
-        const size_t vbase = (((size_t)blk * Hkv + hk) * BT + (k0 % BT)) * dv;
-        const int key = k0 + lane;
-        const bool valid = (key >= first || key < n_kept) && key <= pos;
-        float s = -INFINITY;
-        if (valid) {
-            const ET* krow = Kc + kbase + (size_t)lane * dk;
-            float dot = 0.f;
-            for (int c = 0; c < dk; ++c) dot = fmaf(q[c], ElemIO<ET>::load(krow + c), dot);
-            s = softcap > 0.f ? softcap * tanhf(dot / softcap) : dot;
-            s -= slope * (float)(pos - key);
-        }
-        const float m_new = fmaxf(m, warp_max(s));      // at least one key of the chunk is valid
-        const float p = valid ? expf(s - m_new) : 0.f;
-        const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
-        l = l * corr + warp_sum(p);
+    float first_map[MAPS == 2 ? AW_MAX / 32 : 1];        // the first map's finished result
+#pragma unroll 1
+    for (int map = 0; map < MAPS; ++map) {
+        const ET* qsrc = q_in + (size_t)t * ldq + ((size_t)h * MAPS + map) * dk;
+        __syncwarp();
+        for (int i = lane; i < dk; i += 32) q[i] = ElemIO<ET>::load(qsrc + i) * scale;
+        __syncwarp();
+
+        float acc[AW_MAX / 32];
 #pragma unroll
-        for (int i = 0; i < AW_MAX / 32; ++i) acc[i] *= corr;
-        const int n_here = min(32, pos - k0 + 1);
-        for (int j = 0; j < n_here; ++j) {
-            const float pj = __shfl_sync(0xffffffffu, p, j);
-            if (pj == 0.f) continue;  // uniform across the warp
-            const ET* vrow = Vc + vbase + (size_t)j * dv;
-#pragma unroll
-            for (int i = 0; i < AW_MAX / 32; ++i) {
-                const int c = i * 32 + lane;
-                if (c < dv) acc[i] = fmaf(pj, ElemIO<ET>::load(vrow + c), acc[i]);
+        for (int i = 0; i < AW_MAX / 32; ++i) acc[i] = 0.f;
+        float m = -INFINITY, l = 0.f;
+        for (int k0 = n_kept > 0 ? 0 : win_begin; k0 <= pos; k0 += 32) {
+            if (k0 >= kept_end && k0 < win_begin) { k0 = win_begin - 32; continue; }   // (the chunks between the two ranges)
+            const int blk = table[k0 / BT];
+            if (blk < 0) { lost = true; break; }
+            const size_t kbase = (((size_t)blk * Hkv + hk) * BT + (k0 % BT)) * (MAPS * dk) + map * dk;
+            const size_t vbase = (((size_t)blk * Hkv + hk) * BT + (k0 % BT)) * dv;
+            const int key = k0 + lane;
+            const bool valid = (key >= first || key < n_kept) && key <= pos;
+            float s = -INFINITY;
+            if (valid) {
+                const ET* krow = Kc + kbase + (size_t)lane * (MAPS * dk);
+                float dot = 0.f;
+                for (int c = 0; c < dk; ++c) dot = fmaf(q[c], ElemIO<ET>::load(krow + c), dot);
+                s = softcap > 0.f ? softcap * tanhf(dot / softcap) : dot;
+                s -= slope * (float)(pos - key);
             }
+            const float m_new = fmaxf(m, warp_max(s));      // at least one key of the chunk is valid
+            const float p = valid ? expf(s - m_new) : 0.f;
+            const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
+            l = l * corr + warp_sum(p);
+#pragma unroll
+            for (int i = 0; i < AW_MAX / 32; ++i) acc[i] *= corr;
+            const int n_here = min(32, pos - k0 + 1);
+            for (int j = 0; j < n_here; ++j) {
+                const float pj = __shfl_sync(0xffffffffu, p, j);
+                if (pj == 0.f) continue;  // uniform across the warp
+                const ET* vrow = Vc + vbase + (size_t)j * dv;
+#pragma unroll
+                for (int i = 0; i < AW_MAX / 32; ++i) {
+                    const int c = i * 32 + lane;
+                    if (c < dv) acc[i] = fmaf(pj, ElemIO<ET>::load(vrow + c), acc[i]);
+                }
+            }
+            m = m_new;
         }
-        m = m_new;
-    }
-    if (lost && lane == 0) atomicOr(dev_err, VLRF_DEVERR_NO_BLOCK);
-    if (sink != nullptr) {                               // exp(sink) joins the denominator: no key, no value
-        const float sk = sink[h], m_new = fmaxf(m, sk);
-        const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
-        l = l * corr + expf(sk - m_new);
+        if (MAPS == 2) {
+            const float inv = (l > 0.f) ? 1.f / l : 0.f;
+            if (map == 0) {
 #pragma unroll
-        for (int i = 0; i < AW_MAX / 32; ++i) acc[i] *= corr;
-    }
-    float inv = (l > 0.f) ? out_scale / l : 0.f;
-    if (gate != nullptr) inv *= sigmoid_f(gate[(size_t)t * ld_gate + h]);      // a gate per head on the head's result
-    ET* dst = out + (size_t)t * ld_out + (size_t)h * dv;
+                for (int i = 0; i < AW_MAX / 32; ++i) first_map[MAPS == 2 ? i : 0] = acc[i] * inv;
+                continue;
+            }
+            float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < AW_MAX / 32; ++i) {
-        const int c = i * 32 + lane;
-        if (c < dv) ElemIO<ET>::store(dst + c, acc[i] * inv);
+            for (int i = 0; i < AW_MAX / 32; ++i) {          // (columns behind dv are zero)
+                acc[i] = first_map[MAPS == 2 ? i : 0] - map_factor * (acc[i] * inv);
+                ss = fmaf(acc[i], acc[i], ss);
+            }
+            m = 0.f;                                         // what follows takes acc as it is, divided by the head's root mean square
+            l = sqrtf(warp_sum(ss) / (float)dv + head_eps);
+        }
+        if (lost && lane == 0) atomicOr(dev_err, VLRF_DEVERR_NO_BLOCK);
+        if (sink != nullptr) {                               // exp(sink) joins the denominator: no key, no value
+            const float sk = sink[h], m_new = fmaxf(m, sk);
+            const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
+            l = l * corr + expf(sk - m_new);
+#pragma unroll
+            for (int i = 0; i < AW_MAX / 32; ++i) acc[i] *= corr;
+        }
+        float inv = (l > 0.f) ? out_scale / l : 0.f;
+        if (gate != nullptr) inv *= sigmoid_f(gate[(size_t)t * ld_gate + h]);      // a gate per head on the head's result
+        ET* dst = out + (size_t)t * ld_out + (size_t)h * dv;
+#pragma unroll
+        for (int i = 0; i < AW_MAX / 32; ++i) {
+            const int c = i * 32 + lane;
+            if (c < dv) ElemIO<ET>::store(dst + c, acc[i] * inv);
+        }
     }
 }
 }  // namespace
@@ -310,13 +342,17 @@ attn_window_kernel(const ET* __restrict__ q_in, int ldq, const ET* __restrict__ 
 extern "C" int vlrf_qkv_norm_rope_append(const float* proj, int ld, int q_off, int k_off, int v_off, const float* freq, int rot,
                                          void* q_out, int ldq, void* Kc, void* Vc, int dtype, const int* block_table, int max_blocks,
                                          const int* tok_slot, const int* tok_pos, int T, int H, int Hkv, int dk, int dv, int BT,
-                                         int write_cache, int norm, const float* q_norm, const float* k_norm, float eps, int pairing,
+                                         int maps, int write_cache, int norm, const float* q_norm, const float* k_norm, float eps, int pairing,
                                          float magnitude, int* dev_err, cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && H > 0 && Hkv > 0 && dk > 0 && dv > 0 && BT > 0 && max_blocks > 0, "qkv_rope_append: bad sizes");
+    VLRF_REQUIRE(maps == 1 || maps == 2, "qkv_rope_append: a head has one map or two, not %d", maps);
+    const int Hv = Hkv;
+    H *= maps;
+    Hkv *= maps;
     VLRF_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dk, "qkv_rope_append: %d rotated entries of a head of %d", rot, dk);
     VLRF_REQUIRE(rot == 0 || freq != nullptr, "qkv_rope_append: a rotation needs its frequencies");
     VLRF_REQUIRE(q_off >= 0 && q_off + H * dk <= ld && ldq >= H * dk, "qkv_rope_append: columns lie outside the row");
-    VLRF_REQUIRE(!write_cache || (k_off >= 0 && v_off >= 0 && k_off + Hkv * dk <= ld && v_off + Hkv * dv <= ld && Kc != nullptr && Vc != nullptr),
+    VLRF_REQUIRE(!write_cache || (k_off >= 0 && v_off >= 0 && k_off + Hkv * dk <= ld && v_off + Hv * dv <= ld && Kc != nullptr && Vc != nullptr),
                  "qkv_rope_append: key or value columns lie outside the row");
     VLRF_REQUIRE(norm >= 0 && norm <= 2 && (norm == 0 || (q_norm != nullptr && (k_norm != nullptr || !write_cache) && eps > 0.f)),
                  "qkv_rope_append: a norm of queries and keys needs its weights and a positive eps");
@@ -327,12 +363,12 @@ extern "C" int vlrf_qkv_norm_rope_append(const float* proj, int ld, int q_off, i
     VLRF_REQUIRE(smem <= 48 * 1024, "qkv_rope_append: %d heads are more than the kernel's shared memory takes", H + Hkv);
     if (dtype == VLRF_F32)
         launch_chained(qkv_rope_append_kernel<float>, dim3(T), dim3(128), smem, stream, proj, ld, q_off, k_off, v_off, freq, rot,
-                       (float*)q_out, ldq, (float*)Kc, (float*)Vc, block_table, max_blocks, tok_slot, tok_pos, H, Hkv, dk, dv, BT,
+                       (float*)q_out, ldq, (float*)Kc, (float*)Vc, block_table, max_blocks, tok_slot, tok_pos, H, Hkv, Hv, dk, dv, BT,
                        write_cache, norm, q_norm, k_norm, eps, pairing, magnitude, dev_err);
     else if (dtype == VLRF_BF16)
         launch_chained(qkv_rope_append_kernel<__nv_bfloat16>, dim3(T), dim3(128), smem, stream, proj, ld, q_off, k_off, v_off, freq,
                        rot, (__nv_bfloat16*)q_out, ldq, (__nv_bfloat16*)Kc, (__nv_bfloat16*)Vc, block_table, max_blocks, tok_slot,
-                       tok_pos, H, Hkv, dk, dv, BT, write_cache, norm, q_norm, k_norm, eps, pairing, magnitude, dev_err);
+                       tok_pos, H, Hkv, Hv, dk, dv, BT, write_cache, norm, q_norm, k_norm, eps, pairing, magnitude, dev_err);
     else
         return vlrf_fail(VLRF_ERR_INVALID_ARG, "qkv_rope_append: unknown dtype %d", dtype);
     return vlrf_check_launch("qkv_rope_append");
@@ -344,36 +380,35 @@ extern "C" int vlrf_qkv_rope_append(const float* proj, int ld, int q_off, int k_
                                     int write_cache, int* dev_err, cudaStream_t stream) {
     VLRF_REQUIRE(k_off + Hkv * dk <= ld && v_off + Hkv * dv <= ld, "qkv_rope_append: columns lie outside the row");
     return vlrf_qkv_norm_rope_append(proj, ld, q_off, k_off, v_off, freq, rot, q_out, ldq, Kc, Vc, dtype, block_table, max_blocks,
-                                     tok_slot, tok_pos, T, H, Hkv, dk, dv, BT, write_cache, 0, nullptr, nullptr, 0.f, 0, 1.f, dev_err,
+                                     tok_slot, tok_pos, T, H, Hkv, dk, dv, BT, 1, write_cache, 0, nullptr, nullptr, 0.f, 0, 1.f, dev_err,
                                      stream);
 }
 
 extern "C" int vlrf_attn_window_ex(const void* q, int dtype, int ldq, const void* Kc, const void* Vc, const int* block_table,
                                    int max_blocks, const int* tok_slot, const int* tok_pos, void* out, int ld_out, int T, int H,
                                    int Hkv, int dk, int dv, int BT, float scale, int window, float out_scale, float softcap,
-                                   int keep_first, const float* sink, const float* gate, int ld_gate, const float* slopes, int* dev_err,
-                                   cudaStream_t stream) {
+                                   int keep_first, const float* sink, const float* gate, int ld_gate, const float* slopes, int maps,
+                                   float map_factor, float head_eps, int* dev_err, cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && H > 0 && Hkv > 0 && max_blocks > 0, "attn_window: bad sizes");
     VLRF_REQUIRE(H % Hkv == 0, "attn_window: %d heads cannot share %d key/value heads", H, Hkv);
     VLRF_REQUIRE(dk > 0 && dk <= AW_MAX && dv > 0 && dv <= AW_MAX, "attn_window: head sizes %d and %d are not in 1…%d", dk, dv, AW_MAX);
     VLRF_REQUIRE(BT % 32 == 0, "attn_window: cache blocks of %d tokens are not a multiple of 32", BT);
     VLRF_REQUIRE(window >= 0 && keep_first >= 0 && softcap >= 0.f, "attn_window: negative window, kept tokens or cap");
-    VLRF_REQUIRE(ldq >= H * dk && ld_out >= H * dv && (gate == nullptr || ld_gate >= H), "attn_window: leading sizes are smaller than the rows");
+    VLRF_REQUIRE(maps == 1 || (maps == 2 && sink == nullptr && gate == nullptr && head_eps > 0.f),
+                 "attn_window: one map, or two without sinks and gates and with a positive eps");
+    VLRF_REQUIRE(ldq >= H * maps * dk && ld_out >= H * dv && (gate == nullptr || ld_gate >= H), "attn_window: leading sizes are smaller than the rows");
     VLRF_REQUIRE(dev_err != nullptr, "attn_window: needs the device error word");
     if (T == 0) return VLRF_OK;
     dim3 grid(T, (H + AW_WARPS - 1) / AW_WARPS);
     const size_t smem = (size_t)AW_WARPS * dk * sizeof(float);
-    if (dtype == VLRF_F32)
-        launch_chained(attn_window_kernel<float>, grid, dim3(AW_WARPS * 32), smem, stream, (const float*)q, ldq, (const float*)Kc,
-                       (const float*)Vc, block_table, max_blocks, tok_slot, tok_pos, (float*)out, ld_out, H, Hkv, dk, dv, BT, scale,
-                       window, out_scale, softcap, keep_first, sink, gate, ld_gate, slopes, dev_err);
-    else if (dtype == VLRF_BF16)
-        launch_chained(attn_window_kernel<__nv_bfloat16>, grid, dim3(AW_WARPS * 32), smem, stream, (const __nv_bfloat16*)q, ldq,
-                       (const __nv_bfloat16*)Kc, (const __nv_bfloat16*)Vc, block_table, max_blocks, tok_slot, tok_pos,
-                       (__nv_bfloat16*)out, ld_out, H, Hkv, dk, dv, BT, scale, window, out_scale, softcap, keep_first, sink, gate, ld_gate,
-                       slopes, dev_err);
+#define GO(ET, MAPS) launch_chained(attn_window_kernel<ET, MAPS>, grid, dim3(AW_WARPS * 32), smem, stream, (const ET*)q, ldq, (const ET*)Kc, \
+        (const ET*)Vc, block_table, max_blocks, tok_slot, tok_pos, (ET*)out, ld_out, H, Hkv, dk, dv, BT, scale, window, out_scale, softcap, \
+        keep_first, sink, gate, ld_gate, slopes, map_factor, head_eps, dev_err)
+    if (dtype == VLRF_F32) { if (maps == 2) GO(float, 2); else GO(float, 1); }
+    else if (dtype == VLRF_BF16) { if (maps == 2) GO(__nv_bfloat16, 2); else GO(__nv_bfloat16, 1); }
     else
         return vlrf_fail(VLRF_ERR_INVALID_ARG, "attn_window: unknown dtype %d", dtype);
+#undef GO
     return vlrf_check_launch("attn_window");
 }
 
@@ -382,5 +417,5 @@ extern "C" int vlrf_attn_window(const void* q, int dtype, int ldq, const void* K
                                 int Hkv, int dk, int dv, int BT, float scale, int window, float out_scale, int* dev_err,
                                 cudaStream_t stream) {
     return vlrf_attn_window_ex(q, dtype, ldq, Kc, Vc, block_table, max_blocks, tok_slot, tok_pos, out, ld_out, T, H, Hkv, dk, dv, BT,
-                               scale, window, out_scale, 0.f, 0, nullptr, nullptr, 0, nullptr, dev_err, stream);
+                               scale, window, out_scale, 0.f, 0, nullptr, nullptr, 0, nullptr, 1, 0.f, 0.f, dev_err, stream);
 }

@@ -569,12 +569,12 @@ extern "C" int vlrf_gemm_tcgen05_groups_takes(int rows, int G, int N, int K, int
 
 // offsets != null: rows offsets[g] … offsets[g+1]−1 of X [rows][K] times W[g]ᵀ into the same rows of Y [rows][N]
 // (x_gs = y_gs = 0).  offsets == null: every group (head) multiplies all rows, reading X at column g·x_gs and writing Y at
-// column g·y_gs.  W [G][N][K]; X and W bfloat16, Y bfloat16 or float32; an activation (VLRF_ACT_NONE, _GELU_TANH or _RELU2) on
+// column g·y_gs.  W [G][N][K]; X and W bfloat16, Y bfloat16 or float32; an activation (VLRF_ACT_NONE, _GELU_TANH, _GELU_ERF or _RELU2) on
 // the result, no bias or residual.
 extern "C" int vlrf_gemm_tcgen05_groups(const void* X, int ldx, int x_gs, const void* W, void* Y, int ldy, int y_gs,
                                         const int* offsets, int G, int rows, int N, int K, int out_dtype, int act, int* dev_err,
                                         cudaStream_t stream) {
-    VLRF_REQUIRE(act == VLRF_ACT_NONE || act == VLRF_ACT_GELU_TANH || act == VLRF_ACT_RELU2, "gemm_tcgen05_groups: activation %d is not taken", act);
+    VLRF_REQUIRE(act == VLRF_ACT_NONE || act == VLRF_ACT_GELU_TANH || act == VLRF_ACT_GELU_ERF || act == VLRF_ACT_RELU2, "gemm_tcgen05_groups: activation %d is not taken", act);
     VLRF_REQUIRE(vlrf_gemm_tcgen05_groups_takes(rows, G, N, K, ldx, x_gs, ldy, y_gs, offsets != nullptr),
                  "gemm_tcgen05_groups: does not take rows=%d G=%d N=%d K=%d ldx=%d x_gs=%d ldy=%d y_gs=%d", rows, G, N, K, ldx, x_gs, ldy, y_gs);
     VLRF_REQUIRE(dev_err != nullptr && (out_dtype == VLRF_BF16 || out_dtype == VLRF_F32), "gemm_tcgen05_groups: bad arguments");

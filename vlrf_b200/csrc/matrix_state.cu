@@ -9,6 +9,10 @@
 //   kind 2, stabilized   m' = max(f + m, i),  S ← exp(f + m − m') S + exp(i − m') k vᵀ,  n ← the same with k alone
 //                        with log gates i = c tanh(s0 / c), f = log sigmoid(c tanh(s1 / c)) per head; leaves Sᵀ q in y,
 //                        and n · q and exp(−m') in `den` (what divides one by the other stands with the kernel that reads them)
+//   kind 3, fixed        S ← a S + k vᵀ,                                              o = Sᵀ q
+//                        a: one number per head, the same for every token (`decay` [H])
+// In kind 3 q, k and v may be raw projections that go through x · sigmoid(x) here (`input_act`): a thread applies it to what it has
+// copied into shared memory itself, ahead of the barrier that hands the batch over.
 // Every o and n · q is multiplied by q_scale.  Everything here is float32: gates, exponentials, sums, state.
 //
 // What a sequence keeps lies in one float32 row per (layer, slot), twice, `state` [slots][2][state_row]: per head the
@@ -32,7 +36,10 @@
 namespace {
 constexpr int MS_WARPS = 4;
 constexpr int MS_MAX_BATCH = 32;       // a lane per token works out a batch's gates
-constexpr int MS_DECAYED = 0, MS_DELTA = 1, MS_STABILIZED = 2;
+constexpr int MS_DECAYED = 0, MS_DELTA = 1, MS_STABILIZED = 2, MS_FIXED = 3;
+// kinds with a decay per head, key channel and token, kinds with two more numbers a token
+constexpr bool ms_decays(int mode) { return mode == MS_DECAYED || mode == MS_DELTA; }
+constexpr bool ms_numbers(int mode) { return mode == MS_DELTA || mode == MS_STABILIZED; }
 
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pk2(float lo, float hi) { f32x2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi)); return r; }
@@ -58,7 +65,7 @@ struct MatrixStateArgs {
     float* y;
     int ldy;
     float* den;
-    int H, G, K, V, col_blocks, batch, vec_rows, vec_v, vec_state, max_new, warps;
+    int H, G, K, V, col_blocks, batch, vec_rows, vec_v, vec_state, max_new, warps, silu;
 };
 
 // log sigmoid(x), stable at both ends
@@ -116,7 +123,7 @@ __device__ __forceinline__ void store_state(const f32x2 (&S)[NC][NR / 2], float*
 template <int NR> struct TokenRows { ulonglong2 k[NR / 4], q[NR / 4], d[NR / 4]; };
 
 // One token: S moves on, and p gets the lane's share (its rows) of the read-outs.  a, b: kind 1 (b, k · q), kind 2 (what stays, what
-// comes); v: the columns' values.
+// comes), kind 3 (what stays); v: the columns' values.
 template <int MODE, int NR, int NC>
 __device__ __forceinline__ void advance(f32x2 (&S)[NC][NR / 2], const TokenRows<NR>& X, const float (&v)[NC], float a, float b, int r, float (&p)[NC]) {
     constexpr int NV = NR / 4, NP = NR / 2;
@@ -186,7 +193,7 @@ template <int MODE, int NR, int NC>
 __global__ void __launch_bounds__(MS_WARPS * 32, 1)
 matrix_state_scan_kernel(const MatrixStateArgs A) {
     constexpr int KP = 8 * NR, NV = NR / 4;
-    constexpr bool DECAY = MODE != MS_STABILIZED;
+    constexpr bool DECAY = ms_decays(MODE);
     constexpr int ROWS = DECAY ? 3 : 2;             // k, q (, decay)
     constexpr bool AHEAD = NR <= 16;                // a token's rows are fetched from shared memory while the one before is worked on
     pdl_wait();
@@ -264,6 +271,40 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
             }
         }
     };
+    // x · sigmoid(x) of this thread's own copies of a batch (the same places as in fetch)
+    auto activate = [&](int nb, int st) {
+        float* ks = ms_sm + st * stage_floats;
+        float* qs = ks + B * KP;
+        float* vs = ks + ROWS * B * KP;
+        auto four = [](float* p) {
+            float4 x = *reinterpret_cast<float4*>(p);
+            x.x = silu_f(x.x); x.y = silu_f(x.y); x.z = silu_f(x.z); x.w = silu_f(x.w);
+            *reinterpret_cast<float4*>(p) = x;
+        };
+        if (whole_rows) {
+            for (int ii = ii0; ii < nb; ii += ii_step) { four(ks + ii * KP + q_col); four(qs + ii * KP + q_col); }
+        } else if (A.vec_rows) {
+            const int q4 = K / 4;
+            for (int i = threadIdx.x; i < nb * q4; i += n_thr) {
+                const int ii = i / q4, cc = (i - ii * q4) * 4;
+                four(ks + ii * KP + cc);
+                four(qs + ii * KP + cc);
+            }
+        } else {
+            for (int i = threadIdx.x; i < nb * K; i += n_thr) {
+                const int ii = i / K, at = ii * KP + i - ii * K;
+                ks[at] = silu_f(ks[at]);
+                qs[at] = silu_f(qs[at]);
+            }
+        }
+        if (A.vec_v) {
+            if (pb * CW + v_col < V)
+                for (int ii = v0; ii < nb; ii += v_step) four(vs + ii * CW + v_col);
+        } else {
+            for (int i = threadIdx.x; i < nb * CW; i += n_thr)
+                if (pb * CW + i % CW < V) vs[i] = silu_f(vs[i]);
+        }
+    };
     fetch(0, 0);
     asm volatile("cp.async.commit_group;" ::: "memory");
     f32x2 S[NC][NR / 2];
@@ -271,10 +312,11 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
     // numbers of the batch's tokens: lane ii asks for token ii's, a batch ahead
     float m_run = 0.f, raw0 = 0.f, raw1 = 0.f;
     if (MODE == MS_STABILIZED && active) m_run = A.state[copy_in + max_at + col0];
+    const float fixed = MODE == MS_FIXED ? A.decay[h] : 0.f;
     auto ask = [&](int i0) {
         const int ii = i0 + lane;
         raw0 = raw1 = 0.f;
-        if (MODE != MS_DECAYED && lane < B && ii < n) {
+        if (ms_numbers(MODE) && lane < B && ii < n) {
             raw0 = A.s0[(size_t)(start + ii) * A.ld_s0 + h];
             raw1 = A.s1[(size_t)(start + ii) * A.ld_s1 + (MODE == MS_DELTA ? g : h)];
         }
@@ -283,6 +325,7 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
     for (int i0 = 0, st = 0; i0 < n; i0 += B, st ^= 1) {
         const int nb = min(B, n - i0);
         asm volatile("cp.async.wait_group 0;" ::: "memory");
+        if (MODE == MS_FIXED && A.silu) activate(nb, st);
         __syncthreads();                            // the batch lies in shared memory, and nobody reads the other stage any more
         if (i0 + B < n) fetch(i0 + B, st ^ 1);
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -334,8 +377,8 @@ matrix_state_scan_kernel(const MatrixStateArgs A) {
                     float v[NC];
 #pragma unroll
                     for (int e = 0; e < NC; ++e) v[e] = vs[ii * CW + e];     // (columns that do not exist: anything, it goes nowhere)
-                    float2 ab = make_float2(0.f, 0.f);
-                    if (MODE != MS_DECAYED) ab = *reinterpret_cast<const float2*>(scal + 2 * ii);
+                    float2 ab = make_float2(fixed, 0.f);
+                    if (ms_numbers(MODE)) ab = *reinterpret_cast<const float2*>(scal + 2 * ii);
                     advance<MODE, NR, NC>(S, X[AHEAD ? (t & 1) : 0], v, ab.x, ab.y, r, p[t]);
                 } else {
 #pragma unroll
@@ -392,7 +435,7 @@ template <int MODE, int NR, int NC>
 __global__ void __launch_bounds__(MS_WARPS * 32)
 matrix_state_step_kernel(const MatrixStateArgs A) {
     constexpr int NV = NR / 4;
-    constexpr bool DECAY = MODE != MS_STABILIZED;
+    constexpr bool DECAY = ms_decays(MODE);
     pdl_wait();
     pdl_launch_dependents();
     const int s = blockIdx.y, slot = A.seq_slot[s];
@@ -429,11 +472,25 @@ matrix_state_step_kernel(const MatrixStateArgs A) {
     row_of(A.k + t * A.ldk + (size_t)g * K, X.k);
     row_of(A.q + t * A.ldq + (size_t)g * K, X.q);
     if (DECAY) row_of(A.decay + t * A.ld_decay + (size_t)h * K, X.d);
+    const bool act = MODE == MS_FIXED && A.silu;
+    if (act) {
+        auto both = [](unsigned long long& x) {
+            float lo, hi;
+            asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(x));
+            x = pk2(silu_f(lo), silu_f(hi));
+        };
+#pragma unroll
+        for (int j = 0; j < NV; ++j) { both(X.k[j].x); both(X.k[j].y); both(X.q[j].x); both(X.q[j].y); }
+    }
     float v[NC], p[NC];
 #pragma unroll
     for (int e = 0; e < NC; ++e)
         v[e] = my_col + e < V ? A.v[t * A.ldv + (size_t)h * V + my_col + e] : (MODE == MS_STABILIZED && my_col + e == V) ? 1.f : 0.f;
-    float a = 0.f, b = 0.f, m_new = 0.f;
+    if (act) {
+#pragma unroll
+        for (int e = 0; e < NC; ++e) v[e] = silu_f(v[e]);
+    }
+    float a = MODE == MS_FIXED ? A.decay[h] : 0.f, b = 0.f, m_new = 0.f;
     if (MODE == MS_DELTA) {
         a = sigmoid_f(A.s0[t * A.ld_s0 + h]);
         b = A.s1[t * A.ld_s1 + g];
@@ -461,7 +518,7 @@ matrix_state_step_kernel(const MatrixStateArgs A) {
 }
 
 template <int MODE, int NR, int NC> int launch_scan(MatrixStateArgs& A, int n_seqs, cudaStream_t stream) {
-    constexpr int KP = 8 * NR, ROWS = MODE == MS_STABILIZED ? 2 : 3;
+    constexpr int KP = 8 * NR, ROWS = ms_decays(MODE) ? 3 : 2;
     const int VT = A.V + (MODE == MS_STABILIZED ? 1 : 0), chunks = (VT + 4 * NC - 1) / (4 * NC);
     if (A.max_new == 1) {
         A.col_blocks = chunks;
@@ -512,13 +569,15 @@ extern "C" int vlrf_matrix_state_scan(int kind, const float* q, int ldq, const f
                                       const float* decay, int ld_decay, const float* s0, int ld_s0, const float* s1, int ld_s1,
                                       float q_scale, float cap, float* state, int state_row, const int* seq_slot,
                                       const int* seq_start, const int* seq_pos0, float* y, int ldy, float* den, int n_seqs, int max_new,
-                                      int H, int G, int K, int V, cudaStream_t stream) {
-    VLRF_REQUIRE(kind >= MS_DECAYED && kind <= MS_STABILIZED, "matrix_state_scan: unknown kind %d", kind);
+                                      int H, int G, int K, int V, int input_act, cudaStream_t stream) {
+    VLRF_REQUIRE(kind >= MS_DECAYED && kind <= MS_FIXED, "matrix_state_scan: unknown kind %d", kind);
     VLRF_REQUIRE(n_seqs >= 0 && max_new >= 0 && H > 0 && G > 0 && K > 0 && V > 0 && H % G == 0, "matrix_state_scan: bad sizes (heads %d/%d, state %d by %d)", H, G, K, V);
     VLRF_REQUIRE(K <= 512 && V <= 4096 && n_seqs <= 65535, "matrix_state_scan: a state of %d rows by %d columns is above 512 by 4096, or too many sequences", K, V);
     VLRF_REQUIRE(ldq >= G * K && ldk >= G * K && ldv >= H * V && ldy >= H * V, "matrix_state_scan: columns lie outside the rows");
-    VLRF_REQUIRE(kind == MS_STABILIZED || (decay != nullptr && ld_decay >= H * K), "matrix_state_scan: this kind needs a decay per head and key channel");
-    VLRF_REQUIRE(kind == MS_DECAYED || (s0 != nullptr && s1 != nullptr && ld_s0 >= H && ld_s1 >= (kind == MS_DELTA ? G : H)), "matrix_state_scan: this kind needs two numbers a token");
+    VLRF_REQUIRE(input_act == VLRF_ACT_NONE || (input_act == VLRF_ACT_SILU && kind == MS_FIXED), "matrix_state_scan: input activation %d is not taken by kind %d", input_act, kind);
+    VLRF_REQUIRE(kind != MS_FIXED || decay != nullptr, "matrix_state_scan: this kind needs a decay per head");
+    VLRF_REQUIRE(!ms_decays(kind) || (decay != nullptr && ld_decay >= H * K), "matrix_state_scan: this kind needs a decay per head and key channel");
+    VLRF_REQUIRE(!ms_numbers(kind) || (s0 != nullptr && s1 != nullptr && ld_s0 >= H && ld_s1 >= (kind == MS_DELTA ? G : H)), "matrix_state_scan: this kind needs two numbers a token");
     VLRF_REQUIRE(kind != MS_STABILIZED || (den != nullptr && cap > 0.f), "matrix_state_scan: this kind needs a place for the denominators and a positive cap");
     const long long need = kind == MS_STABILIZED ? (long long)H * (V + 1) * (K + 1) : (long long)H * V * K;
     VLRF_REQUIRE(need <= state_row, "matrix_state_scan: the state row of %d numbers is shorter than %lld", state_row, need);
@@ -529,9 +588,9 @@ extern "C" int vlrf_matrix_state_scan(int kind, const float* q, int ldq, const f
     A.q_scale = q_scale; A.cap = cap; A.state = state; A.state_row = state_row;
     A.seq_slot = seq_slot; A.seq_start = seq_start; A.seq_pos0 = seq_pos0;
     A.y = y; A.ldy = ldy; A.den = den; A.H = H; A.G = G; A.K = K; A.V = V; A.col_blocks = 1;
-    A.max_new = max_new; A.warps = ms_forced_warps ? ms_forced_warps : 4;
+    A.max_new = max_new; A.silu = input_act == VLRF_ACT_SILU; A.warps = ms_forced_warps ? ms_forced_warps : 4;
     A.batch = max_new < MS_MAX_BATCH ? max_new : MS_MAX_BATCH;
-    A.vec_rows = K % 4 == 0 && on16(q) && on16(k) && ldq % 4 == 0 && ldk % 4 == 0 && (decay == nullptr || (on16(decay) && ld_decay % 4 == 0));
+    A.vec_rows = K % 4 == 0 && on16(q) && on16(k) && ldq % 4 == 0 && ldk % 4 == 0 && (!ms_decays(kind) || (on16(decay) && ld_decay % 4 == 0));
     A.vec_v = V % 4 == 0 && on16(v) && ldv % 4 == 0;
     A.vec_state = K % 4 == 0 && on16(state) && state_row % 4 == 0;
     // columns a lane (measured): single tokens 2; prompts 1 where the step's columns are fewer than warps for every scheduler of
@@ -545,6 +604,7 @@ extern "C" int vlrf_matrix_state_scan(int kind, const float* q, int ldq, const f
     switch (kind) {
         case MS_DECAYED: return pick_scan<MS_DECAYED>(A, nc, n_seqs, stream);
         case MS_DELTA: return pick_scan<MS_DELTA>(A, nc, n_seqs, stream);
+        case MS_FIXED: return pick_scan<MS_FIXED>(A, nc, n_seqs, stream);
         default: return pick_scan<MS_STABILIZED>(A, nc, n_seqs, stream);
     }
 }

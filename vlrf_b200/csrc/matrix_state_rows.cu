@@ -13,7 +13,8 @@
 //   Two such products, each with its own rows, weights and f, run in one launch.
 // head_rows: out[t][h·V + i] = factor · o / sqrt(mean(o²) + eps) · w · act(gate[t][h·V + i]) with the mean over the head's V
 //   numbers; o = y, or y / (max(|n·q|, floor) + 1e-6) where `den` gives (n·q, floor) per token and head; w one vector of V
-//   numbers for all heads or of H·V numbers; act sigmoid(z) or z · sigmoid(z); rounded to the activation dtype.
+//   numbers for all heads or of H·V numbers; act sigmoid(z) or z · sigmoid(z); rounded to the activation dtype.  A warp per token
+//   and head, or, where heads are wide (all heads of a mixer normed as one row, H = 1), a CTA.
 // norm_pair_add: x[t] += factor · (RMSnorm(a[t]) · wa + RMSnorm(b[t]) · wb), float32; the rows fit registers.
 #include "common.cuh"
 #include <type_traits>
@@ -418,6 +419,63 @@ head_rows_kernel(const float* __restrict__ y, int ldy, const float* __restrict__
     }
 }
 
+// A CTA per (token, head) for wide heads.  NV: quads of columns a thread holds in registers (rows on 16-byte boundaries, V a
+// multiple of 4 up to 1024·NV); 0: any sizes, a column at a time.
+template <typename OT, int NV>
+__global__ void __launch_bounds__(256)
+head_rows_wide_kernel(const float* __restrict__ y, int ldy, const float* __restrict__ den, const float* __restrict__ w, int w_per_head,
+                      const float* __restrict__ gate, int ld_gate, int act, OT* __restrict__ out, int ld_out, int H, int V, float eps, float factor) {
+    pdl_wait();
+    pdl_launch_dependents();
+    __shared__ float red[8];
+    const int t = blockIdx.x / H, h = blockIdx.x - t * H, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float* yr = y + (size_t)t * ldy + (size_t)h * V;
+    const float* gr = gate + (size_t)t * ld_gate + (size_t)h * V;
+    const float* wr = w + (w_per_head ? (size_t)h * V : 0);
+    OT* o = out + (size_t)t * ld_out + (size_t)h * V;
+    float inv_den = 1.f;
+    if (den != nullptr) {
+        const float2 d = *reinterpret_cast<const float2*>(den + (size_t)blockIdx.x * 2);
+        inv_den = 1.f / (fmaxf(fabsf(d.x), d.y) + DEN_EPS);
+    }
+    auto gated = [&](float z) { return act == VLRF_ACT_SILU ? silu_f(z) : sigmoid_f(z); };
+    auto all = [&](float ss) -> float {             // the sum over the CTA
+        ss = warp_sum(ss);
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        return ((red[0] + red[1]) + (red[2] + red[3])) + ((red[4] + red[5]) + (red[6] + red[7]));
+    };
+    float ss = 0.f;
+    if constexpr (NV > 0) {
+        float4 v[NV], gt[NV];
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int i = 4 * (threadIdx.x + 256 * k);
+            v[k] = gt[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < V) { v[k] = *reinterpret_cast<const float4*>(yr + i); gt[k] = *reinterpret_cast<const float4*>(gr + i); }
+        }
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            v[k].x *= inv_den; v[k].y *= inv_den; v[k].z *= inv_den; v[k].w *= inv_den;
+            ss = fmaf(v[k].x, v[k].x, ss); ss = fmaf(v[k].y, v[k].y, ss); ss = fmaf(v[k].z, v[k].z, ss); ss = fmaf(v[k].w, v[k].w, ss);
+        }
+        const float inv = factor / sqrtf(all(ss) / (float)V + eps);
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int i = 4 * (threadIdx.x + 256 * k);
+            if (i < V) {
+                const float4 ww = *reinterpret_cast<const float4*>(wr + i);
+                store4<OT>(o + i, v[k].x * inv * ww.x * gated(gt[k].x), v[k].y * inv * ww.y * gated(gt[k].y),
+                           v[k].z * inv * ww.z * gated(gt[k].z), v[k].w * inv * ww.w * gated(gt[k].w));
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < V; i += 256) { const float v = yr[i] * inv_den; ss = fmaf(v, v, ss); }
+        const float inv = factor / sqrtf(all(ss) / (float)V + eps);
+        for (int i = threadIdx.x; i < V; i += 256) ElemIO<OT>::store(o + i, yr[i] * inv_den * inv * wr[i] * gated(gr[i]));
+    }
+}
+
 // ---- two normed rows added to the residual ------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256)
 norm_pair_add_kernel(const float* __restrict__ a, const float* __restrict__ b, const float* __restrict__ wa, const float* __restrict__ wb,
@@ -532,11 +590,22 @@ extern "C" int vlrf_head_rows(const float* y, int ldy, const float* den, const f
     VLRF_REQUIRE(act == VLRF_ACT_SILU || act == VLRF_ACT_SIGMOID, "head_rows: the gate is sigmoid(z) or z·sigmoid(z)");
     if (T == 0) return VLRF_OK;
     const long long warps = (long long)T * H;
-    VLRF_REQUIRE((warps + 3) / 4 <= 0x7fffffffLL, "head_rows: too many rows");
+    VLRF_REQUIRE(warps <= 0x7fffffffLL, "head_rows: too many rows");
     const dim3 grid((unsigned)((warps + 3) / 4)), block(128);
     const int es = out_dtype == VLRF_BF16 ? 8 : 16;
-    const bool vec = V % 4 == 0 && V <= 512 && rows16(y) && ldy % 4 == 0 && rows16(gate) && ld_gate % 4 == 0 && rows16(w) &&
+    const bool quads = V % 4 == 0 && rows16(y) && ldy % 4 == 0 && rows16(gate) && ld_gate % 4 == 0 && rows16(w) &&
                      (reinterpret_cast<uintptr_t>(out) & (es - 1)) == 0 && ld_out % 4 == 0;
+    if (V > 512) {                                  // wide heads: a CTA each
+#define WIDE(OT, NV) launch_chained(head_rows_wide_kernel<OT, NV>, dim3((unsigned)warps), dim3(256), (size_t)0, stream, y, ldy, den, w, w_per_head, gate, ld_gate, act, (OT*)out, ld_out, H, V, eps, factor)
+#define WIDE_NV(OT) do { if (!quads || V > 8192) WIDE(OT, 0); else if (V <= 1024) WIDE(OT, 1); else if (V <= 2048) WIDE(OT, 2); else if (V <= 4096) WIDE(OT, 4); else WIDE(OT, 8); } while (0)
+        if (out_dtype == VLRF_F32) WIDE_NV(float);
+        else if (out_dtype == VLRF_BF16) WIDE_NV(__nv_bfloat16);
+        else return vlrf_fail(VLRF_ERR_INVALID_ARG, "head_rows: unknown output dtype %d", out_dtype);
+#undef WIDE_NV
+#undef WIDE
+        return vlrf_check_launch("head_rows");
+    }
+    const bool vec = quads;
 #define GO(OT, VEC) launch_chained(head_rows_kernel<OT, VEC>, grid, block, (size_t)0, stream, y, ldy, den, w, w_per_head, gate, ld_gate, act, (OT*)out, ld_out, T, H, V, eps, factor)
     if (out_dtype == VLRF_F32) { if (vec) GO(float, true); else GO(float, false); }
     else if (out_dtype == VLRF_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }

@@ -10,7 +10,8 @@
 //                score is largest; the weights are the chosen s · scale, not renormalized.  The last n_identity
 //                router outputs stand for experts that return their input: they get id −2, no rank and no row, and
 //                moe_combine adds weight · input for them.  With `scoring` 1 the scores are sigmoid(logit), each
-//                output by itself, instead of the softmax over all of them; everything else is the same.
+//                output by itself, instead of the softmax over all of them; everything else is the same.  With `renormalize` a
+//                chosen score is divided by the sum of the chosen (+ 1e-20) before the scale.
 //   moe_plan     offsets[e] = rows of the experts before e (E + 1 entries); the counters are left zero.
 //   moe_gather   pair (token, j) gets row offsets[expert] + rank of the expert-sorted buffer: the token's input row
 //                is copied there, multiplied by the pair's weight where the weights act on the experts' inputs, and the
@@ -84,7 +85,7 @@ moe_route_kernel(const float* __restrict__ z, int ld_z, int E, int top, int shar
 template <int NI>
 __global__ void __launch_bounds__(128)
 moe_route_scored_kernel(const float* __restrict__ z, int ld_z, int E, int top, int groups, int keep, int n_identity, float scale,
-                        int scoring, const float* __restrict__ correction, const int* __restrict__ tok_slot, int* __restrict__ ids,
+                        int scoring, int renormalize, const float* __restrict__ correction, const int* __restrict__ tok_slot, int* __restrict__ ids,
                         float* __restrict__ wts, int* __restrict__ rank, int* __restrict__ counts, int T) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
@@ -181,8 +182,10 @@ moe_route_scored_kernel(const float* __restrict__ z, int ld_z, int E, int top, i
             if (oi != 0x7fffffff && (idx == 0x7fffffff || ob > best || (ob == best && oi < idx))) { best = ob; idx = oi; sb = os; }
         }
         if ((idx & 31) == lane) taken |= 1u << (idx >> 5);
-        if ((j & 31) == lane) { my_w = sb * scale; my_id = idx; }
+        if ((j & 31) == lane) { my_w = sb; my_id = idx; }
     }
+    if (renormalize) my_w /= warp_sum(my_w) + 1e-20f;          // (lanes behind `top` hold zeros)
+    my_w *= scale;
     if (lane < top) {
         const bool identity = my_id >= E - n_identity;
         ids[(size_t)t * top + lane] = identity ? -2 : my_id;
@@ -256,7 +259,7 @@ extern "C" int vlrf_moe_route(const float* z, int ld_z, int E, int top, int shar
 }
 
 extern "C" int vlrf_moe_route_scored(const float* z, int ld_z, int E, int top, int groups, int keep, int n_identity, float scale,
-                                     int scoring, const float* correction, const int* tok_slot, int* ids, float* wts, int* rank, int* counts,
+                                     int scoring, int renormalize, const float* correction, const int* tok_slot, int* ids, float* wts, int* rank, int* counts,
                                      int T, cudaStream_t stream) {
     VLRF_REQUIRE(T >= 0 && E > 0 && E <= ROUTE_MAX_E && ld_z >= E, "moe_route_scored: takes 1…%d router outputs, not %d", ROUTE_MAX_E, E);
     VLRF_REQUIRE(groups > 0 && E % groups == 0 && keep > 0 && keep <= groups, "moe_route_scored: %d outputs in %d groups of which %d are kept", E, groups, keep);
@@ -265,7 +268,7 @@ extern "C" int vlrf_moe_route_scored(const float* z, int ld_z, int E, int top, i
     VLRF_REQUIRE(scoring == 0 || scoring == 1, "moe_route_scored: scores are a softmax over all outputs (0) or sigmoids (1), not %d", scoring);
     if (T == 0) return VLRF_OK;
     const dim3 grid((T + 3) / 4), block(128);
-#define VLRF_ROUTE_SCORED(NI) launch_chained(moe_route_scored_kernel<NI>, grid, block, (size_t)(0), stream, z, ld_z, E, top, groups, keep, n_identity, scale, scoring, correction, tok_slot, ids, wts, rank, counts, T)
+#define VLRF_ROUTE_SCORED(NI) launch_chained(moe_route_scored_kernel<NI>, grid, block, (size_t)(0), stream, z, ld_z, E, top, groups, keep, n_identity, scale, scoring, renormalize, correction, tok_slot, ids, wts, rank, counts, T)
     if (E <= 32) VLRF_ROUTE_SCORED(1);
     else if (E <= 64) VLRF_ROUTE_SCORED(2);
     else if (E <= 128) VLRF_ROUTE_SCORED(4);

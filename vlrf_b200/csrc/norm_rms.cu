@@ -11,7 +11,7 @@
 //
 // cast_rows: float32 rows to the activation dtype (what a sublayer reads of the float32 residual stream).
 // gate_mul: out = act(a) · b element by element (act: x·sigmoid(x) or max(x, 0) for gated feed-forwards, sigmoid(x) for
-// gates on an attention's merged heads), float32 arithmetic.  gate_mul_groups: one column of a for every `per`
+// gates on an attention's merged heads), float32 arithmetic, optionally times a constant.  gate_mul_groups: one column of a for every `per`
 // consecutive columns of b (a gate per head on the merged heads).
 //
 // rmsnorm_shift: the plain RMS norm of a token's residual row followed by a token shift: with n_t the normed row,
@@ -111,7 +111,7 @@ __global__ void cast_rows_kernel(const float* __restrict__ x, OT* __restrict__ o
 
 // the same, eight bfloat16 a thread (rows and columns on 16-byte boundaries)
 __global__ void gate_mul_bf16x8_kernel(const __nv_bfloat16* a, int lda, const __nv_bfloat16* b, int ldb, __nv_bfloat16* out, int ldo,
-                                       int rows, int cols8, int act) {
+                                       int rows, int cols8, int act, float factor) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -124,7 +124,7 @@ __global__ void gate_mul_bf16x8_kernel(const __nv_bfloat16* a, int lda, const __
     for (int k = 0; k < 4; ++k) {
         const float g0 = __uint_as_float(gw[k] << 16), g1 = __uint_as_float(gw[k] & 0xffff0000u);
         const float v0 = __uint_as_float(vw[k] << 16), v1 = __uint_as_float(vw[k] & 0xffff0000u);
-        const float f0 = gate_f(act, g0), f1 = gate_f(act, g1);
+        const float f0 = gate_f(act, g0) * factor, f1 = gate_f(act, g1) * factor;
         const __nv_bfloat162 p = __floats2bfloat162_rn(f0 * v0, f1 * v1);
         o[k] = *reinterpret_cast<const uint32_t*>(&p);
     }
@@ -133,15 +133,15 @@ __global__ void gate_mul_bf16x8_kernel(const __nv_bfloat16* a, int lda, const __
 
 // float32 gate and value, bfloat16 result, four a thread (rows and columns on 16-byte boundaries)
 __global__ void gate_mul_f32x4_kernel(const float* a, int lda, const float* b, int ldb, __nv_bfloat16* out, int ldo, int rows, int cols4,
-                                      int act) {
+                                      int act, float factor) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (long long)rows * cols4) return;
     const int r = (int)(i / cols4), c = (int)(i - (long long)r * cols4) * 4;
     const float4 g = *reinterpret_cast<const float4*>(a + (size_t)r * lda + c), v = *reinterpret_cast<const float4*>(b + (size_t)r * ldb + c);
-    const __nv_bfloat162 lo = __floats2bfloat162_rn(gate_f(act, g.x) * v.x, gate_f(act, g.y) * v.y);
-    const __nv_bfloat162 hi = __floats2bfloat162_rn(gate_f(act, g.z) * v.z, gate_f(act, g.w) * v.w);
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(gate_f(act, g.x) * factor * v.x, gate_f(act, g.y) * factor * v.y);
+    const __nv_bfloat162 hi = __floats2bfloat162_rn(gate_f(act, g.z) * factor * v.z, gate_f(act, g.w) * factor * v.w);
     *reinterpret_cast<uint2*>(out + (size_t)r * ldo + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
 }
 
@@ -167,7 +167,8 @@ __global__ void gate_mul_groups_bf16x8_kernel(const float* a, int lda, const __n
 }
 
 template <typename AT, typename BT, typename OT>
-__global__ void gate_mul_kernel(const AT* a, int lda, const BT* b, int ldb, OT* out, int ldo, int rows, int cols, int act, int per) {
+__global__ void gate_mul_kernel(const AT* a, int lda, const BT* b, int ldb, OT* out, int ldo, int rows, int cols, int act, int per,
+                                float factor) {
     pdl_wait();                 // chained launch: nothing is read before the kernels ahead have finished
     pdl_launch_dependents();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -175,7 +176,7 @@ __global__ void gate_mul_kernel(const AT* a, int lda, const BT* b, int ldb, OT* 
     const int r = (int)(i / cols), c = (int)(i - (long long)r * cols);
     const float g = ElemIO<AT>::load(a + (size_t)r * lda + c / per);
     const float v = ElemIO<BT>::load(b + (size_t)r * ldb + c);
-    const float f = gate_f(act, g);
+    const float f = gate_f(act, g) * factor;
     ElemIO<OT>::store(out + (size_t)r * ldo + c, f * v);
 }
 
@@ -496,7 +497,7 @@ extern "C" int vlrf_cast_rows(const float* x, void* out, int out_dtype, long lon
 }
 
 static int gate_mul_any(const void* a, int lda, int a_dtype, const void* b, int ldb, int b_dtype, void* out, int ldo,
-                        int out_dtype, int rows, int cols, int per, int act, cudaStream_t stream);
+                        int out_dtype, int rows, int cols, int per, int act, float factor, cudaStream_t stream);
 
 extern "C" int vlrf_gate_mul_clamped(const void* a, int lda, int a_dtype, const void* b, int ldb, int b_dtype, void* out, int ldo,
                                      int out_dtype, int rows, int cols, float limit, float alpha, cudaStream_t stream) {
@@ -521,18 +522,18 @@ extern "C" int vlrf_gate_mul_clamped(const void* a, int lda, int a_dtype, const 
 }
 
 extern "C" int vlrf_gate_mul(const void* a, int lda, int a_dtype, const void* b, int ldb, int b_dtype, void* out, int ldo,
-                             int out_dtype, int rows, int cols, int act, cudaStream_t stream) {
-    return gate_mul_any(a, lda, a_dtype, b, ldb, b_dtype, out, ldo, out_dtype, rows, cols, 1, act, stream);
+                             int out_dtype, int rows, int cols, int act, float factor, cudaStream_t stream) {
+    return gate_mul_any(a, lda, a_dtype, b, ldb, b_dtype, out, ldo, out_dtype, rows, cols, 1, act, factor, stream);
 }
 
 extern "C" int vlrf_gate_mul_groups(const void* a, int lda, int a_dtype, const void* b, int ldb, int b_dtype, void* out, int ldo,
                                     int out_dtype, int rows, int cols, int per, int act, cudaStream_t stream) {
     VLRF_REQUIRE(per > 0 && cols % per == 0, "gate_mul_groups: %d columns are no whole groups of %d", cols, per);
-    return gate_mul_any(a, lda, a_dtype, b, ldb, b_dtype, out, ldo, out_dtype, rows, cols, per, act, stream);
+    return gate_mul_any(a, lda, a_dtype, b, ldb, b_dtype, out, ldo, out_dtype, rows, cols, per, act, 1.f, stream);
 }
 
 static int gate_mul_any(const void* a, int lda, int a_dtype, const void* b, int ldb, int b_dtype, void* out, int ldo,
-                        int out_dtype, int rows, int cols, int per, int act, cudaStream_t stream) {
+                        int out_dtype, int rows, int cols, int per, int act, float factor, cudaStream_t stream) {
     VLRF_REQUIRE(rows >= 0 && cols > 0 && per > 0 && lda >= cols / per && ldb >= cols && ldo >= cols, "gate_mul: bad sizes");
     VLRF_REQUIRE(act == VLRF_ACT_SILU || act == VLRF_ACT_SIGMOID || act == VLRF_ACT_RELU || act == VLRF_ACT_GELU_TANH,
                  "gate_mul: the gate is x*sigmoid(x), sigmoid(x), max(x, 0) or the tanh form of GELU, not %d", act);
@@ -542,20 +543,20 @@ static int gate_mul_any(const void* a, int lda, int a_dtype, const void* b, int 
     const bool aligned = per == 1 && ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 &&
                          cols % 8 == 0 && lda % 8 == 0 && ldb % 8 == 0 && ldo % 8 == 0;
     typedef __nv_bfloat16 bf;
-#define GO(AT, BT, OT) launch_chained(gate_mul_kernel<AT, BT, OT>, blocks, dim3(256), (size_t)0, stream, (const AT*)a, lda, (const BT*)b, ldb, (OT*)out, ldo, rows, cols, act, per)
+#define GO(AT, BT, OT) launch_chained(gate_mul_kernel<AT, BT, OT>, blocks, dim3(256), (size_t)0, stream, (const AT*)a, lda, (const BT*)b, ldb, (OT*)out, ldo, rows, cols, act, per, factor)
     if (per > 1 && per % 8 == 0 && a_dtype == VLRF_F32 && b_dtype == VLRF_BF16 && out_dtype == VLRF_BF16 && ldb % 8 == 0 && ldo % 8 == 0 &&
         ((reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(out)) & 15) == 0)
         launch_chained(gate_mul_groups_bf16x8_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), (size_t)0, stream, (const float*)a, lda,
                        (const bf*)b, ldb, (bf*)out, ldo, rows, cols / 8, per / 8, act);
     else if (a_dtype == VLRF_BF16 && b_dtype == VLRF_BF16 && out_dtype == VLRF_BF16 && aligned)
         launch_chained(gate_mul_bf16x8_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), (size_t)0, stream, (const bf*)a, lda, (const bf*)b, ldb,
-                       (bf*)out, ldo, rows, cols / 8, act);
+                       (bf*)out, ldo, rows, cols / 8, act, factor);
     else if (a_dtype == VLRF_BF16 && b_dtype == VLRF_BF16 && out_dtype == VLRF_BF16) GO(bf, bf, bf);
     else if (a_dtype == VLRF_F32 && b_dtype == VLRF_F32 && out_dtype == VLRF_F32) GO(float, float, float);
     else if (a_dtype == VLRF_F32 && b_dtype == VLRF_BF16 && out_dtype == VLRF_BF16) GO(float, bf, bf);
     else if (a_dtype == VLRF_F32 && b_dtype == VLRF_F32 && out_dtype == VLRF_BF16 && aligned && lda % 4 == 0 && ldb % 4 == 0)
         launch_chained(gate_mul_f32x4_kernel, dim3((unsigned)((n / 4 + 255) / 256)), dim3(256), (size_t)0, stream, (const float*)a, lda,
-                       (const float*)b, ldb, (bf*)out, ldo, rows, cols / 4, act);
+                       (const float*)b, ldb, (bf*)out, ldo, rows, cols / 4, act, factor);
     else if (a_dtype == VLRF_F32 && b_dtype == VLRF_F32 && out_dtype == VLRF_BF16) GO(float, float, bf);
     else return vlrf_fail(VLRF_ERR_INVALID_ARG, "gate_mul: dtypes %d, %d -> %d are not taken", a_dtype, b_dtype, out_dtype);
 #undef GO

@@ -616,10 +616,10 @@ def cast_rows(x, out, n_rows: int) -> None:
     call("vlrf_cast_rows", _ptr(x), _ptr(out), dtype_code(out.dtype), n_rows * x.shape[1], _stream())
 
 
-def gate_mul(a, b, out, gate: str, n_rows: int, cols: int, per: int = 1) -> None:
-    """out[r, :cols] = gate(a[r, :cols]) · b[r, :cols]; gate "silu", "sigmoid" or "relu".  a, b and out may be column ranges
+def gate_mul(a, b, out, gate: str, n_rows: int, cols: int, per: int = 1, factor: float = 1.0) -> None:
+    """out[r, :cols] = gate(a[r, :cols]) · b[r, :cols] · factor; gate "silu", "sigmoid" or "relu".  a, b and out may be column ranges
     of wider rows, and out may be a or b.  a and b may be float32 where out is bfloat16 (see the kernel library's header).
-    per > 1: one column of a for every `per` consecutive columns of b (a gate per head on merged heads)."""
+    per > 1: one column of a for every `per` consecutive columns of b (a gate per head on merged heads; no factor)."""
     for name, t in (("a", a), ("b", b), ("out", out)):
         _rows(t, name)
         if t.shape[0] < n_rows or t.shape[1] < (cols // per if name == "a" else cols):
@@ -627,11 +627,13 @@ def gate_mul(a, b, out, gate: str, n_rows: int, cols: int, per: int = 1) -> None
     if per != 1:
         if per < 1 or cols % per != 0:
             raise KernelError(f"gate_mul: {cols} columns are no whole groups of {per}")
+        if factor != 1.0:
+            raise KernelError("gate_mul: a gate per group takes no factor")
         call("vlrf_gate_mul_groups", _ptr(a), a.stride(0), dtype_code(a.dtype), _ptr(b), b.stride(0), dtype_code(b.dtype), _ptr(out),
              out.stride(0), dtype_code(out.dtype), n_rows, cols, int(per), GATE[gate], _stream())
         return
     call("vlrf_gate_mul", _ptr(a), a.stride(0), dtype_code(a.dtype), _ptr(b), b.stride(0), dtype_code(b.dtype), _ptr(out),
-         out.stride(0), dtype_code(out.dtype), n_rows, cols, GATE[gate], _stream())
+         out.stride(0), dtype_code(out.dtype), n_rows, cols, GATE[gate], float(factor), _stream())
 
 
 # ---- products per head and per group ---------------------------------------------------------------------------------
@@ -661,8 +663,8 @@ def linear_heads(x, w, out, n_rows: int) -> None:
 
 def linear_grouped(x, w, out, offsets, n_rows: int, act=None) -> None:
     """Rows offsets[g] … offsets[g+1]−1 of x [P, K] times w[g]ᵀ (w [G, N, K]) into the same rows of out [P, N];
-    offsets: int32 [G + 1] on the device.  act: None, "gelu_tanh" or "relu2" on the result."""
-    if act not in (None, "none", "gelu_tanh", "relu2"):
+    offsets: int32 [G + 1] on the device.  act: None, "gelu_tanh", "gelu_erf" or "relu2" on the result."""
+    if act not in (None, "none", "gelu_tanh", "gelu_erf", "relu2"):
         raise KernelError(f"linear_grouped: activation '{act}' is not taken")
     _dev(x, "x"); _dev(w, "w", x.dtype); _dev(out, "out"); _dev(offsets, "offsets", torch.int32)
     G, N, K = w.shape
@@ -681,8 +683,9 @@ def linear_grouped(x, w, out, offsets, n_rows: int, act=None) -> None:
 # ---- attention over a cache of latents --------------------------------------------------------------------------------
 
 def latent_append(proj, C: int, R: int, norm_weight, eps: float, inv_freq, rot_dims: int, cache, block_table, tok_slot,
-                  tok_pos, n_tokens: int, dev_err, interleaved: bool = False) -> None:
-    """Each token's row [RMSnorm(proj[:C]) · weight | rotate(proj[C:C+R])] into the paged cache [block, BT, row]."""
+                  tok_pos, n_tokens: int, dev_err, interleaved: bool = False, magnitude: float = 1.0) -> None:
+    """Each token's row [RMSnorm(proj[:C]) · weight | rotate(proj[C:C+R])] into the paged cache [block, BT, row]; magnitude: a
+    factor on the rotation's cosines and sines."""
     _rows(proj, "proj", torch.float32); _dev(norm_weight, "norm_weight", torch.float32); _dev(cache, "cache")
     _dev(block_table, "block_table", torch.int32); _dev(tok_slot, "tok_slot", torch.int32)
     _dev(tok_pos, "tok_pos", torch.int32); _dev(dev_err, "dev_err", torch.int32)
@@ -693,12 +696,12 @@ def latent_append(proj, C: int, R: int, norm_weight, eps: float, inv_freq, rot_d
     if proj.shape[1] < C + R or cache.shape[2] < C + R or norm_weight.shape[0] != C or proj.shape[0] < n_tokens:
         raise KernelError("latent_append: sizes do not match")
     call("vlrf_latent_append", _ptr(proj), proj.stride(0), C, R, _ptr(norm_weight), float(eps), _ptr(inv_freq), int(rot_dims),
-         1 if interleaved else 0, _ptr(cache), dtype_code(cache.dtype), cache.shape[2], _ptr(block_table), block_table.shape[1], _ptr(tok_slot),
+         1 if interleaved else 0, float(magnitude), _ptr(cache), dtype_code(cache.dtype), cache.shape[2], _ptr(block_table), block_table.shape[1], _ptr(tok_slot),
          _ptr(tok_pos), n_tokens, cache.shape[1], _ptr(dev_err), _stream())
 
 
 def latent_q_rows(q, n_heads: int, dim: int, R: int, inv_freq, rot_dims: int, tok_pos, qn, qp, C: int, n_tokens: int,
-                  interleaved: bool = False) -> None:
+                  interleaved: bool = False, magnitude: float = 1.0) -> None:
     """q float32 [T, H·(dim + R)] → qn [T, H·dim] (unrotated parts) and the last R columns of each head's C + R columns
     of qp (rotated parts, rotated by position)."""
     _rows(q, "q", torch.float32); _dev(qn, "qn"); _dev(qp, "qp", qn.dtype); _dev(tok_pos, "tok_pos", torch.int32)
@@ -706,7 +709,7 @@ def latent_q_rows(q, n_heads: int, dim: int, R: int, inv_freq, rot_dims: int, to
         _dev(inv_freq, "inv_freq", torch.float32)
     if q.shape[1] != n_heads * (dim + R) or qn.shape[1] != n_heads * dim or qp.shape[1] != n_heads * (C + R):
         raise KernelError("latent_q_rows: sizes do not match")
-    call("vlrf_latent_q_rows", _ptr(q), q.stride(0), n_heads, dim, R, _ptr(inv_freq), int(rot_dims), 1 if interleaved else 0, _ptr(tok_pos), _ptr(qn),
+    call("vlrf_latent_q_rows", _ptr(q), q.stride(0), n_heads, dim, R, _ptr(inv_freq), int(rot_dims), 1 if interleaved else 0, float(magnitude), _ptr(tok_pos), _ptr(qn),
          qn.shape[1], _ptr(qp), qp.shape[1], C, dtype_code(qn.dtype), n_tokens, _stream())
 
 
@@ -746,9 +749,11 @@ def attention_rows_strides_ok(dim: int, R: int, vdim: int, ld_qn: int, ld_qr: in
 
 
 def attention_rows(qn, qr, kn, kr, v, seq_start, out, n_seqs: int, max_new: int, n_heads: int, dim: int, R: int, vdim: int,
-                   scale: float) -> None:
+                   scale: float, window: int = 0, sink=None, out_scale: float = 1.0) -> None:
     """Causal attention of sequences that begin at position 0 over keys and values in plain rows (see the kernel library's
-    header): qn, kn [T, H·dim]; qr [T, H·R], kr [T, R] (None with R = 0); v, out [T, H·vdim]; bfloat16."""
+    header): qn, kn [T, H·dim]; qr [T, H·R], kr [T, R] (None with R = 0); v, out [T, H·vdim]; bfloat16.  window > 0: the last
+    `window` keys; sink: float32 [heads], exp(sink) joins the softmax's denominator; out_scale: a factor on the result."""
+    _check_sink(sink, n_heads)
     for name, t in (("qn", qn), ("kn", kn), ("v", v), ("out", out)):          # (column ranges of wider rows are taken)
         _rows(t, name, torch.bfloat16)
     if R > 0:
@@ -762,7 +767,8 @@ def attention_rows(qn, qr, kn, kr, v, seq_start, out, n_seqs: int, max_new: int,
     if not lib_takes:
         raise KernelError("attention_rows: these sizes or row strides are not taken")
     call("vlrf_attn_rows", _ptr(qn), qn.stride(0), _ptr(qr) if R > 0 else 0, qr.stride(0) if R > 0 else 0, _ptr(kn), kn.stride(0),
-         _ptr(kr) if R > 0 else 0, kr.stride(0) if R > 0 else 0, _ptr(v), v.stride(0), _ptr(seq_start), _ptr(out), out.stride(0), n_seqs, max_new, n_heads, dim, R, vdim, float(scale), _stream())
+         _ptr(kr) if R > 0 else 0, kr.stride(0) if R > 0 else 0, _ptr(v), v.stride(0), _ptr(seq_start), _ptr(out), out.stride(0), n_seqs, max_new, n_heads, dim, R, vdim, float(scale),
+         int(window), _ptr(sink), float(out_scale), _stream())
 
 
 LATENT_ATTENTION_MMA = True          # off: every step takes the general kernel (for measurements and cross-checks)
@@ -795,10 +801,12 @@ def latent_decode_splits(n_rows: int, n_heads: int, max_context: int, C: int, R:
 
 
 def attention_latent(qp, cache, C: int, R: int, block_table, tok_slot, tok_pos, out, n_tokens: int, n_heads: int, scale: float,
-                     window: int, dev_err, ctx=None) -> None:
+                     window: int, dev_err, ctx=None, sink=None, out_scale: float = 1.0) -> None:
     """Each token's heads (queries in latent space, [T, H·(C + R)]) attend the rows 0…position of the token's slot in
     the latent cache [block, BT, row]; out [T, H·C] receives Σ_j p_j c_j per head.  With the step's context (`ctx`:
-    its sequence tables and scratch) bfloat16 steps of sizes that the tensor-core kernel takes run there."""
+    its sequence tables and scratch) bfloat16 steps of sizes that the tensor-core kernel takes run there.  sink: float32
+    [heads], exp(sink) joins the softmax's denominator; out_scale: a factor on the result."""
+    _check_sink(sink, n_heads)
     _dev(qp, "qp"); _dev(cache, "cache", qp.dtype); _dev(out, "out", qp.dtype)
     _dev(block_table, "block_table", torch.int32); _dev(tok_slot, "tok_slot", torch.int32)
     _dev(tok_pos, "tok_pos", torch.int32); _dev(dev_err, "dev_err", torch.int32)
@@ -808,17 +816,18 @@ def attention_latent(qp, cache, C: int, R: int, block_table, tok_slot, tok_pos, 
     if ctx is not None and _latent_mma_takes(qp.dtype, C, R, cache.shape[2], cache.shape[1], qp.shape[1]):
         n_split, partials = 1, None
         if ctx.max_new == 1:
-            n_split = latent_decode_splits(ctx.n_seqs, n_heads, ctx.max_context, C, R)
+            reach = min(ctx.max_context, window + 31) if window > 0 else ctx.max_context       # (a window may begin inside a tile)
+            n_split = latent_decode_splits(ctx.n_seqs, n_heads, reach, C, R)
             if n_split > 1:
                 partials = ctx.ws.get("latent_attn_partials", ctx.n_seqs * ((n_heads + 15) // 16) * n_split * 16, C + 2, torch.float32)
         call("vlrf_attn_latent_mma", _ptr(qp), qp.shape[1], _ptr(cache), cache.shape[2], C, R, _ptr(block_table),
              block_table.shape[1], _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(out), out.shape[1],
              ctx.n_seqs, ctx.max_new, n_heads, cache.shape[1], float(scale), int(window), n_split, _ptr(partials),
-             _ptr(dev_err), _stream())
+             _ptr(sink), float(out_scale), _ptr(dev_err), _stream())
         return
     call("vlrf_attn_latent", _ptr(qp), dtype_code(qp.dtype), qp.shape[1], _ptr(cache), cache.shape[2], C, R, _ptr(block_table),
          block_table.shape[1], _ptr(tok_slot), _ptr(tok_pos), _ptr(out), out.shape[1], n_tokens, n_heads, cache.shape[1],
-         float(scale), int(window), _ptr(dev_err), _stream())
+         float(scale), int(window), _ptr(sink), float(out_scale), _ptr(dev_err), _stream())
 
 
 # ---- routed experts --------------------------------------------------------------------------------------------------
@@ -844,10 +853,11 @@ def moe_route(z, n_experts: int, top: int, shared_gate: bool, tok_slot, ids, wts
 
 
 def moe_route_scored(z, n_outputs: int, top: int, groups: int, keep: int, n_identity: int, scale: float, correction, tok_slot,
-                     ids, wts, rank, counts, n_tokens: int, scoring: str = "softmax") -> None:
+                     ids, wts, rank, counts, n_tokens: int, scoring: str = "softmax", renormalize: bool = False) -> None:
     """From float32 router logits z [T, ≥ n_outputs]: softmax over all outputs (scoring "sigmoid": the sigmoid of each),
     the choice by score + correction inside the `keep` best of `groups` groups, weights score · scale; the last
-    n_identity outputs get id −2 and no rank (see the kernel library's header)."""
+    n_identity outputs get id −2 and no rank (see the kernel library's header).  renormalize: the chosen scores are divided by
+    their sum (+ 1e-20) first."""
     if scoring not in ("softmax", "sigmoid"):
         raise KernelError(f"moe_route_scored: scoring '{scoring}' is neither 'softmax' nor 'sigmoid'")
     _rows(z, "z", torch.float32); _dev(ids, "ids", torch.int32); _dev(wts, "wts", torch.float32)
@@ -858,7 +868,7 @@ def moe_route_scored(z, n_outputs: int, top: int, groups: int, keep: int, n_iden
             or counts.numel() < max(n_outputs - n_identity, 1):
         raise KernelError("moe_route_scored: sizes do not match")
     call("vlrf_moe_route_scored", _ptr(z), z.stride(0), n_outputs, top, int(groups), int(keep), int(n_identity), float(scale),
-         1 if scoring == "sigmoid" else 0, _ptr(correction), _ptr(tok_slot), _ptr(ids), _ptr(wts), _ptr(rank), _ptr(counts), n_tokens, _stream())
+         1 if scoring == "sigmoid" else 0, 1 if renormalize else 0, _ptr(correction), _ptr(tok_slot), _ptr(ids), _ptr(wts), _ptr(rank), _ptr(counts), n_tokens, _stream())
 
 
 def moe_plan(counts, offsets, n_experts: int) -> None:
@@ -1001,16 +1011,17 @@ def gate_mul_clamped(a, b, out, limit: float, alpha: float, n_rows: int, cols: i
 def qkv_rope_append(proj, q_off: int, k_off: int, v_off: int, freq, rot: int, q_out, k_cache, v_cache, block_table, tok_slot,
                     tok_pos, n_tokens: int, n_heads: int, n_kv_heads: int, dk: int, dv: int, write_cache: bool, dev_err, *,
                     norm: str | None = None, q_norm=None, k_norm=None, eps: float = 0.0, interleaved: bool = False,
-                    magnitude: float = 1.0) -> None:
+                    magnitude: float = 1.0, maps: int = 1) -> None:
     """Queries (rotated) into q_out, keys (rotated) and values into the paged cache, from the float32 rows of a layer's
     input product.  proj may be a range of columns of wider rows.  norm "head" / "all": an RMS norm of queries and keys
     ahead of the rotation, every head by itself (weights of dk entries shared by the heads) or the whole projection as
     one row (weights of heads · dk entries); interleaved: entry 2i pairs with 2i + 1; magnitude: a factor on cosines and
-    sines.  With write_cache False the key and value columns are not read (k_off, v_off, k_norm are ignored)."""
+    sines.  With write_cache False the key and value columns are not read (k_off, v_off, k_norm are ignored).  maps 2:
+    every query and key head is two maps of dk entries, each rotated by itself; the cache's key rows hold both."""
     _rows(proj, "proj", torch.float32); _dev(q_out, "q_out"); _dev(k_cache, "k_cache", q_out.dtype); _dev(v_cache, "v_cache", q_out.dtype)
     _dev(block_table, "block_table", torch.int32); _dev(tok_slot, "tok_slot", torch.int32); _dev(tok_pos, "tok_pos", torch.int32)
     nb, hkv, bt, kd = k_cache.shape
-    if hkv != n_kv_heads or kd != dk or tuple(v_cache.shape) != (nb, hkv, bt, dv):
+    if hkv != n_kv_heads or kd != maps * dk or tuple(v_cache.shape) != (nb, hkv, bt, dv):
         raise KernelError("qkv_rope_append: cache shape does not match the heads")
     if rot > 0:
         _dev(freq, "freq", torch.float32)
@@ -1023,17 +1034,34 @@ def qkv_rope_append(proj, q_off: int, k_off: int, v_off: int, freq, rot: int, q_
         raise KernelError(f"qkv_rope_append: norm '{norm}' is neither 'head' nor 'all'")
     if code:
         _dev(q_norm, "q_norm", torch.float32)
-        if q_norm.numel() != (dk if code == 1 else n_heads * dk):
+        if q_norm.numel() != (dk if code == 1 else n_heads * maps * dk):
             raise KernelError("qkv_rope_append: the queries' norm weights do not match")
         if write_cache:
             _dev(k_norm, "k_norm", torch.float32)
-            if k_norm.numel() != (dk if code == 1 else n_kv_heads * dk):
+            if k_norm.numel() != (dk if code == 1 else n_kv_heads * maps * dk):
                 raise KernelError("qkv_rope_append: the keys' norm weights do not match")
     call("vlrf_qkv_norm_rope_append", _ptr(proj), proj.stride(0), q_off, k_off if write_cache else 0, v_off if write_cache else 0,
          _ptr(freq) if rot > 0 else 0, int(rot), _ptr(q_out), q_out.shape[1], _ptr(k_cache), _ptr(v_cache), dtype_code(q_out.dtype),
          _ptr(block_table), block_table.shape[1], _ptr(tok_slot), _ptr(tok_pos), n_tokens, n_heads, n_kv_heads, dk, dv, bt,
-         1 if write_cache else 0, code, _ptr(q_norm) if code else 0, _ptr(k_norm) if code and write_cache else 0, float(eps),
+         int(maps), 1 if write_cache else 0, code, _ptr(q_norm) if code else 0, _ptr(k_norm) if code and write_cache else 0, float(eps),
          1 if interleaved else 0, float(magnitude), _ptr(dev_err), _stream())
+
+
+def _check_sink(sink, n_heads: int) -> None:
+    if sink is not None:
+        _dev(sink, "sink", torch.float32)
+        if sink.numel() != n_heads:
+            raise KernelError("attention: one sink per query head")
+
+
+def _map_args(second, sink, gate) -> tuple:
+    """(maps, factor, eps) of the kernels from `second` = None or (factor, eps)."""
+    if second is None:
+        return 1, 0.0, 0.0
+    factor, eps = second
+    if sink is not None or gate is not None or not eps > 0.0:
+        raise KernelError("attention_window: two maps a head go without sinks and gates and with a positive eps")
+    return 2, float(factor), float(eps)
 
 
 def _check_slopes(slopes, n_heads: int) -> None:
@@ -1052,28 +1080,29 @@ def _check_head_gate(gate, n_rows: int, n_heads: int) -> None:
 
 def attention_window(q, k_cache, v_cache, block_table, tok_slot, tok_pos, out, n_tokens: int, n_heads: int, n_kv_heads: int,
                      dk: int, dv: int, scale: float, window: int, out_scale: float, dev_err, *, softcap: float = 0.0,
-                     keep_first: int = 0, sink=None, gate=None, slopes=None) -> None:
+                     keep_first: int = 0, sink=None, gate=None, slopes=None, second_map=None) -> None:
     """Each token's queries attend the visible keys of its slot; out may be a range of columns of wider rows.  softcap > 0
     squashes the scaled scores; keys at positions below keep_first stay visible whatever the window; sink: float32
     [heads], exp(sink) joins the softmax's denominator; gate: float32 [T, ≥ heads] (a range of columns of wider rows will
-    do), head h's result times sigmoid(gate[t, h]); slopes: float32 [heads], slope · distance is taken off every score."""
+    do), head h's result times sigmoid(gate[t, h]); slopes: float32 [heads], slope · distance is taken off every score.
+    second_map = (factor, eps): differential attention (see the kernel library's header): heads of two maps of dk numbers
+    side by side (q [T, heads·2·dk], key rows of 2·dk), the second map's result times factor off the first's, then
+    divided by sqrt(mean of squares + eps) per head."""
+    maps, map_factor, head_eps = _map_args(second_map, sink, gate)
     _check_head_gate(gate, n_tokens, n_heads)
     _check_slopes(slopes, n_heads)
-    if sink is not None:
-        _dev(sink, "sink", torch.float32)
-        if sink.numel() != n_heads:
-            raise KernelError("attention_window: one sink per query head")
+    _check_sink(sink, n_heads)
     _dev(q, "q"); _dev(k_cache, "k_cache", q.dtype); _dev(v_cache, "v_cache", q.dtype); _rows(out, "out", q.dtype)
     _dev(block_table, "block_table", torch.int32); _dev(tok_slot, "tok_slot", torch.int32); _dev(tok_pos, "tok_pos", torch.int32)
     nb, hkv, bt, kd = k_cache.shape
-    if hkv != n_kv_heads or kd != dk or tuple(v_cache.shape) != (nb, hkv, bt, dv):
+    if hkv != n_kv_heads or kd != maps * dk or tuple(v_cache.shape) != (nb, hkv, bt, dv) or q.shape[1] < n_heads * maps * dk:
         raise KernelError("attention_window: cache shape does not match the heads")
     if out.shape[1] < n_heads * dv or out.shape[0] < n_tokens or q.shape[0] < n_tokens:
         raise KernelError("attention_window: output does not match")
     call("vlrf_attn_window_ex", _ptr(q), dtype_code(q.dtype), q.shape[1], _ptr(k_cache), _ptr(v_cache), _ptr(block_table),
          block_table.shape[1], _ptr(tok_slot), _ptr(tok_pos), _ptr(out), out.stride(0), n_tokens, n_heads, n_kv_heads, dk, dv, bt,
          float(scale), int(window), float(out_scale), float(softcap), int(keep_first), _ptr(sink), _ptr(gate),
-         gate.stride(0) if gate is not None else 0, _ptr(slopes), _ptr(dev_err), _stream())
+         gate.stride(0) if gate is not None else 0, _ptr(slopes), maps, map_factor, head_eps, _ptr(dev_err), _stream())
 
 
 # ---- a state-space recurrence with a matrix state per head -----------------------------------------------------------------
@@ -1152,32 +1181,34 @@ def window_decode_splits(n_rows: int, n_kv_heads: int, max_context: int, window:
 
 def attention_window_step(q, k_cache, v_cache, block_table, out, ctx, n_heads: int, n_kv_heads: int, dk: int, dv: int, scale: float,
                           window: int, out_scale: float, *, softcap: float = 0.0, keep_first: int = 0, sink=None, gate=None,
-                          slopes=None) -> None:
+                          slopes=None, second_map=None) -> None:
     """The attention of a step (prompt tokens, single tokens or a mix) with the kernel that suits it: bfloat16 sizes that
     the tensor-core kernel takes go there (a decode step's contexts cut into parts), everything else to the kernel
     that takes a warp per token and head."""
     bt = k_cache.shape[2]
+    maps, map_factor, head_eps = _map_args(second_map, sink, gate)
     if _window_mma_takes(q.dtype, n_heads, n_kv_heads, dk, dv, bt, q.shape[1], out.stride(0)) and q.data_ptr() % 16 == 0 \
             and out.data_ptr() % 4 == 0:
         _rows(out, "out", q.dtype)
+        if k_cache.shape[3] != maps * dk or v_cache.shape[3] != dv or q.shape[1] < n_heads * maps * dk or out.shape[1] < n_heads * dv:
+            raise KernelError("attention_window: cache shape, queries or output do not match the heads")
         n_split, partials = 1, None
         if ctx.max_new == 1:
             n_split = window_decode_splits(ctx.n_tokens, n_kv_heads, ctx.max_context, window, keep_first)
             if n_split > 1:
-                partials = ctx.ws.get("window_partials", ctx.n_tokens * n_heads * n_split, dv + 2, torch.float32)
-        if sink is not None:
-            _dev(sink, "sink", torch.float32)
-            if sink.numel() != n_heads:
-                raise KernelError("attention_window: one sink per query head")
+                partials = ctx.ws.get("window_partials", ctx.n_tokens * n_heads * maps * n_split, dv + 2, torch.float32)
+        _check_sink(sink, n_heads)
         _check_head_gate(gate, ctx.n_tokens, n_heads)
         _check_slopes(slopes, n_heads)
         call("vlrf_attn_window_mma_ex", _ptr(q), q.shape[1], _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
              _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(out), out.stride(0), _ptr(partials), ctx.n_seqs,
              ctx.max_new, n_heads, n_kv_heads, dk, dv, bt, float(scale), int(window), float(out_scale), n_split, float(softcap),
-             int(keep_first), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(slopes), _ptr(ctx.dev_err), _stream())
+             int(keep_first), _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(slopes), maps, map_factor,
+             head_eps, _ptr(ctx.dev_err), _stream())
         return
     attention_window(q, k_cache, v_cache, block_table, ctx.tok_slot, ctx.tok_pos, out, ctx.n_tokens, n_heads, n_kv_heads, dk, dv,
-                     scale, window, out_scale, ctx.dev_err, softcap=softcap, keep_first=keep_first, sink=sink, gate=gate, slopes=slopes)
+                     scale, window, out_scale, ctx.dev_err, softcap=softcap, keep_first=keep_first, sink=sink, gate=gate, slopes=slopes,
+                     second_map=second_map)
 
 
 def ssd_scan_step(xbc, proj, dt_off: int, dt_bias, a_log, d_skip, state, ctx, y, n_heads: int, n_groups: int, n_state: int, p: int) -> None:
@@ -1190,7 +1221,7 @@ def ssd_scan_step(xbc, proj, dt_off: int, dt_bias, a_log, d_skip, state, ctx, y,
 
 #: kinds of `matrix_state_scan` (see the kernel library's header), the most state rows and columns, channels of a
 #: convolved head and taps
-MATRIX_STATE_KINDS = {"decayed": 0, "delta": 1, "stabilized": 2}
+MATRIX_STATE_KINDS = {"decayed": 0, "delta": 1, "stabilized": 2, "fixed": 3}
 MATRIX_STATE_MAX_ROWS, MATRIX_STATE_MAX_COLUMNS, CONV_UNIT_MAX_HEAD, CONV_UNIT_MAX_TAPS = 512, 4096, 512, 16
 LOWRANK_FUNCTIONS = {"plain": 0, "sigmoid_power": 1, "softplus_decay": 2}
 
@@ -1206,12 +1237,19 @@ def embed_sinusoid(table, freq, scale: float, ctx, out) -> None:
 
 
 def matrix_state_scan(kind: str, q, k, v, state, ctx, y, n_heads: int, n_groups: int, rows: int, cols: int, *, q_scale: float,
-                      decay=None, s0=None, s1=None, cap: float = 0.0, den=None) -> None:
+                      decay=None, s0=None, s1=None, cap: float = 0.0, den=None, input_act: str = "none") -> None:
     """The recurrence of a step over every sequence's new tokens, from and into the state rows (see the kernel library's
     header): float32 q, k [T, groups·rows], v [T, heads·cols] (column ranges of wider rows will do), decay [T, heads·rows],
-    s0, s1 [T, heads or groups], state [slots, 2, state_row]; y [T, heads·cols], den [T, heads·2]."""
+    s0, s1 [T, heads or groups], state [slots, 2, state_row]; y [T, heads·cols], den [T, heads·2].  kind "fixed": decay float32
+    [heads]; input_act "silu": q, k and v go through x·sigmoid(x) first."""
     T = ctx.n_tokens
-    for name, t, n in (("q", q, n_groups * rows), ("k", k, n_groups * rows), ("v", v, n_heads * cols), ("decay", decay, n_heads * rows),
+    if input_act not in ("none", "silu"):
+        raise KernelError(f"matrix_state_scan: input activation '{input_act}' is neither 'none' nor 'silu'")
+    if kind == "fixed":
+        if decay is None or decay.numel() != n_heads:
+            raise KernelError("matrix_state_scan: one decay per head")
+        _dev(decay, "decay", torch.float32)
+    for name, t, n in (("q", q, n_groups * rows), ("k", k, n_groups * rows), ("v", v, n_heads * cols), ("decay", decay if kind != "fixed" else None, n_heads * rows),
                        ("s0", s0, n_heads), ("s1", s1, n_groups if kind == "delta" else n_heads), ("y", y, n_heads * cols),
                        ("den", den, 2 * n_heads)):
         if t is not None:
@@ -1221,11 +1259,11 @@ def matrix_state_scan(kind: str, q, k, v, state, ctx, y, n_heads: int, n_groups:
     _dev(state, "state", torch.float32)
     if state.dim() != 3 or state.shape[1] != 2 or (den is not None and den.stride(0) != 2 * n_heads):
         raise KernelError("matrix_state_scan: the state is [slots, 2, row] and the denominators are [T, heads·2]")
-    ld = lambda t: t.stride(0) if t is not None else 0   # noqa: E731
+    ld = lambda t: t.stride(0) if t is not None and t.dim() > 1 else 0   # noqa: E731
     call("vlrf_matrix_state_scan", MATRIX_STATE_KINDS[kind], _ptr(q), ld(q), _ptr(k), ld(k), _ptr(v), ld(v), _ptr(decay), ld(decay),
          _ptr(s0), ld(s0), _ptr(s1), ld(s1), float(q_scale), float(cap), _ptr(state), state.shape[2], _ptr(ctx.seq_slot),
          _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(y), ld(y), _ptr(den), ctx.n_seqs, ctx.max_new, n_heads, n_groups, rows, cols,
-         _stream())
+         GATE["silu"] if input_act == "silu" else 0, _stream())
 
 
 def conv_unit(proj, x_off: int, weight, state, conv_off: int, ctx, out, kq, n_heads: int, n_groups: int, rows: int, cols: int) -> None:

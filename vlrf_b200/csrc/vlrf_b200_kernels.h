@@ -92,7 +92,7 @@ int vlrf_gemm_tcgen05(const void* X, const void* W, const float* bias, const flo
 // The same kernel with a weight matrix per group.  offsets != null (device, G + 1 entries): rows offsets[g] …
 // offsets[g+1]−1 of X [rows][K] times W[g]ᵀ into the same rows of Y [rows][N] (experts over rows sorted by expert;
 // x_gs = y_gs = 0).  offsets == null: every group multiplies all rows, reading X at column g·x_gs and writing Y at
-// column g·y_gs (heads).  W [G][N][K]; an activation on the result (VLRF_ACT_NONE, _GELU_TANH, _RELU2); no bias,
+// column g·y_gs (heads).  W [G][N][K]; an activation on the result (VLRF_ACT_NONE, _GELU_TANH, _GELU_ERF, _RELU2); no bias,
 // residual or scatter.
 int vlrf_gemm_tcgen05_groups_takes(int rows, int G, int N, int K, int ldx, int x_gs, int ldy, int y_gs, int by_offsets);
 int vlrf_gemm_tcgen05_groups(const void* X, int ldx, int x_gs, const void* W, void* Y, int ldy, int y_gs, const int* offsets,
@@ -187,10 +187,10 @@ int vlrf_group_rmsnorm(const float* y, int ld_y, const int* rows, const float* w
                        int n_rows, int d, int groups, float eps, int accumulate, void* also_bf16, cudaStream_t stream);
 // n float32 numbers to out_dtype.
 int vlrf_cast_rows(const float* x, void* out, int out_dtype, long long n, cudaStream_t stream);
-// out[r][c] = act(a[r][c]) · b[r][c], act VLRF_ACT_SILU, VLRF_ACT_SIGMOID, VLRF_ACT_RELU or VLRF_ACT_GELU_TANH, each with a row stride of its own (out may be
+// out[r][c] = act(a[r][c]) · b[r][c] · factor, act VLRF_ACT_SILU, VLRF_ACT_SIGMOID, VLRF_ACT_RELU or VLRF_ACT_GELU_TANH, each with a row stride of its own (out may be
 // a or b).  Dtypes (a, b → out): all bfloat16; all float32; float32, bfloat16 → bfloat16; float32, float32 → bfloat16.
 int vlrf_gate_mul(const void* a, int lda, int a_dtype, const void* b, int ldb, int b_dtype, void* out, int ldo, int out_dtype,
-                  int rows, int cols, int act, cudaStream_t stream);
+                  int rows, int cols, int act, float factor, cudaStream_t stream);
 // The same with one column of a for every `per` consecutive columns of b: out[r][c] = act(a[r][c / per]) · b[r][c] (a gate
 // per head on the merged heads); cols a multiple of per.
 int vlrf_gate_mul_groups(const void* a, int lda, int a_dtype, const void* b, int ldb, int b_dtype, void* out, int ldo, int out_dtype,
@@ -255,10 +255,11 @@ int vlrf_qkv_rope_append(const float* proj, int ld, int q_off, int k_off, int v_
 // of dk entries for all heads; norm 2: all heads of the projection as one row, weights of H·dk and Hkv·dk entries; 0: none),
 // the pairing of rotated entries (0: entry i with i + rot/2; 1: entry 2i with 2i + 1) and a factor on every cosine and
 // sine.  Values are read as projected, so v_off = k_off keeps the keys from before norm and rotation as values.  With
-// write_cache = 0 the key and value columns are not read.
+// write_cache = 0 the key and value columns are not read.  maps 2: every query and key head is two maps of dk entries side by
+// side, each rotated (and normed) like a head of its own; the cache's key rows hold both, [block][Hkv][BT][2·dk].
 int vlrf_qkv_norm_rope_append(const float* proj, int ld, int q_off, int k_off, int v_off, const float* freq, int rot, void* q_out,
                               int ldq, void* Kc, void* Vc, int dtype, const int* block_table, int max_blocks, const int* tok_slot,
-                              const int* tok_pos, int T, int H, int Hkv, int dk, int dv, int BT, int write_cache, int norm,
+                              const int* tok_pos, int T, int H, int Hkv, int dk, int dv, int BT, int maps, int write_cache, int norm,
                               const float* q_norm, const float* k_norm, float eps, int pairing, float magnitude, int* dev_err,
                               cudaStream_t stream);
 // out[t][h·dv …] = out_scale · softmax over the visible keys of (q·k · scale) · V: a token sees the keys of its slot at
@@ -270,11 +271,13 @@ int vlrf_attn_window(const void* q, int dtype, int ldq, const void* Kc, const vo
 // positions below keep_first visible whatever the window, and sink (null, or a float32 per query head): exp(sink[h])
 // is one more term of the softmax's denominator, with nothing in the numerator.  gate (null, or float32 [T][ld_gate], a logit
 // per query head): head h's result is multiplied by sigmoid(gate[t][h]).  slopes (null, or a float32 per query head): slope ·
-// (query position − key position) is taken off every score, behind the cap.
+// (query position − key position) is taken off every score, behind the cap.  maps 2 (differential attention; no sink, no gate): a
+// query and a key head are two maps of dk numbers side by side, each a softmax of its own over the same values, and with
+// o = a₁ − map_factor · a₂ the head's result is out_scale · o / sqrt(mean(o²) + head_eps); maps 1: the last two are not read.
 int vlrf_attn_window_ex(const void* q, int dtype, int ldq, const void* Kc, const void* Vc, const int* block_table, int max_blocks,
                         const int* tok_slot, const int* tok_pos, void* out, int ld_out, int T, int H, int Hkv, int dk, int dv, int BT,
                         float scale, int window, float out_scale, float softcap, int keep_first, const float* sink, const float* gate,
-                        int ld_gate, const float* slopes, int* dev_err, cudaStream_t stream);
+                        int ld_gate, const float* slopes, int maps, float map_factor, float head_eps, int* dev_err, cudaStream_t stream);
 
 // The same attention on the tensor cores (attention_window_mma.cu; bfloat16): a CTA per key/value head, sequence and tile
 // of 64 (token, query head) rows, for prompt steps (rows seq_start[i] … of q are sequence i's new tokens, the first at
@@ -285,12 +288,13 @@ int vlrf_attn_window_mma(const void* q, int ldq, const void* Kc, const void* Vc,
                          const int* seq_slot, const int* seq_start, const int* seq_pos0, void* out, int ld_out, float* partials,
                          int n_seqs, int max_new, int H, int Hkv, int dk, int dv, int BT, float scale, int window, float out_scale,
                          int n_split, int* dev_err, cudaStream_t stream);
-// … with the cap, the kept first keys, the sinks, the gate per head and the slopes of vlrf_attn_window_ex.
+// … with the cap, the kept first keys, the sinks, the gate per head, the slopes and the two maps of vlrf_attn_window_ex (scratch for
+// cut contexts: rows · H · maps · n_split · (dv + 2) numbers).
 int vlrf_attn_window_mma_ex(const void* q, int ldq, const void* Kc, const void* Vc, const int* block_table, int max_blocks,
                             const int* seq_slot, const int* seq_start, const int* seq_pos0, void* out, int ld_out, float* partials,
                             int n_seqs, int max_new, int H, int Hkv, int dk, int dv, int BT, float scale, int window, float out_scale,
                             int n_split, float softcap, int keep_first, const float* sink, const float* gate, int ld_gate,
-                            const float* slopes, int* dev_err, cudaStream_t stream);
+                            const float* slopes, int maps, float map_factor, float head_eps, int* dev_err, cudaStream_t stream);
 
 // ---- a state-space recurrence with a matrix state per head (ssd.cu) ----------------------------------------------------------
 // What a sequence keeps lies in `state`, float32 [slots][2][state_row]: per copy the heads' states [H][N][P] and, at
@@ -314,13 +318,15 @@ int vlrf_ssd_gate_norm(const float* y, const float* proj, int ld, int z_off, con
 
 // ---- recurrences with a matrix state per head (matrix_state.cu, matrix_state_rows.cu) ----------------------------------------
 // kind 0: S ← diag(a) S + k vᵀ; kind 1: S ← diag(a) S, u = sigmoid(s0)(v − Sᵀk), S ← S + k uᵀ (s1: k · q per group); kind 2: the
-// memory with exponential gates and a running maximum (s0, s1: raw input and forget gate logits, capped by `cap`).  o = Sᵀ q ·
+// memory with exponential gates and a running maximum (s0, s1: raw input and forget gate logits, capped by `cap`); kind 3:
+// S ← a S + k vᵀ with one number a per head, the same for every token (decay float32 [H]).  input_act VLRF_ACT_SILU: q, k and v go
+// through x·sigmoid(x) first (VLRF_ACT_NONE: as they are; kind 3 only).  o = Sᵀ q ·
 // q_scale into y [T][H·V]; kind 2 also (n · q · q_scale, exp(−m)) into den [T][H][2].  q, k [T][G·K], v [T][H·V], decay a [T][H·K]
 // float32 (column ranges of wider rows will do).  state float32 [slots][2][state_row], see the source for its layout.
 int vlrf_matrix_state_scan(int kind, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* decay,
                            int ld_decay, const float* s0, int ld_s0, const float* s1, int ld_s1, float q_scale, float cap, float* state,
                            int state_row, const int* seq_slot, const int* seq_start, const int* seq_pos0, float* y, int ldy, float* den,
-                           int n_seqs, int max_new, int H, int G, int K, int V, cudaStream_t stream);
+                           int n_seqs, int max_new, int H, int G, int K, int V, int input_act, cudaStream_t stream);
 int vlrf_matrix_state_force(int columns, int warps);    // for measurements and tests: columns a lane, warps a CTA (0: chosen)
 // Convolution, x·sigmoid(x) and unit norms of q and k over columns [q: G·K | k: G·K | v: H·V] of the float32 rows `proj`; out
 // [T][2·G·K + H·V]; kq [T][G] = k · q; the kept inputs lie at conv_off of the state rows.
@@ -353,22 +359,23 @@ int vlrf_gemm_grouped(const void* X, const void* W, void* Y, const int* offsets,
 // The cache of one layer is [n_blocks][BT][row_w] of `dtype`: per token a row [c | r], the normed latent (C numbers)
 // and a rotated key part shared by all heads (R numbers, R may be 0).  Rotation: of the first rot_dims entries, entry
 // i pairs with entry i + rot_dims/2 (interleaved != 0: entry 2i with entry 2i + 1); angle = position · inv_freq[i]
-// (float32 table of rot_dims/2 entries).
+// (float32 table of rot_dims/2 entries); cosines and sines are multiplied by magnitude.
 // proj: float32 [T][ld], columns 0…C−1 the latent before its RMS norm (weight norm_w, eps), C…C+R−1 the key part
 // before its rotation; the token's row is written at (tok_slot, tok_pos).
 int vlrf_latent_append(const float* proj, int ld, int C, int R, const float* norm_w, float eps, const float* inv_freq,
-                       int rot_dims, int interleaved, void* cache, int dtype, int row_w, const int* block_table, int max_blocks,
+                       int rot_dims, int interleaved, float magnitude, void* cache, int dtype, int row_w, const int* block_table, int max_blocks,
                        const int* tok_slot, const int* tok_pos, int T, int BT, int* dev_err, cudaStream_t stream);
 // q: float32 [T][ld_q], per head [dim | R].  qn [T][ld_qn]: the heads' first dim columns, compact; qp [T][ld_qp]:
 // per head a row of C + R columns whose last R receive the rotated part (the first C are left for vlrf_gemm_heads).
-int vlrf_latent_q_rows(const float* q, int ld_q, int H, int dim, int R, const float* inv_freq, int rot_dims, int interleaved, const int* tok_pos,
+int vlrf_latent_q_rows(const float* q, int ld_q, int H, int dim, int R, const float* inv_freq, int rot_dims, int interleaved, float magnitude, const int* tok_pos,
                        void* qn, int ld_qn, void* qp, int ld_qp, int C, int dtype, int T, cudaStream_t stream);
 // qp [T][ld_q]: per head C + R numbers (the query in latent space, then its rotated part).  out [T][ld_out]: per head
 // the C numbers Σ_j p_j c_j with p = softmax_j((qp_h · row_j) · scale) over the visible rows j ≤ position (and, with
-// window > 0, position − j < window).  Any mix of tokens; rows with slot −1 get zeros.  C ≤ 1024.
+// window > 0, position − j < window), times out_scale.  sink (null, or a float32 per head): exp(sink[h]) is one more term of the
+// softmax's denominator.  Any mix of tokens; rows with slot −1 get zeros.  C ≤ 1024.
 int vlrf_attn_latent(const void* qp, int dtype, int ld_q, const void* cache, int row_w, int C, int R, const int* block_table,
                      int max_blocks, const int* tok_slot, const int* tok_pos, void* out, int ld_out, int T, int H, int BT,
-                     float scale, int window, int* dev_err, cudaStream_t stream);
+                     float scale, int window, const float* sink, float out_scale, int* dev_err, cudaStream_t stream);
 // The cache rows of the step's tokens as plain matrices: out_c [T][C] (latents) and out_r [T][R] (rotated key parts; null
 // with R = 0); rows of padding tokens are zeros.
 int vlrf_latent_gather(const void* cache, int dtype, int row_w, int C, int R, const int* block_table, int max_blocks,
@@ -377,11 +384,12 @@ int vlrf_latent_gather(const void* cache, int dtype, int row_w, int C, int R, co
 // Prompt attention over keys and values in plain rows (attention_rows.cu; bfloat16, `mma.sync`), for steps whose
 // sequences all begin at their first token: sequence i is the rows seq_start[i] … seq_start[i+1]−1, positions from 0.
 // Queries and keys in two parts: per head qn, kn [T][H·dim]; with a shared key part qr [T][H·R], kr [T][≥ R] (R may be
-// 0).  score = (qn·kn + qr·kr)·scale over keys j ≤ i; v, out [T][H·vdim].  dim + R one of 32, 64, 96, 128, 192, 256.
+// 0).  score = (qn·kn + qr·kr)·scale over keys j ≤ i (window > 0: i − j < window);
+// v, out [T][H·vdim]; sink and out_scale as above.  dim + R one of 32, 64, 96, 128, 192, 256.
 int vlrf_attn_rows_takes(int dim, int R, int vdim, int ld_qn, int ld_qr, int ld_kn, int ld_kr, int ld_v, int ld_out);
 int vlrf_attn_rows(const void* qn, int ld_qn, const void* qr, int ld_qr, const void* kn, int ld_kn, const void* kr, int ld_kr,
                    const void* v, int ld_v, const int* seq_start, void* out, int ld_out, int n_seqs, int max_new, int H, int dim,
-                   int R, int vdim, float scale, cudaStream_t stream);
+                   int R, int vdim, float scale, int window, const float* sink, float out_scale, cudaStream_t stream);
 // The same on the tensor cores (`mma.sync`, bfloat16; attention_latent_mma.cu): a token's heads are the rows of the
 // MMAs, tiles of 32 cache rows lie in shared memory once for all heads.  Sequence i brings the rows seq_start[i] …
 // seq_start[i+1]−1 at positions seq_pos0[i] … of slot seq_slot[i] (−1: padding, zeros); max_new is the longest run.
@@ -394,7 +402,7 @@ int vlrf_attn_latent_mma_ctas_per_sm(int C, int R);     // decode CTAs an SM hol
 int vlrf_attn_latent_mma(const void* qp, int ld_q, const void* cache, int row_w, int C, int R, const int* block_table,
                          int max_blocks, const int* seq_slot, const int* seq_start, const int* seq_pos0, void* out, int ld_out,
                          int n_seqs, int max_new, int H, int BT, float scale, int window, int n_split, float* partials,
-                         int* dev_err, cudaStream_t stream);
+                         const float* sink, float out_scale, int* dev_err, cudaStream_t stream);
 
 // ---- routed experts (moe.cu) ---------------------------------------------------------------------------------------
 // z: float32 router logits [T][ld_z] (column E: the logit of a shared expert's gate, if shared_gate).  ids, wts, rank
@@ -407,8 +415,9 @@ int vlrf_moe_route(const float* z, int ld_z, int E, int top, int shared_gate, co
 // ties to the lower index everywhere) and weighs the chosen by s · scale.  The last n_identity outputs stand for
 // experts without matrices that return their input: such a pair gets ids −2 and no row (padding rows: −1); counts
 // int32 [E − n_identity], zero before.  top ≤ keep · E / groups.  scoring 1: s = sigmoid(z), each output by itself.
+// renormalize: a chosen score is divided by (the sum of the chosen scores + 1e-20) before the scale.
 int vlrf_moe_route_scored(const float* z, int ld_z, int E, int top, int groups, int keep, int n_identity, float scale,
-                          int scoring, const float* correction, const int* tok_slot, int* ids, float* wts, int* rank, int* counts, int T,
+                          int scoring, int renormalize, const float* correction, const int* tok_slot, int* ids, float* wts, int* rank, int* counts, int T,
                           cudaStream_t stream);
 // offsets[e] = Σ counts[< e], E + 1 entries; counts are left zero.
 int vlrf_moe_plan(int* counts, int* offsets, int E, cudaStream_t stream);

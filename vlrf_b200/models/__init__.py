@@ -5,3 +5,4 @@ from . import kotisun  # noqa: F401
 from . import rakelorn  # noqa: F401
 from . import suposun  # noqa: F401
 from . import pelenex  # noqa: F401
+from . import vilodra  # noqa: F401

@@ -68,7 +68,9 @@ class GatedMLP:
     fuses_norm = False
     leaves_row_stats = False
 
-    def __init__(self, w_gate, w_up, w_down, *, activation: str):
+    def __init__(self, w_gate, w_up, w_down, *, activation: str, out_factor: float = 1.0):
+        """out_factor: a factor on everything the part adds, taken at the gate."""
+        self.out_factor = float(out_factor)
         if activation not in GATES:
             raise ValueError(f"GatedMLP: gate '{activation}' is not one of {', '.join(GATES)}")
         if w_gate.shape != w_up.shape or w_down.shape[1] != w_gate.shape[0] or w_down.shape[0] != w_gate.shape[1]:
@@ -82,7 +84,7 @@ class GatedMLP:
 
     def core(self, proj, merged, ctx: StepContext, h=None) -> None:
         ff = self.inner
-        ops.gate_mul(proj[:, :ff], proj[:, ff:2 * ff], merged, self.activation, ctx.n_tokens, ff)
+        ops.gate_mul(proj[:, :ff], proj[:, ff:2 * ff], merged, self.activation, ctx.n_tokens, ff, factor=self.out_factor)
 
     def forward(self, h, x: torch.Tensor, ctx: StepContext, norm=None, accumulate: bool = True) -> None:
         T, ff = ctx.n_tokens, self.inner

@@ -13,7 +13,11 @@ head).  That is the same arithmetic with the sums taken in another order.
 What is a parameter: how queries are made (directly, h·W_qᵀ, or through a latent of their own, RMSnorm(h·W_dqᵀ)·W_uqᵀ);
 the rotated part and its rotation (a position part that acts on q/k, with the pairing it names, or none); a sigmoid
 gate on the merged heads (W_g, from the same input: a row per merged column, or a row per head); whether the layer owns a cache row (W_dkv and its norm) or reads another layer's, as the
-model's schedule says (`writes_cache=False`: it then has no W_dkv and uses the rows as they lie in the cache).
+model's schedule says (`writes_cache=False`: it then has no W_dkv and uses the rows as they lie in the cache); a sliding
+window (position i sees j with i − j < window); a sink per head (one more term exp(sink_h) in the softmax's denominator, with
+nothing in the numerator); `out_factor`, a factor on everything the mixer adds to the residual.  Layers that share a cache
+may have windows of their own: `cache_window` is then what all of them must keep (the widest; 0: every row), the same
+number in each.
 Norms, rotation angles, scores and softmax are float32; products take operands in the activation dtype.
 """
 from __future__ import annotations
@@ -30,7 +34,8 @@ from .registry import register_part
 class LatentAttention:
     def __init__(self, *, n_heads: int, dim: int, vdim: int, kv_rank: int, rot_dim: int = 0, scale: float,
                  w_uk, w_uv, w_out, w_q=None, w_dq=None, dq_norm=None, w_uq=None, w_dkv=None, dkv_norm=None,
-                 w_gate=None, rotary=None, eps: float = 1e-5, window: int = 0):
+                 w_gate=None, rotary=None, eps: float = 1e-5, window: int = 0, cache_window: int | None = None, sink=None,
+                 out_factor: float = 1.0):
         H, C, R = int(n_heads), int(kv_rank), int(rot_dim)
         per_q = dim + R
         if (w_q is None) == (w_dq is None):
@@ -57,6 +62,13 @@ class LatentAttention:
             raise ValueError(f"latent attention: a latent of {C} numbers is wider than the {ops.LATENT_MAX_RANK} the kernels hold")
         self.n_heads, self.dim, self.vdim, self.kv_rank, self.rot_dim = H, int(dim), int(vdim), C, R
         self.scale, self.eps, self.window = float(scale), float(eps), int(window)
+        self.cache_window = self.window if cache_window is None else int(cache_window)
+        if self.window < 0 or self.cache_window < 0 or (self.cache_window > 0 and not 0 < self.window <= self.cache_window):
+            raise ValueError(f"latent attention: a cache that keeps {self.cache_window} rows does not serve a window of {self.window}")
+        if sink is not None and sink.numel() != H:
+            raise ValueError("latent attention: one sink per head")
+        self.sink = sink.float().contiguous() if sink is not None else None
+        self.out_factor = float(out_factor)
         self.w_q, self.w_dq, self.dq_norm, self.w_uq = w_q, w_dq, dq_norm, w_uq
         self.w_dkv, self.dkv_norm, self.w_gate, self.w_out = w_dkv, dkv_norm, w_gate, w_out
         self.rotary = rotary if R > 0 else None
@@ -81,8 +93,8 @@ class LatentAttention:
         self.w_in = torch.cat(parts, dim=0).contiguous() if parts else None
 
     def cache_need(self):
-        if self.window > 0:
-            return LatentNeed(self.kv_rank + self.rot_dim, "window", self.window)
+        if self.cache_window > 0:
+            return LatentNeed(self.kv_rank + self.rot_dim, "window", self.cache_window)
         return LatentNeed(self.kv_rank + self.rot_dim)
 
     fuses_norm = False
@@ -98,7 +110,7 @@ class LatentAttention:
         D = C + R
         inv_freq = self.rotary.inv_freq if self.rotary is not None else None
         rot_dims = self.rotary.dims if self.rotary is not None else 0
-        pairs = bool(getattr(self.rotary, "interleaved", False))
+        turn = dict(interleaved=bool(getattr(self.rotary, "interleaved", False)), magnitude=float(getattr(self.rotary, "magnitude", 1.0)))
         if writes_cache and self.w_dkv is None:
             raise ValueError("latent attention: a layer without W_dkv reads another layer's cache and cannot write one")
         # few rows (a decode step): the gate's logits ride in the same product, as float32; many rows: they are a
@@ -117,12 +129,12 @@ class LatentAttention:
 
         if writes_cache:
             ops.latent_append(cols("kv"), C, R, self.dkv_norm, self.eps, inv_freq, rot_dims, view.rows, view.block_table,
-                              ctx.tok_slot, ctx.tok_pos, T, ctx.dev_err, interleaved=pairs)
+                              ctx.tok_slot, ctx.tok_pos, T, ctx.dev_err, **turn)
         # A prompt step whose sequences all begin at position 0 holds every key and value it needs itself: they are
         # formed (two products of the step's latents) and attended as plain rows, which takes (dim + R) + vdim
         # multiplications per query, key and head instead of the latent-space form's (C + R) + C.  Every other step
         # (a prompt's later portions, decode steps, mixed steps) attends the cache rows in latent space.
-        as_rows = (ctx.max_new > 1 and self.window == 0 and len(ctx.host_seq_pos0) == ctx.n_seqs
+        as_rows = (ctx.max_new > 1 and len(ctx.host_seq_pos0) == ctx.n_seqs
                    and not any(ctx.host_seq_pos0) and ops.attention_rows_takes(act, dim, R, vdim, H))
         # queries: per head [dim | R]
         qp = ws.get("latent_qr", T, H * R, act) if as_rows and R > 0 else (None if as_rows else ws.get("latent_qp", T, H * D, act))
@@ -136,11 +148,11 @@ class LatentAttention:
             else:
                 q32 = ws.get("latent_q32", T, H * (dim + R), torch.float32)
                 ops.linear(cq, self.w_uq, None, q32)
-                ops.latent_q_rows(q32, H, dim, R, inv_freq, rot_dims, ctx.tok_pos, qn, qp, q_c, T, interleaved=pairs)
+                ops.latent_q_rows(q32, H, dim, R, inv_freq, rot_dims, ctx.tok_pos, qn, qp, q_c, T, **turn)
         elif R == 0:
             ops.linear(h, self.w_q, None, qn)
         else:
-            ops.latent_q_rows(cols("q"), H, dim, R, inv_freq, rot_dims, ctx.tok_pos, qn, qp, q_c, T, interleaved=pairs)
+            ops.latent_q_rows(cols("q"), H, dim, R, inv_freq, rot_dims, ctx.tok_pos, qn, qp, q_c, T, **turn)
         merged = ws.get("attn_out", T, H * vdim, act)
         if as_rows:
             rows_c = ws.get("latent_step_c", T, C, act)
@@ -148,12 +160,13 @@ class LatentAttention:
             ops.latent_gather(view.rows, C, R, view.block_table, ctx.tok_slot, ctx.tok_pos, rows_c, rows_r, T, ctx.dev_err)
             kv = ws.get("latent_keys_values", T, H * (dim + vdim), act)
             ops.linear(rows_c, self.w_ukv_rows, None, kv)
-            ops.attention_rows(qn, qp, kv[:, :H * dim], rows_r, kv[:, H * dim:], ctx.seq_start, merged, ctx.n_seqs, ctx.max_new, H, dim, R, vdim, self.scale)
+            ops.attention_rows(qn, qp, kv[:, :H * dim], rows_r, kv[:, H * dim:], ctx.seq_start, merged, ctx.n_seqs, ctx.max_new, H, dim, R, vdim, self.scale,
+                               window=self.window, sink=self.sink, out_scale=self.out_factor)
         else:
             ops.linear_heads(qn.view(T, H, dim), self.w_uk_t, qp.view(T, H, D)[:, :, :C], T)
             o = ws.get("latent_o", T, H * C, act)
             ops.attention_latent(qp, view.rows, C, R, view.block_table, ctx.tok_slot, ctx.tok_pos, o, T, H, self.scale,
-                                 self.window, ctx.dev_err, ctx=ctx)
+                                 self.window, ctx.dev_err, ctx=ctx, sink=self.sink, out_scale=self.out_factor)
             ops.linear_heads(o.view(T, H, C), self.w_uv, merged.view(T, H, vdim), T)
         if gate_apart:
             g = ws.get("latent_gate", T, H * vdim, act)

@@ -1,6 +1,6 @@
 """Recurrent mixers whose heads keep a matrix S of `dim` rows (key channels) by `vdim` columns (value channels).
 
-Three kinds, all float32 from the input product's results on (gates, decays, exponentials, norms, state):
+Four kinds, all float32 from the input product's results on (gates, decays, exponentials, norms, state):
 
   decayed_memory     a decay per key channel:  S ← diag(a) S + k vᵀ,  o = Sᵀ q
   delta_memory       the same decay, and a write that first takes out what the key already holds:
@@ -8,9 +8,11 @@ Three kinds, all float32 from the input product's results on (gates, decays, exp
   stabilized_memory  exponential input and forget gates per head with their running maximum m (which starts at 0) taken
                      out:  m' = max(f + m, i),  S ← e^(f + m − m') S + e^(i − m') k vᵀ,  n likewise with k alone,
                      o = Sᵀ q / (max(|n · q|, e^(−m')) + 1e-6)
+  fixed_memory       one decay per head, the same for every token:  S ← a S + k vᵀ,  o = Sᵀ q, with q, k and v through
+                     x·sigmoid(x)
 
-Behind the recurrence every head's o goes through an RMS norm of its own and a weight, is multiplied by a gate computed
-from the mixer's input, and the concatenated heads are projected.
+Behind the recurrence every head's o (in the fixed kind: all heads together) goes through an RMS norm of its own and a weight,
+is multiplied by a gate computed from the mixer's input, and the concatenated heads are projected.
 
 Per sequence a mixer keeps its heads' states (and m and n, or the last inputs of its convolution): one float32 row, held
 twice (`StateNeed((2, n))`; the kernels read the copy of the parity of the position a step begins at and write that of the
@@ -44,6 +46,7 @@ class MatrixStateMixer:
     fuses_norm = False
     leaves_row_stats = False
     in_bias = None
+    out_factor = 1.0            # a factor on everything the mixer adds to the residual
 
     def _sizes(self, what, n_heads, n_groups, dim, vdim, eps):
         self.n_heads, self.n_groups, self.dim, self.vdim, self.eps = int(n_heads), int(n_groups), int(dim), int(vdim), float(eps)
@@ -85,7 +88,7 @@ class MatrixStateMixer:
         proj = ctx.ws.get("matrix_state_in_proj", ctx.n_tokens, self.in_width, torch.float32)
         ops.linear(h, self.in_weight, self.in_bias, proj)
         merged = ctx.ws.get("matrix_state_merged", ctx.n_tokens, self.merged_width, ctx.act_dtype)
-        self.core(proj, merged, ctx, view, writes_cache)
+        self.core(proj, merged, ctx, view, writes_cache, self.out_factor)
         ops.linear(merged, self.out_weight, None, x, residual=x if accumulate else None)
 
 
@@ -196,3 +199,28 @@ class DeltaMemory(MatrixStateMixer):
         ops.matrix_state_scan("delta", qkv[:, :n], qkv[:, n:2 * n], qkv[:, 2 * n:], view.state, ctx, y, H, G, K, V, q_scale=K ** -0.5,
                               decay=decay, s0=cols(proj, "b"), s1=kq)
         ops.head_rows(y, self.norm_w, gate, "sigmoid", merged, T, H, V, self.eps, factor)
+
+
+@register_part("mixer", "fixed_memory")
+class FixedMemory(MatrixStateMixer):
+    """q = silu(W_q h), k = silu(W_k h), v = silu(W_v h); decay: one number per head; the concatenated heads normed as one row
+    (a weight of heads·vdim numbers) times sigmoid(W_g h).  The activation runs inside the recurrence's kernels."""
+
+    def __init__(self, w_q, w_k, w_v, w_g, norm_w, w_out, *, n_heads: int, dim: int, vdim: int, decay, eps: float, out_factor: float = 1.0):
+        what = "fixed memory"
+        self._sizes(what, n_heads, n_heads, dim, vdim, eps)
+        H, K, V = self.n_heads, self.dim, self.vdim
+        if len(decay) != H:
+            raise ValueError(f"{what}: {len(decay)} decays for {H} heads")
+        self._weights(what, [("q", w_q, H * K), ("k", w_k, H * K), ("v", w_v, H * V), ("g", w_g, H * V)], w_out, norm_w, (H * V,))
+        self.decay = torch.tensor([float(a) for a in decay], dtype=torch.float64).to(torch.float32).to(w_q.device).contiguous()
+        self.out_factor = float(out_factor)
+        self.state_numbers = H * K * V
+
+    def core(self, proj, merged, ctx: StepContext, view, writes_cache: bool = True, factor: float = 1.0) -> None:
+        self._own_state(writes_cache)
+        T, H, K, V, cols = ctx.n_tokens, self.n_heads, self.dim, self.vdim, self._columns_of
+        y = ctx.ws.get("matrix_state_y", T, H * V, torch.float32)
+        ops.matrix_state_scan("fixed", cols(proj, "q"), cols(proj, "k"), cols(proj, "v"), view.state, ctx, y, H, H, K, V, q_scale=1.0,
+                              decay=self.decay, input_act="silu")
+        ops.head_rows(y, self.norm_w, cols(proj, "g"), "sigmoid", merged, T, 1, H * V, self.eps, factor)

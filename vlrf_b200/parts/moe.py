@@ -5,12 +5,14 @@ lower index), weighted by the softmax over the chosen logits alone.  An expert i
 W_down (silu(W_gate h) · (W_up h)).  A shared expert of the same form, if there is one, runs for every token and is
 added, multiplied by sigmoid(w_sg · h), one number per token.
 
-What else is a parameter.  An expert without a gate (`w_gate=None`): W_down relu(W_up h)².  Routing by scores
+What else is a parameter.  An expert without a gate (`w_gate=None`): W_down act(W_up h), act the square of relu or one of the
+GELUs (`activation`).  Routing by scores
 (`scoring="softmax_all"`): s = softmax(z) over all router outputs; a token chooses by s + `correction` (a vector; the
 weights do not see it) among the outputs of the `keep` best of `groups` equal groups of neighbours, a group's score
 being its largest s + correction, and weighs the chosen by s · `weight_scale` without renormalizing.  Identity
 experts (`n_identity`): the router's last n_identity outputs stand for experts without matrices that return their
-input, so the router has n_identity more rows than there are expert matrices.  `scoring="sigmoid"`: the same rule with
+input, so the router has n_identity more rows than there are expert matrices.  `renormalize=True`: the chosen
+scores are divided by their sum (+ 1e-20) ahead of `weight_scale`.  `scoring="sigmoid"`: the same rule with
 s = sigmoid(z), each output by itself.  `gate="clamped"` (with `limit`, `gate_alpha`): an expert is
 W_down (g · sigmoid(gate_alpha · g) · (u + 1)) with g = min(W_gate h, limit) and u = clamp(W_up h, −limit, limit).
 `weights_on="input"`: the output is Σ expert(weight · h) instead of Σ weight · expert(h).
@@ -34,7 +36,8 @@ from .registry import register_part
 class RoutedExperts:
     def __init__(self, w_router, b_router, w_gate, w_up, w_down, *, top: int, shared=None, scoring: str = "softmax_chosen",
                  correction=None, groups: int = 1, keep: int = 1, weight_scale: float = 1.0, n_identity: int = 0,
-                 gate: str = "silu", limit: float | None = None, gate_alpha: float = 1.0, weights_on: str = "output"):
+                 gate: str = "silu", limit: float | None = None, gate_alpha: float = 1.0, weights_on: str = "output",
+                 activation: str = "relu2", renormalize: bool = False):
         """w_router [E + n_identity, width], b_router [E + n_identity] float32 or None; w_gate (or None), w_up [E, ff, width],
         w_down [E, width, ff]; shared: None or (w_gate [ffs, width], w_up [ffs, width], w_down [width, ffs], w_sg [1, width]
         or None); correction: float32 [E + n_identity] or None."""
@@ -54,7 +57,11 @@ class RoutedExperts:
             raise ValueError("routed experts: the experts' gate is 'silu', or 'clamped' with gate matrices and a positive limit")
         if weights_on not in ("output", "input") or (weights_on == "input" and n_identity):
             raise ValueError("routed experts: a weight multiplies an expert's 'output' or its 'input' (and then no expert is the identity)")
-        self.weights_on = weights_on
+        if activation not in ("relu2", "gelu_tanh", "gelu_erf"):
+            raise ValueError(f"routed experts: the activation of an expert without a gate is none of relu2, gelu_tanh, gelu_erf: '{activation}'")
+        if renormalize and scoring == "softmax_chosen":
+            raise ValueError("routed experts: the softmax over the chosen sums to one already")
+        self.weights_on, self.activation, self.renormalize = weights_on, activation, bool(renormalize)
         self.gate, self.limit, self.gate_alpha = gate, float(limit) if limit is not None else 0.0, float(gate_alpha)
         if scoring == "softmax_chosen" and (n_identity or correction is not None or groups != 1 or weight_scale != 1.0):
             raise ValueError("routed experts: identity experts, a correction, groups and a weight scale belong to scoring 'softmax_all'")
@@ -174,7 +181,8 @@ class RoutedExperts:
         offsets = ws.get("moe_offsets", 1, max(E, 1) + 1, torch.int32)
         if self.scoring != "softmax_chosen":
             ops.moe_route_scored(z, self.n_outputs, top, self.groups, self.keep, self.n_identity, self.weight_scale, self.correction,
-                                 ctx.tok_slot, ids, wts, rank, counts, T, scoring="sigmoid" if self.scoring == "sigmoid" else "softmax")
+                                 ctx.tok_slot, ids, wts, rank, counts, T, scoring="sigmoid" if self.scoring == "sigmoid" else "softmax",
+                                 renormalize=self.renormalize)
         else:
             ops.moe_route(z, E, top, self.shared_gate, ctx.tok_slot, ids, wts, rank, gate, counts, T)
         ops.moe_plan(counts, offsets, max(E, 1))
@@ -192,7 +200,7 @@ class RoutedExperts:
                 else:
                     ops.gate_mul(u[:, :ff], u[:, ff:], a, "silu", P, ff)
             else:
-                ops.linear_grouped(rows, self.w_gate_up, a, offsets, P, act="relu2")     # (the activation in the product's epilogue)
+                ops.linear_grouped(rows, self.w_gate_up, a, offsets, P, act=self.activation)     # (the activation in the product's epilogue)
             ops.linear_grouped(a, self.w_down, out, offsets, P)
         residual = x if accumulate else None
         if self.n_identity:

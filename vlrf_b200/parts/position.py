@@ -52,12 +52,15 @@ class RotaryPositions:
     slow pairs instead: with n(t) = dims · ln(original / (2π t)) / (2 ln base) the (real-valued) index of the pair that
     turns t times over `original` positions, lo = max(⌊n(fast)⌋, 0), hi = min(⌈n(slow)⌉, dims − 1) and
     r_i = clamp((i − lo) / max(hi − lo, 0.001), 0, 1), the frequency is f_i / factor · r_i + f_i · (1 − r_i), and every
-    cosine and sine is multiplied by `magnitude` = 0.1 · ln(factor) + 1.  The part holds the table f (float32, made
+    cosine and sine is multiplied by `magnitude` = 0.1 · ln(factor) + 1.  `wavelengths` = (factor, low, high, original) slows by
+the wavelength l = 2π / f instead: a frequency stays where l < original / high, becomes f / factor where l > original / low, and
+between the two, with s = (original / l − low) / (high − low), is (1 − s) · f / factor + s · f.  The part holds the table f (float32, made
     in 64-bit); the mixer that is given the part applies it inside its own kernels, with angles in float32."""
 
     where = "qk"
 
-    def __init__(self, base: float, dims: int, device, scaling_factor: float = 1.0, pairing: str = "half", yarn=None):
+    def __init__(self, base: float, dims: int, device, scaling_factor: float = 1.0, pairing: str = "half", yarn=None,
+                 wavelengths=None):
         if pairing not in ("half", "interleaved"):
             raise ValueError(f"RotaryPositions: pairing '{pairing}' is neither 'half' nor 'interleaved'")
         self.pairing, self.interleaved = pairing, pairing == "interleaved"
@@ -82,5 +85,22 @@ class RotaryPositions:
             ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(half)]
             f = [fi / factor * r + fi * (1.0 - r) for fi, r in zip(f, ramp)]
             self.magnitude = 0.1 * math.log(factor) + 1.0
+        self.wavelengths = None
+        if wavelengths is not None:
+            import math
+            factor, low, high, original = (float(v) for v in wavelengths)
+            if yarn is not None or not (factor > 0.0 and original > 0.0 and 0.0 < low < high):
+                raise ValueError(f"RotaryPositions: a scaling by wavelength of {wavelengths} goes without another and with 0 < low < high")
+            self.wavelengths = (factor, low, high, original)
+
+            def stretched(fi):
+                length = 2.0 * math.pi / fi
+                if length < original / high:
+                    return fi
+                if length > original / low:
+                    return fi / factor
+                s = (original / length - low) / (high - low)
+                return (1.0 - s) * fi / factor + s * fi
+            f = [stretched(fi) for fi in f]
         f = torch.tensor(f, dtype=torch.float64)
         self.inv_freq = f.to(torch.float32).to(device).contiguous()

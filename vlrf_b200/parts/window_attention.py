@@ -23,6 +23,11 @@ What else is a parameter, each absent by default:
   slopes [heads]           a distance bias: slopes_h · (i − j) is taken off every score (behind the cap, ahead of the softmax)
   w_gate [heads, width]    head h's result is multiplied by sigmoid(w_gate_h · input) ahead of the output projection; the
                            gate's logits ride in the input product as `heads` more float32 columns
+  second_map (f, eps)      differential attention: every query and key head is two maps of `dim` entries side by side (W_q
+                           [heads·2·dim, width], W_k [kv_heads·2·dim, width]), each rotated like a head and each a softmax of its
+                           own over the same values; with o = a₁ − f · a₂ the head's result is o / sqrt(mean(o²) + eps).  Goes
+                           without sinks and gates
+  out_factor               a factor on everything the mixer adds to the residual, taken where the heads' results are written
 
 The mixer is written in three stages so that another mixer can run it beside a second branch on the same input:
 `in_weight` / `in_bias` (the rows of the input product), `core(proj, merged, …, factor)` (from the product's float32
@@ -43,7 +48,8 @@ class WindowAttention:
     def __init__(self, w_q, w_k, w_v, w_out, *, n_heads: int, n_kv_heads: int, dim: int, vdim: int, scale: float,
                  b_q=None, b_k=None, b_v=None, window: int = 0, rotary=None, qk_norm: str | None = None, q_norm=None, k_norm=None,
                  norm_eps: float = 0.0, softcap: float | None = None, keep_first: int = 0, sink=None, w_gate=None,
-                 slopes=None):
+                 slopes=None, second_map: tuple | None = None, out_factor: float = 1.0):
+        maps = 2 if second_map is not None else 1
         H, G = int(n_heads), int(n_kv_heads)
         if H <= 0 or G <= 0 or H % G != 0:
             raise ValueError(f"window attention: {H} heads cannot share {G} key/value heads")
@@ -52,9 +58,12 @@ class WindowAttention:
             raise ValueError("window attention: values of its own need keys of its own")
         if self.values_are_keys and vdim != dim:
             raise ValueError(f"window attention: values that are the keys have their size ({dim}), not {vdim}")
-        if tuple(w_q.shape)[0] != H * dim or (w_k is not None and tuple(w_k.shape)[0] != G * dim) \
+        if tuple(w_q.shape)[0] != H * maps * dim or (w_k is not None and tuple(w_k.shape)[0] != G * maps * dim) \
                 or (w_v is not None and tuple(w_v.shape)[0] != G * vdim):
-            raise ValueError("window attention: W_q is [heads·dim, width], W_k [kv_heads·dim, width], W_v [kv_heads·vdim, width]")
+            raise ValueError("window attention: W_q is [heads·dim, width], W_k [kv_heads·dim, width], W_v [kv_heads·vdim, width]"
+                             + (" with twice the rows in W_q and W_k for two maps" if maps == 2 else ""))
+        if maps == 2 and (sink is not None or w_gate is not None or self.values_are_keys or not second_map[1] > 0.0):
+            raise ValueError("window attention: two maps a head go without sinks and gates, with values of their own and a positive eps")
         if w_out.shape[1] != H * vdim:
             raise ValueError("window attention: the output projection does not take the merged heads")
         if max(dim, vdim) > ops.WINDOW_HEAD_MAX:
@@ -72,7 +81,7 @@ class WindowAttention:
         if qk_norm is not None:
             if qk_norm == "head" and q_norm is None and k_norm is None:      # a norm without weights
                 q_norm = k_norm = torch.ones(dim, dtype=torch.float32, device=w_q.device)
-            nq, nk = (dim, dim) if qk_norm == "head" else (H * dim, G * dim)
+            nq, nk = (dim, dim) if qk_norm == "head" else (H * maps * dim, G * maps * dim)
             if q_norm is None or q_norm.numel() != nq or (self.own_kv and (k_norm is None or k_norm.numel() != nk)) or not norm_eps > 0.0:
                 raise ValueError("window attention: the norm of queries and keys needs its weights and a positive eps")
         if sink is not None and sink.numel() != H:
@@ -95,10 +104,12 @@ class WindowAttention:
         self.softcap, self.keep_first = float(softcap) if softcap is not None else 0.0, int(keep_first)
         self.sink = sink.float().contiguous() if sink is not None else None
         self.slopes = slopes.float().contiguous() if slopes is not None else None
-        self.q_off, self.k_off = 0, H * dim
-        self.v_off = self.k_off if self.values_are_keys else H * dim + G * dim
-        width_kv = (G * dim if w_k is not None else 0) + (G * vdim if w_v is not None else 0)
-        self.gate_off = H * dim + width_kv if w_gate is not None else None
+        self.maps, self.out_factor = maps, float(out_factor)
+        self.second_map = (float(second_map[0]), float(second_map[1])) if second_map is not None else None
+        self.q_off, self.k_off = 0, H * maps * dim
+        self.v_off = self.k_off if self.values_are_keys else self.k_off + G * maps * dim
+        width_kv = (G * maps * dim if w_k is not None else 0) + (G * vdim if w_v is not None else 0)
+        self.gate_off = self.k_off + width_kv if w_gate is not None else None
         if w_gate is not None:
             weights.append(w_gate.to(w_q.dtype))
         self.in_weight = torch.cat(weights, dim=0).contiguous()
@@ -111,7 +122,8 @@ class WindowAttention:
         """Keys and values per token; a layer without projections of its own states the need of the cache it reads (the
         model checks that the two agree) and writes nothing."""
         kind = "window" if self.window > 0 else "full"
-        return KVNeed(self.n_kv_heads, self.dim, kind, self.window, v_dim=self.vdim if self.vdim != self.dim else 0,
+        k_dim = self.maps * self.dim               # (a key head's maps lie side by side)
+        return KVNeed(self.n_kv_heads, k_dim, kind, self.window, v_dim=self.vdim if self.vdim != k_dim else 0,
                       keep_first=self.keep_first)
 
     fuses_norm = False
@@ -124,17 +136,17 @@ class WindowAttention:
         T, H, G = ctx.n_tokens, self.n_heads, self.n_kv_heads
         if writes_cache and not self.own_kv:
             raise ValueError("window attention: a layer without keys and values of its own must read another layer's cache")
-        q = ctx.ws.get("window_q", T, H * self.dim, ctx.act_dtype)
+        q = ctx.ws.get("window_q", T, H * self.maps * self.dim, ctx.act_dtype)
         freq = self.rotary.inv_freq if self.rotary is not None else None
         rot = self.rotary.dims if self.rotary is not None else 0
         ops.qkv_rope_append(proj, self.q_off, self.k_off, self.v_off, freq, rot, q, view.k, view.v, view.block_table, ctx.tok_slot,
                             ctx.tok_pos, T, H, G, self.dim, self.vdim, writes_cache and self.own_kv, ctx.dev_err, norm=self.qk_norm,
                             q_norm=self.q_norm, k_norm=self.k_norm, eps=self.norm_eps,
                             interleaved=bool(getattr(self.rotary, "interleaved", False)),
-                            magnitude=float(getattr(self.rotary, "magnitude", 1.0)))
+                            magnitude=float(getattr(self.rotary, "magnitude", 1.0)), maps=self.maps)
         ops.attention_window_step(q, view.k, view.v, view.block_table, merged, ctx, H, G, self.dim, self.vdim, self.scale,
-                                  self.window, factor, softcap=self.softcap, keep_first=self.keep_first, sink=self.sink,
-                                  slopes=self.slopes,
+                                  self.window, factor * self.out_factor, softcap=self.softcap, keep_first=self.keep_first, sink=self.sink,
+                                  slopes=self.slopes, second_map=self.second_map,
                                   # head h times sigmoid of its gate logit (a float32 column of the input product), applied by
                                   # the attention kernel where it writes the head's result
                                   gate=proj[:, self.gate_off:self.gate_off + H] if self.gate_off is not None else None)
