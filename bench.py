@@ -1252,9 +1252,189 @@ def pelenex_kernels(z: dict, hbm_gbs: float, bf16_tflops: float) -> dict:
     return out
 
 
+#: Vilodra at two sizes that resemble a real model's layers, beside a Rakelorn (its closest relative in the framework: latent
+#: attention, a recurrence, experts by scores without a gate) of the same width, depth, latent heads and sizes and experts.
+#: Vilodra's layers: latent attention + dense, differential attention + experts, latent attention reading the first layer's
+#: latents + dense, lightning recurrence + experts; Rakelorn's: latent attention, latent attention, minGRU, latent attention,
+#: all with experts.
+VILODRA_SIZES = {
+    "s": dict(width=1024, heads=16, dim=64, rot=32, vdim=64, kv_rank=256, q_rank=384, window=512, d_heads=8, d_kv=4, d_dim=64, d_vdim=128,
+              r_heads=8, r_dim=128, r_vdim=128, ff_gated=2816, experts=16, top=2, expert_ff=1024, gru=1024, vocab=32000),
+    "m": dict(width=2048, heads=16, dim=128, rot=64, vdim=128, kv_rank=512, q_rank=768, window=1024, d_heads=16, d_kv=4, d_dim=64, d_vdim=128,
+              r_heads=16, r_dim=128, r_vdim=128, ff_gated=5632, experts=32, top=4, expert_ff=1408, gru=2048, vocab=32000),
+}
+
+
+def vilodra_config(z: dict) -> dict:
+    def lat(kv_from=None):
+        m = {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot"], "vdim": z["vdim"], "kv_rank": z["kv_rank"], "scale": (z["dim"] + z["rot"]) ** -0.5,
+             "mask": {"size": z["window"]},
+             "rot": {"base": 10000.0, "dims": z["rot"], "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        if kv_from is not None:
+            m["kv_from"] = kv_from
+        return {"type": "latent_attention", "mixer": m}
+    diff = {"type": "attention", "mixer": {"heads": z["d_heads"], "kv_heads": z["d_kv"], "dim": z["d_dim"], "vdim": z["d_vdim"], "scale": z["d_dim"] ** -0.5,
+                                           "diff": 0.7, "rot": {"base": 500000.0, "dims": z["d_dim"],
+                                                                "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    n = z["r_heads"]
+    light = {"type": "lightning", "mixer": {"heads": n, "dim": z["r_dim"], "vdim": z["r_vdim"], "decay": [1.0 - 2.0 ** (-1.0 - 8.0 * h / n) for h in range(n)]}}
+    dense = {"kind": "dense", "ff": z["ff_gated"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"], "scale": 1.5}}
+    return {"architecture": "Vilodra", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.6,
+            "layers": [dict(lat(), mlp=dense), dict(diff, mlp=moe), dict(lat(0), mlp=dense), dict(light, mlp=moe)]}
+
+
+def rakelorn_config_like(z: dict) -> dict:
+    cfg = rakelorn_config(dict(z, identity=2, groups=2, keep=1))
+    att, gru = cfg["layers"][0], cfg["layers"][1]
+    del cfg["loop"]
+    return dict(cfg, layers=[att, att, gru, att])
+
+
+def vilodra_kernels(z: dict, hbm_gbs: float, bf16_tflops: float) -> dict:
+    """Vilodra's own kernels alone, each beside the like kernel that was there (20 launches replayed as one graph, inputs rotated over
+    more than L2 where a kernel is bound by bytes, cache blocks dealt at random): differential attention beside attention with
+    one map of the same sizes; latent attention with a window and sinks, in latent space and over plain rows, beside the same
+    reach without them; the preparation of queries and keys with two maps beside one; the recurrence with a fixed decay beside
+    Pelenex's with a decay per channel; the read-out of a whole row beside Pelenex's per head; the router, an expert's first
+    product and the gate beside those without renormalizing, with relu² and without a factor."""
+    import types
+    import torch
+    from vlrf_b200.csrc import ops
+    from vlrf_b200.parts.context import Workspace
+    dev, bf = "cuda", torch.bfloat16
+    width = z["width"]
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)   # noqa: E731
+
+    def timed(fn, reps=20):
+        for i in range(3):
+            fn(i)
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for i in range(reps):
+                fn(i)
+        graph.replay()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        graph.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / reps * 1e3
+
+    def bytes_point(us, nbytes, flops=0.0):
+        pt = {"us": round(us, 1), "gb_s": round(nbytes / us / 1e3, 1), "frac_hbm": round(nbytes / us / 1e3 / hbm_gbs, 3), "mib": round(nbytes / 2**20, 1)}
+        return dict(pt, tflops=round(flops / us / 1e6, 2)) if flops else pt
+
+    def flops_point(us, fl):
+        return {"us": round(us, 1), "tflops": round(fl / us / 1e6, 1), "frac_tensor": round(fl / us / 1e6 / bf16_tflops, 4)}
+
+    def rotated(make, nbytes):
+        """Enough tensors that together they exceed L2."""
+        return [make() for _ in range(max(2, min(64, int(300e6 // max(nbytes, 1)) + 1)))]
+
+    warm = torch.zeros(4096, 4096, device=dev)
+    t_end = time.time() + 0.2
+    while time.time() < t_end:
+        warm.add_(1.0)
+        torch.cuda.synchronize()
+    del warm
+    out = {}
+    S, L, B = 2, 1024, 64
+    err = torch.zeros(1, dtype=torch.int32, device=dev)
+
+    def step(n_seq, n_new, ctx_len):
+        return types.SimpleNamespace(n_tokens=n_seq * n_new, n_seqs=n_seq, max_new=n_new, max_context=ctx_len, ws=Workspace(dev), dev_err=err,
+                                     seq_slot=i32(list(range(n_seq))), seq_start=i32([i * n_new for i in range(n_seq + 1)]),
+                                     seq_pos0=i32([ctx_len - n_new] * n_seq), tok_slot=i32([s for s in range(n_seq) for _ in range(n_new)]),
+                                     tok_pos=i32([ctx_len - n_new + j for _ in range(n_seq) for j in range(n_new)]))
+    rnd = lambda *sh: torch.randn(*sh, device=dev)   # noqa: E731
+    for label, c in (("prompt", step(S, L, L)), ("decode", step(B, 1, L))):
+        T, n_seq, per = c.n_tokens, c.n_seqs, L // 64
+        pairs = n_seq * L * (L + 1) / 2
+        table = torch.randperm(n_seq * per, device=dev).to(torch.int32).view(n_seq, per).contiguous()
+        # -- differential attention ---------------------------------------------------------------------------------------------
+        H, G, dk, dv = z["d_heads"], z["d_kv"], z["d_dim"], z["d_vdim"]
+        for who, maps in (("vilodra", 2), ("one_map", 1)):
+            size = n_seq * per * G * 64 * (maps * dk + dv) * 2
+            caches = rotated(lambda: (rnd(n_seq * per, G, 64, maps * dk).to(bf), rnd(n_seq * per, G, 64, dv).to(bf)), size if label == "decode" else 2e8)
+            q, o = rnd(T, H * maps * dk).to(bf), torch.zeros(T, H * dv, dtype=bf, device=dev)
+            us = timed(lambda i: ops.attention_window_step(q, *caches[i % len(caches)], table, o, c, H, G, dk, dv, dk ** -0.5, 0, 1.0,
+                                                           second_map=(0.5, 1e-5) if maps == 2 else None))
+            out.setdefault("attention_" + label, {})[who] = bytes_point(us, size) if label == "decode" else flops_point(us, 2.0 * maps * pairs * H * (dk + dv))
+            n_in = (H + G) * maps * dk + G * dv
+            projs, freq = rotated(lambda: rnd(T, n_in), T * n_in * 4), torch.ones(dk // 2, device=dev)
+            us = timed(lambda i: ops.qkv_rope_append(projs[i % len(projs)], 0, H * maps * dk, (H + G) * maps * dk, freq, dk, q, *caches[0], table, c.tok_slot,
+                                                     c.tok_pos, T, H, G, dk, dv, True, err, interleaved=True, maps=maps))
+            out.setdefault("prepare_" + label, {})[who] = bytes_point(us, T * n_in * 6)
+            del caches, projs
+        # -- latent attention ------------------------------------------------------------------------------------------------------
+        H, C, R, dim, vdim, W = z["heads"], z["kv_rank"], z["rot"], z["dim"], z["vdim"], z["window"]
+        D, sink = C + R, torch.zeros(H, device=dev)
+        caches = rotated(lambda: rnd(n_seq * per, 64, D).to(bf), n_seq * per * 64 * D * 2 if label == "decode" else 2e8)
+        qp, o = rnd(T, H * D).to(bf), torch.zeros(T, H * C, dtype=bf, device=dev)
+        seen = sum(min(p + 1, W) for p in range(L)) * n_seq
+        short = step(n_seq, c.max_new, min(L, W)) if label == "decode" else c
+        for who, cc, kw, win in (("vilodra", c, dict(sink=sink, out_scale=0.6), W), ("plain", short, {}, 0)):
+            us = timed(lambda i: ops.attention_latent(qp, caches[i % len(caches)], C, R, table, cc.tok_slot, cc.tok_pos, o, T, H, 0.1, win, err, ctx=cc, **kw), reps=10)
+            out.setdefault("latent_" + label, {})[who] = bytes_point(us, n_seq * min(L, W) * D * 2) if label == "decode" else \
+                flops_point(us, 2.0 * (seen if win else pairs) * H * (dim + R + vdim))
+        if label == "prompt" and ops.attention_rows_takes(bf, dim, R, vdim, H):
+            qn, qr, kn, kr = (rnd(T, n).to(bf) for n in (H * dim, H * R, H * dim, R))
+            v, om = rnd(T, H * vdim).to(bf), torch.zeros(T, H * vdim, dtype=bf, device=dev)
+            for who, kw, n in (("vilodra", dict(window=W, sink=sink, out_scale=0.6), seen), ("plain", {}, pairs)):
+                us = timed(lambda i: ops.attention_rows(qn, qr, kn, kr, v, c.seq_start, om, n_seq, L, H, dim, R, vdim, 0.1, **kw), reps=10)
+                out.setdefault("latent_rows_prompt", {})[who] = flops_point(us, 2.0 * n * H * (dim + R + vdim))
+        del caches
+        # -- the recurrence and its read-out ---------------------------------------------------------------------------------------
+        H, K, V = z["r_heads"], z["r_dim"], z["r_vdim"]
+        row = H * K * V
+        states = rotated(lambda: torch.zeros(n_seq, 2, row, device=dev), n_seq * row * 8) if label == "decode" else [torch.zeros(n_seq, 2, row, device=dev)]
+        qkv, y = rnd(T, H * (2 * K + V)), torch.zeros(T, H * V, device=dev)
+        q, k, v = qkv[:, :H * K], qkv[:, H * K:2 * H * K], qkv[:, 2 * H * K:]
+        per_ch, fixed = torch.rand(T, H * K, device=dev) * 0.1 + 0.9, torch.full((H,), 0.99, device=dev)
+        fl = 2.0 * T * H * K * V * 2
+        us = timed(lambda i: ops.matrix_state_scan("fixed", q, k, v, states[i % len(states)], c, y, H, H, K, V, q_scale=1.0, decay=fixed, input_act="silu"), reps=10)
+        out["scan_" + label] = {"vilodra": bytes_point(us, n_seq * 2 * row * 4 + T * 2 * H * (K + V) * 4, fl)}
+        us = timed(lambda i: ops.matrix_state_scan("decayed", q, k, v, states[i % len(states)], c, y, H, H, K, V, q_scale=1.0, decay=per_ch), reps=10)
+        out["scan_" + label]["pelenex_decayed"] = bytes_point(us, n_seq * 2 * row * 4 + T * H * (3 * K + 2 * V) * 4, fl)
+        del states, qkv
+        ys, gs = rotated(lambda: rnd(T, H * V), T * H * V * 4), rotated(lambda: rnd(T, H * V), T * H * V * 4)
+        m = torch.zeros(T, H * V, dtype=bf, device=dev)
+        for who, heads, cols in (("vilodra", 1, H * V), ("per_head", H, V)):
+            w = torch.ones(H * V, device=dev)
+            us = timed(lambda i: ops.head_rows(ys[i % len(ys)], w, gs[i % len(gs)], "sigmoid", m, T, heads, cols, 1e-5))
+            out.setdefault("read_out_" + label, {})[who] = bytes_point(us, T * H * V * 10)
+        del ys, gs
+        # -- router, an expert's first product, the dense feed-forward's gate --------------------------------------------------------
+        E, top, ff = z["experts"], z["top"], z["expert_ff"]
+        P = T * top
+        zl, corr = rnd(T, E), torch.zeros(E, device=dev)
+        ids, rank, wts = (torch.zeros(T, top, dtype=dt, device=dev) for dt in (torch.int32, torch.int32, torch.float32))
+        counts = torch.zeros(E, dtype=torch.int32, device=dev)
+        for who, kw in (("vilodra", dict(renormalize=True)), ("as_they_are", {})):
+            us = timed(lambda i: (counts.zero_(), ops.moe_route_scored(zl, E, top, 1, 1, 0, 1.5, corr, None, ids, wts, rank, counts, T, **kw)))
+            out.setdefault("router_" + label, {})[who] = bytes_point(us, T * (E + 3 * top) * 4)
+        ws = rotated(lambda: (rnd(E, ff, width) * 0.02).to(bf), E * ff * width * 2)
+        x, u = rnd(P, width).to(bf), torch.zeros(P, ff, dtype=bf, device=dev)
+        offs = i32([P * e // E for e in range(E + 1)])
+        for who, act in (("vilodra", "gelu_erf"), ("relu2", "relu2")):
+            us = timed(lambda i: ops.linear_grouped(x, ws[i % len(ws)], u, offs, P, act=act))
+            out.setdefault("expert_up_" + label, {})[who] = flops_point(us, 2.0 * P * ff * width) if label == "prompt" else bytes_point(us, E * ff * width * 2)
+        del ws
+        fg = z["ff_gated"]
+        gus, a = rotated(lambda: rnd(T, 2 * fg), T * 2 * fg * 4), torch.zeros(T, fg, dtype=bf, device=dev)
+        for who, f in (("vilodra", 0.6), ("no_factor", 1.0)):
+            us = timed(lambda i: ops.gate_mul(gus[i % len(gus)][:, :fg], gus[i % len(gus)][:, fg:], a, "silu", T, fg, factor=f))
+            out.setdefault("gate_" + label, {})[who] = bytes_point(us, T * fg * 10)
+        del gus
+    return out
+
+
 def design_bench(args) -> int:
     """`--design NAME`: the design at sizes like a real model's layers (random weights) beside its closest existing
-    model of equal size (GPT-2; for Rakelorn and Suposun, Kuvusun; for Pelenex, Kotisun): prefill and decode throughput, and each kernel's time.  One JSON line."""
+    model of equal size (GPT-2; for Rakelorn and Suposun, Kuvusun; for Pelenex, Kotisun; for Vilodra, Rakelorn): prefill and decode throughput, and each kernel's time.  One JSON line."""
     import vlrf_b200.models  # noqa: F401
     from vlrf_b200.weights import write_random_model
     hbm_gbs, bf16_tflops, peak_src = peaks()
@@ -1264,9 +1444,10 @@ def design_bench(args) -> int:
                                     "kotisun": (KOTISUN_SIZES, kotisun_config, kotisun_kernels),
                                     "rakelorn": (RAKELORN_SIZES, rakelorn_config, rakelorn_kernels),
                                     "suposun": (SUPOSUN_SIZES, suposun_config, suposun_kernels),
-                                    "pelenex": (PELENEX_SIZES, pelenex_config, pelenex_kernels)}[args.design]
+                                    "pelenex": (PELENEX_SIZES, pelenex_config, pelenex_kernels),
+                                    "vilodra": (VILODRA_SIZES, vilodra_config, vilodra_kernels)}[args.design]
     beside, beside_of = {"rakelorn": ("kuvusun", kuvusun_config_like), "suposun": ("kuvusun", kuvusun_config),
-                         "pelenex": ("kotisun", kotisun_config_like)}.get(args.design, ("gpt2", gpt2_config_like))
+                         "pelenex": ("kotisun", kotisun_config_like), "vilodra": ("rakelorn", rakelorn_config_like)}.get(args.design, ("gpt2", gpt2_config_like))
     line["beside"] = beside
     for name in args.design_sizes.split(","):
         z = sizes[name]
@@ -1327,9 +1508,9 @@ def main() -> int:
                     help="with --only decode or prefill and VLRF_B200_KERNEL_TRACE=1: print where the last step's kernels spent their time")
     ap.add_argument("--only", default="all", choices=["all", "decode", "prefill"],
                     help="measure one part only and print a short line (for profiling runs); the full line needs 'all'")
-    ap.add_argument("--design", default=None, choices=["kuvusun", "kotisun", "rakelorn", "suposun", "pelenex"],
+    ap.add_argument("--design", default=None, choices=["kuvusun", "kotisun", "rakelorn", "suposun", "pelenex", "vilodra"],
                     help="instead of the default workload: this design at sizes like a real model's layers beside its closest "
-                         "existing model of equal size (GPT-2; for rakelorn and suposun, Kuvusun)")
+                         "existing model of equal size (GPT-2; for rakelorn and suposun, Kuvusun; for pelenex, Kotisun; for vilodra, Rakelorn)")
     ap.add_argument("--design-sizes", default="s,m", help="with --design: which of the sizes %s" % ",".join(DESIGN_SIZES))
     ap.add_argument("--design-no-kernels", action="store_true", help="with --design: whole steps only, not each kernel alone")
     ap.add_argument("--design-only-kernels", action="store_true", help="with --design: each kernel alone only")

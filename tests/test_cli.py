@@ -182,3 +182,25 @@ def test_run_generates_with_a_pelenex_model_what_the_plain_implementation_would(
                    "--dtype", "float32"], capsys)
     outputs = [line for prev, line in zip(out.splitlines(), out.splitlines()[1:]) if prev.startswith("--- Output")]
     assert [[int(t) for t in line.split()] for line in outputs] == [plain_pelenex.greedy_generate(cfg, w, p, 6) for p in ([5, 17, 3, 400, 44], [7])]
+
+
+def test_init_and_info_take_a_vilodra_preset(tmp_path, capsys):
+    run_cli(["init", "--config", "vilodra-tiny", "--out", str(tmp_path / "v"), "--seed", "3"], capsys)
+    info = run_cli(["info", "--model", str(tmp_path / "v")], capsys)
+    assert "architecture: Vilodra" in info
+    shown = json.loads(info[info.index("{"):info.rindex("}") + 1])
+    assert [layer["type"] for layer in shown["layers"]] == ["latent_attention", "lightning", "attention", "latent_attention"]
+    assert shown["residual_mult"] == 0.8 and shown["layers"][3]["mixer"]["kv_from"] == 0
+
+
+@pytest.mark.gpu
+def test_run_generates_with_a_vilodra_model_what_the_plain_implementation_would(tmp_path, capsys):
+    import plain_vilodra
+    run_cli(["init", "--config", "vilodra-tiny", "--out", str(tmp_path / "v"), "--seed", "3"], capsys)
+    cfg, w = plain_vilodra.read_model_dir(tmp_path / "v")
+    f = tmp_path / "prompts.txt"
+    f.write_text("5 17 3 400 44\n7\n")
+    out = run_cli(["run", "--model", str(tmp_path / "v"), "--prompts-file", str(f), "--tokens", "6", "--greedy", "--stop-id", "999",
+                   "--dtype", "float32"], capsys)
+    outputs = [line for prev, line in zip(out.splitlines(), out.splitlines()[1:]) if prev.startswith("--- Output")]
+    assert [[int(t) for t in line.split()] for line in outputs] == [plain_vilodra.greedy_generate(cfg, w, p, 6) for p in ([5, 17, 3, 400, 44], [7])]
