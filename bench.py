@@ -1399,6 +1399,11 @@ def vilodra_kernels(z: dict, hbm_gbs: float, bf16_tflops: float) -> dict:
         out["scan_" + label] = {"vilodra": bytes_point(us, n_seq * 2 * row * 4 + T * 2 * H * (K + V) * 4, fl)}
         us = timed(lambda i: ops.matrix_state_scan("decayed", q, k, v, states[i % len(states)], c, y, H, H, K, V, q_scale=1.0, decay=per_ch), reps=10)
         out["scan_" + label]["pelenex_decayed"] = bytes_point(us, n_seq * 2 * row * 4 + T * H * (3 * K + 2 * V) * 4, fl)
+        if label == "prompt":                       # in chunks on the tensor cores, beside the same token by token
+            out["scan_prompt"]["vilodra_token_by_token"] = out["scan_prompt"].pop("vilodra")
+            half = qkv.to(bf)
+            us = timed(lambda i: ops.fixed_state_chunks(half[:, :H * K], half[:, H * K:2 * H * K], half[:, 2 * H * K:], fixed, states[0], c, y, H, K, V), reps=10)
+            out["scan_prompt"]["vilodra"] = bytes_point(us, n_seq * 2 * row * 4 + T * H * (4 * K + 6 * V), fl)
         del states, qkv
         ys, gs = rotated(lambda: rnd(T, H * V), T * H * V * 4), rotated(lambda: rnd(T, H * V), T * H * V * 4)
         m = torch.zeros(T, H * V, dtype=bf, device=dev)

@@ -421,6 +421,92 @@ def test_fixed_memory_of_seventy_single_tokens():
         close(torch.cat(got[s]), plain_memory(seqs[s], decay, "silu"), 2e-5, f"sequence {s}")
 
 
+def chunk_step(d, decay, state, ctx, scale=1.0):
+    """One step in chunks from bfloat16 rows [q | k | v]; the scratch is NaN before."""
+    from vlrf_b200.csrc import ops
+    T, H, K = d["q"].shape
+    V = d["v"].shape[2]
+    n = H * (2 * K + V)
+    wide = dev(torch.cat([torch.full((T, 8), float("nan"), dtype=F64)] + [d[x].reshape(T, -1) for x in "qkv"], 1), torch.bfloat16)[:, 8:]
+    ctx.ws.get("fixed_state_chunks", (T // 64 + ctx.n_seqs) * H, K * V, torch.float32).fill_(float("nan"))
+    y = torch.full((T, H * V), float("nan"), device="cuda")
+    assert wide.shape[1] == n and ops.fixed_state_chunks_takes(torch.bfloat16, types.SimpleNamespace(max_new=64, n_tokens=T, n_seqs=ctx.n_seqs), H, K, V, state.shape[2])
+    ops.fixed_state_chunks(wide[:, :H * K], wide[:, H * K:2 * H * K], wide[:, 2 * H * K:], dev(decay, torch.float32), state, ctx, y, H, K, V, q_scale=scale)
+    return y.view(T, H, V)
+
+
+@pytest.mark.parametrize("H,K,V", [(2, 16, 16), (3, 24, 40), (1, 128, 128), (5, 64, 64), (2, 72, 136), (1, 256, 32), (6, 8, 8), (3, 48, 264), (2, 136, 96)])
+def test_fixed_memory_in_chunks(H, K, V):
+    """Nine sequences at and around the chunks' edges in one step, twice (the second step goes on from states at odd and even
+    positions), a padding sequence among them; then the token-by-token kernel goes on from the states that the chunks left."""
+    from vlrf_b200.parts.context import Workspace
+    lens = [1, 63, 64, 65, 127, 128, 129, 200, 33]
+    more = [64, 1, 130, 2, 65, 63, 7, 128, 96]
+    seqs, decay = draw_memory(H, K, V, [a + b + 1 for a, b in zip(lens, more)], K + V)
+    seqs = [{name: t.bfloat16().double() for name, t in d.items()} for d in seqs]
+    want = [plain_memory(d, decay, "none") * 0.8 for d in seqs]
+    slots = [7, 3, 0, 9, 5, 1, 2, 8, 4]
+    state = torch.full((11, 2, H * K * V), float("nan"), device="cuda")
+    state[slots] = 0.0
+    pad = {name: torch.full((1,) + tuple(t.shape[1:]), float("nan"), dtype=F64) for name, t in seqs[0].items()}
+    done = [0] * len(lens)
+    for step, news in enumerate((lens, more, [1] * len(lens))):
+        ctx, runs = step_ctx([(s, p, n) for s, p, n in zip(slots, done, news)], pad_rows=(2,))
+        ctx.ws = Workspace("cuda")
+        rows = {name: torch.cat([seqs[slots.index(s)][name][p:p + n] if s >= 0 else pad[name] for s, p, n in runs]) for name in pad}
+        if step < 2:
+            y = chunk_step(rows, decay, state, ctx, 0.8)
+        else:
+            y = memory_step(rows, decay, state, ctx, "none") * 0.8
+        at = 0
+        for s, p, n in runs:
+            if s >= 0:
+                i = slots.index(s)
+                close(y[at:at + n], want[i][p:p + n], 1e-4, f"step {step}, sequence {i}")
+            at += n
+        done = [a + n for a, n in zip(done, news)]
+    assert torch.isnan(state[[6, 10]]).all(), "a state of another slot was written"
+
+
+def test_fixed_memory_in_chunks_carries_a_far_token():
+    """What the first of 1,500 tokens wrote under a key that only the last ones ask for."""
+    from vlrf_b200.parts.context import Workspace
+    H, K, V, n = 2, 24, 24, 1500
+    (d,), _ = draw_memory(H, K, V, [n], 5)
+    decay = torch.tensor([0.9995, 0.998], dtype=torch.float32).double()
+    d["k"][0, :, 0], d["k"][1:, :, 0], d["q"][n - 3:] = 4.0, 0.0, 0.0
+    d["q"][n - 3:, :, 0], d["v"][0] = 3.0, 5.0
+    d = {name: t.bfloat16().double() for name, t in d.items()}
+    want = plain_memory(d, decay, "none")
+    state = torch.zeros(2, 2, H * K * V, device="cuda")
+    ctx, _ = step_ctx([(1, 0, n)])
+    ctx.ws = Workspace("cuda")
+    got = chunk_step(d, decay, state, ctx)
+    close(got, want, 1e-4, "all")
+    close(got[n - 3:], want[n - 3:], 1e-4, "the far token")
+
+
+@pytest.mark.parametrize("M,N,K", [(70, 96, 64), (300, 200, 128), (129, 37, 72), (2000, 640, 256)])
+def test_a_product_with_silu_in_its_epilogue(M, N, K):
+    from vlrf_b200.csrc import KernelError, ops
+    g = torch.Generator().manual_seed(M)
+    x, w = torch.randn(M, K, generator=g).bfloat16(), (3 * torch.randn(N, K, generator=g) / K ** 0.5).bfloat16()
+    want = F.silu(x.double() @ w.double().T)
+    for od, t in ((torch.bfloat16, 5e-3), (torch.float32, 1e-5)):
+        out = torch.full((M, N), float("nan"), dtype=od, device="cuda")
+        ops.linear(dev(x), dev(w), None, out, act="silu")
+        close(out, want, t, f"to {od}")
+    big = torch.full((M, K), 60.0).bfloat16()              # (both ends: sums of some thousand, and of minus some thousand)
+    out = torch.zeros(M, N, dtype=torch.bfloat16, device="cuda")
+    ones = torch.ones(N, K).bfloat16()
+    ones[::2] = -1.0
+    ops.linear(dev(big), dev(ones), None, out, act="silu")
+    assert float(out[:, ::2].float().abs().max()) == 0.0
+    close(out[:, 1::2], (60.0 * K * torch.ones(M, N // 2)).double(), 5e-3, "large")
+    with pytest.raises(KernelError, match="epilogue"):
+        ops.linear(dev(x[:8]), dev(w), None, out[:8], act="silu")
+
+
 @pytest.mark.parametrize("dt", DT)
 @pytest.mark.parametrize("H,V", [(1, 700), (1, 1024), (1, 2048), (1, 513), (2, 3000), (1, 8192), (1, 9001), (3, 516)])
 def test_the_read_out_of_wide_rows(H, V, dt):

@@ -134,6 +134,9 @@ _SIGNATURES = {
         _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_float, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
         _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
         "vlrf_matrix_state_force": [_c_int, _c_int],
+        "vlrf_fixed_state_chunks_takes": [_c_int] * 7,
+        "vlrf_fixed_state_chunks": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_int,
+        _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
         "vlrf_conv_unit": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p,
         _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
         "vlrf_lowrank_rows": [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_float, _c_int,

@@ -165,6 +165,8 @@ __device__ __forceinline__ float gelu_erf_f(float x) {
 __device__ __forceinline__ float relu2_f(float x) { const float r = fmaxf(x, 0.f); return r * r; }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f(x); }
+// x · sigmoid(x) for results that are rounded to bfloat16 anyway
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 template <int ACT> __device__ __forceinline__ float apply_act(float x) {
     if (ACT == VLRF_ACT_GELU_TANH) return gelu_tanh_f(x);
     if (ACT == VLRF_ACT_GELU_ERF) return gelu_erf_f(x);
@@ -202,6 +204,7 @@ template <typename OT, int ACT> __device__ __forceinline__ float apply_act_const
     if (ACT == VLRF_ACT_GELU_TANH) return sizeof(OT) == 2 ? gelu_tanh_fast(x) : gelu_tanh_f(x);
     if (ACT == VLRF_ACT_GELU_ERF) return gelu_erf_f(x);
     if (ACT == VLRF_ACT_RELU2) return relu2_f(x);
+    if (ACT == VLRF_ACT_SILU) return sizeof(OT) == 2 ? silu_fast(x) : silu_f(x);
     return x;
 }
 __device__ __forceinline__ float apply_act_rt(float x, int act) {

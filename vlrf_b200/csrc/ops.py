@@ -101,7 +101,7 @@ def layernorm(x, gamma, beta, eps: float, out, rows=None) -> None:
 def linear(x, w, bias, out, *, act=None, residual=None, rows: int | None = None, kv_scatter=None,
            stats: "RowStats | None" = None) -> bool:
     """out = act(x · wᵀ + bias) (+ residual).  x [M,K], w [N,K] (same dtype), bias/residual float32,
-    out [M,N] float32 or bfloat16.  `rows` limits M to the first rows of x/out/residual.  `kv_scatter`
+    out [M,N] float32 or bfloat16.  act: "gelu_tanh", "gelu_erf", "relu2"; "silu" where `linear_takes_silu` says so.  `rows` limits M to the first rows of x/out/residual.  `kv_scatter`
     (see linear_layernorm) asks the kernel to write K/V columns into a cache as well; the return value
     says whether it did (only the tensor-core kernels can).  `stats`: where the statistics of float32 result rows
     are left when the kernel that takes the shape computes them (and where stale ones of `out` are forgotten)."""
@@ -123,7 +123,16 @@ def linear(x, w, bias, out, *, act=None, residual=None, rows: int | None = None,
         raise KernelError("linear: float32 input gives float32 output")
     if stats is not None:
         stats.written(out)
+    if act == "silu":
+        if not linear_takes_silu(x.dtype, M, N, K):
+            raise KernelError(f"linear: no product of {M} x {N} x {K} in {x.dtype} takes x·sigmoid(x) in its epilogue")
+        return _linear_dispatch(x, w, bias, out, GATE[act], residual, M, N, K, kv_scatter, stats)
     return _linear_dispatch(x, w, bias, out, ACT[act], residual, M, N, K, kv_scatter, stats)
+
+
+def linear_takes_silu(dtype: torch.dtype, M: int, N: int, K: int) -> bool:
+    """Whether `linear` of this shape runs on the many-row tensor-core kernel, whose epilogue takes x·sigmoid(x)."""
+    return dtype == torch.bfloat16 and M > SKINNY_MAX_ROWS and K % 8 == 0 and USE_TCGEN05
 
 
 #: head sizes that the attention kernels take (each checks it again; parts refuse others when they are built)
@@ -1264,6 +1273,39 @@ def matrix_state_scan(kind: str, q, k, v, state, ctx, y, n_heads: int, n_groups:
          _ptr(s0), ld(s0), _ptr(s1), ld(s1), float(q_scale), float(cap), _ptr(state), state.shape[2], _ptr(ctx.seq_slot),
          _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(y), ld(y), _ptr(den), ctx.n_seqs, ctx.max_new, n_heads, n_groups, rows, cols,
          GATE["silu"] if input_act == "silu" else 0, _stream())
+
+
+#: prompts of the fixed-decay recurrence in chunks on the tensor cores where the sizes are taken (off: token by token); the fewest
+#: tokens of a step's longest run for which that pays, and the most scratch it may ask for
+FIXED_CHUNKS, FIXED_CHUNKS_MIN_RUN, FIXED_CHUNKS_MAX_BYTES = True, 32, 8 << 30
+
+
+def fixed_state_chunks_takes(dtype: torch.dtype, ctx, n_heads: int, rows: int, cols: int, state_row: int) -> bool:
+    """Whether a step's recurrence with a fixed decay runs in chunks (inputs as one product's bfloat16 rows [q | k | v])."""
+    if dtype != torch.bfloat16 or not FIXED_CHUNKS or ctx.max_new < FIXED_CHUNKS_MIN_RUN:
+        return False
+    if (ctx.n_tokens // 64 + ctx.n_seqs) * n_heads * rows * cols * 4 > FIXED_CHUNKS_MAX_BYTES:
+        return False
+    from . import library
+    ld = n_heads * (2 * rows + cols)
+    return bool(library().vlrf_fixed_state_chunks_takes(rows, cols, ld, ld, ld, n_heads * cols, state_row))
+
+
+def fixed_state_chunks(q, k, v, decay, state, ctx, y, n_heads: int, rows: int, cols: int, q_scale: float = 1.0) -> None:
+    """The recurrence S ← a S + k vᵀ, o = Sᵀ q of a prompt step in chunks (see the kernel library's header): bfloat16 q, k [T, H·rows],
+    v [T, H·cols] (column ranges of wider rows), decay float32 [H], state [slots, 2, state_row], y float32 [T, H·cols]."""
+    T = ctx.n_tokens
+    for name, t, n in (("q", q, n_heads * rows), ("k", k, n_heads * rows), ("v", v, n_heads * cols), ("y", y, n_heads * cols)):
+        _rows(t, name, torch.float32 if name == "y" else torch.bfloat16)
+        if t.shape[0] < T or t.shape[1] < n:
+            raise KernelError(f"fixed_state_chunks: {name} does not match")
+    _dev(decay, "decay", torch.float32); _dev(state, "state", torch.float32)
+    if decay.numel() != n_heads or state.dim() != 3 or state.shape[1] != 2:
+        raise KernelError("fixed_state_chunks: one decay per head, and the state is [slots, 2, row]")
+    scratch = ctx.ws.get("fixed_state_chunks", (T // 64 + ctx.n_seqs) * n_heads, rows * cols, torch.float32)
+    call("vlrf_fixed_state_chunks", _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(decay), float(q_scale), _ptr(scratch),
+         _ptr(state), state.shape[2], _ptr(ctx.seq_slot), _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(y), y.stride(0), ctx.n_seqs, ctx.max_new,
+         n_heads, rows, cols, _stream())
 
 
 def conv_unit(proj, x_off: int, weight, state, conv_off: int, ctx, out, kq, n_heads: int, n_groups: int, rows: int, cols: int) -> None:

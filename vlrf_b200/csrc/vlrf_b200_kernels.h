@@ -36,8 +36,8 @@ extern "C" {
 #define VLRF_ACT_GELU_TANH 1
 #define VLRF_ACT_GELU_ERF 2
 #define VLRF_ACT_RELU2 3          // relu(x)^2
-#define VLRF_ACT_LAST_FUSED 3     // the last activation that the products' epilogues take
-#define VLRF_ACT_SILU 4           // x * sigmoid(x): vlrf_gate_mul only
+#define VLRF_ACT_LAST_FUSED 3     // the last activation that every product's epilogue takes
+#define VLRF_ACT_SILU 4           // x * sigmoid(x): vlrf_gate_mul, and of the products vlrf_gemm_tcgen05
 #define VLRF_ACT_SIGMOID 5        // vlrf_gate_mul only
 #define VLRF_ACT_RELU 6           // max(x, 0): vlrf_gate_mul only
 
@@ -327,6 +327,13 @@ int vlrf_matrix_state_scan(int kind, const float* q, int ldq, const float* k, in
                            int ld_decay, const float* s0, int ld_s0, const float* s1, int ld_s1, float q_scale, float cap, float* state,
                            int state_row, const int* seq_slot, const int* seq_start, const int* seq_pos0, float* y, int ldy, float* den,
                            int n_seqs, int max_new, int H, int G, int K, int V, int input_act, cudaStream_t stream);
+// kind 3 over prompts on the tensor cores, 64 tokens at a time (fixed_state_chunks.cu): q, k, v bfloat16 (activated already), scratch
+// float32 (vlrf_fixed_state_chunks_scratch numbers), the rest as above.  K ≤ 256, K and V multiples of 8.
+int vlrf_fixed_state_chunks_takes(int K, int V, int ldq, int ldk, int ldv, int ldy, int state_row);
+long long vlrf_fixed_state_chunks_scratch(int T, int n_seqs, int H, int K, int V);
+int vlrf_fixed_state_chunks(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv, const float* decay, float q_scale,
+                            float* scratch, float* state, int state_row, const int* seq_slot, const int* seq_start, const int* seq_pos0,
+                            float* y, int ldy, int n_seqs, int max_new, int H, int K, int V, cudaStream_t stream);
 int vlrf_matrix_state_force(int columns, int warps);    // for measurements and tests: columns a lane, warps a CTA (0: chosen)
 // Convolution, x·sigmoid(x) and unit norms of q and k over columns [q: G·K | k: G·K | v: H·V] of the float32 rows `proj`; out
 // [T][2·G·K + H·V]; kq [T][G] = k · q; the kept inputs lie at conv_off of the state rows.

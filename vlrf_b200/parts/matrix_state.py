@@ -204,7 +204,9 @@ class DeltaMemory(MatrixStateMixer):
 @register_part("mixer", "fixed_memory")
 class FixedMemory(MatrixStateMixer):
     """q = silu(W_q h), k = silu(W_k h), v = silu(W_v h); decay: one number per head; the concatenated heads normed as one row
-    (a weight of heads·vdim numbers) times sigmoid(W_g h).  The activation runs inside the recurrence's kernels."""
+    (a weight of heads·vdim numbers) times sigmoid(W_g h).  Over prompts in bfloat16 the activation is the input product's
+    epilogue and the recurrence runs in chunks on the tensor cores (csrc/fixed_state_chunks.cu); elsewhere it goes token by
+    token with the activation inside the recurrence's kernels."""
 
     def __init__(self, w_q, w_k, w_v, w_g, norm_w, w_out, *, n_heads: int, dim: int, vdim: int, decay, eps: float, out_factor: float = 1.0):
         what = "fixed memory"
@@ -224,3 +226,20 @@ class FixedMemory(MatrixStateMixer):
         ops.matrix_state_scan("fixed", cols(proj, "q"), cols(proj, "k"), cols(proj, "v"), view.state, ctx, y, H, H, K, V, q_scale=1.0,
                               decay=self.decay, input_act="silu")
         ops.head_rows(y, self.norm_w, cols(proj, "g"), "sigmoid", merged, T, 1, H * V, self.eps, factor)
+
+    def forward(self, h, x: torch.Tensor, ctx: StepContext, view, writes_cache: bool = True, accumulate: bool = True) -> None:
+        T, ws, H, K, V, n = ctx.n_tokens, ctx.ws, self.n_heads, self.dim, self.vdim, self.at["g"][0]
+        if not (ops.fixed_state_chunks_takes(ctx.act_dtype, ctx, H, K, V, view.state.shape[2]) and ops.linear_takes_silu(h.dtype, T, n, h.shape[1])):
+            super().forward(h, x, ctx, view, writes_cache, accumulate)
+            return
+        self._own_state(writes_cache)
+        qkv = ws.get("fixed_memory_qkv", T, n, ctx.act_dtype)
+        ops.linear(h, self.in_weight[:n], None, qkv, act="silu")
+        gate = ws.get("fixed_memory_gate", T, H * V, torch.float32)
+        ops.linear(h, self.in_weight[n:], None, gate)
+        y = ws.get("matrix_state_y", T, H * V, torch.float32)
+        cols = lambda name: qkv[:, self.at[name][0]:self.at[name][1]]   # noqa: E731
+        ops.fixed_state_chunks(cols("q"), cols("k"), cols("v"), self.decay, view.state, ctx, y, H, K, V)
+        merged = ws.get("matrix_state_merged", T, self.merged_width, ctx.act_dtype)
+        ops.head_rows(y, self.norm_w, gate, "sigmoid", merged, T, 1, H * V, self.eps, self.out_factor)
+        ops.linear(merged, self.out_weight, None, x, residual=x if accumulate else None)
